@@ -61,6 +61,9 @@ class CacheNeeds:
     # a state that stays the run's own where it reads another run's cache (what a block
     # keeps beside its mixer: the last inputs of a short convolution, say)
     own_state: StateSpec | None = None
+    # further states beside ``state``: (name, StateSpec) each (a convolution's last inputs, a
+    # normaliser, a running maximum); the mixer finds them by name in ``CacheView.states``
+    states: tuple = ()
 
 
 @dataclass
@@ -132,6 +135,8 @@ class CacheManager:
         by_spec: dict[PagedKVSpec, LayerGroup] = {}
         self._own_state: dict[int, object] = {}  # run -> its own state tensor, never shared
         self._own_state_specs: dict[int, StateSpec] = {}
+        self._named_states: dict[int, dict] = {}      # run -> {name: state tensor}
+        self._named_state_specs: dict[int, tuple] = {}
         for run, need in enumerate(needs):
             if need is not None and getattr(need, "own_state", None) is not None:
                 self._own_state_specs[run] = need.own_state
@@ -149,6 +154,8 @@ class CacheManager:
                 self._run_group[run] = (group.index, len(group.units) - 1)
             if need.state is not None:
                 self._state_specs[run] = need.state
+            if getattr(need, "states", ()):
+                self._named_state_specs[run] = tuple(need.states)
         for run, source in self.shares.items():
             if source not in self._run_group and source not in self._state_specs:
                 raise ValueError(f"run {run} shares the cache of run {source}, which keeps none")
@@ -191,6 +198,11 @@ class CacheManager:
             self._own_state[run] = torch.zeros(
                 (self.max_requests + 1, *spec.shape), dtype=getattr(torch, spec.dtype), device=self.device
             )
+        for run, named in self._named_state_specs.items():
+            self._named_states[run] = {
+                name: torch.zeros((self.max_requests + 1, *spec.shape), dtype=getattr(torch, spec.dtype), device=self.device)
+                for name, spec in named
+            }
 
     def bytes_per_token(self) -> int:
         """Bytes of keys and values one token occupies over all groups (unwindowed view)."""
@@ -233,6 +245,7 @@ class CacheManager:
             owns=run not in self.shares,
             state=self.state_of_run(run),
             own_state=self._own_state.get(run),
+            states=self._named_states.get(self.shares.get(run, run), {}),
         )
 
     def state_of_run(self, run: int):
@@ -259,7 +272,8 @@ class CacheManager:
         if key in self._requests:
             raise ValueError(f"request {key!r} is already live")
         slot = self.slots.lease()
-        for state in (*self._run_state.values(), *self._own_state.values()):
+        named = (state for states in self._named_states.values() for state in states.values())
+        for state in (*self._run_state.values(), *self._own_state.values(), *named):
             state[slot].zero_()
         entry = RequestCache(key, slot, 0, [BlockTable() for _ in self.groups])
         self._requests[key] = entry

@@ -1,6 +1,7 @@
 """Configuration: part specs, the Qwen3 config, engine settings and the registry."""
 
 from .engine import EngineConfig, SchedulerConfig
+from .lofuvik import LofuvikConfig
 from .nuvivik import NuvivikConfig
 from .qwen3 import Qwen3Config
 from .registry import (
@@ -12,6 +13,7 @@ from .registry import (
 )
 from .specs import (
     AttentionSpec,
+    DeltaRuleSpec,
     DenseMLPSpec,
     DifferentialSpec,
     GatedMLPSpec,
@@ -20,6 +22,7 @@ from .specs import (
     LayerNormSpec,
     LayerSpec,
     LinearRecurrenceSpec,
+    MatrixMemorySpec,
     ModelSpec,
     NoPositionSpec,
     NormSpec,
@@ -28,7 +31,9 @@ from .specs import (
     RoutedMLPSpec,
     RunSpec,
     SandwichConvSpec,
+    SideBySideSpec,
     StreamMixSpec,
+    WKVSpec,
 )
 from .tekilorn import TekilornConfig
 from .zabutar import ZabutarConfig
@@ -57,9 +62,15 @@ register_architecture(
     replace=True,
 )
 
+register_architecture(
+    Architecture("Lofuvik", LofuvikConfig.from_dict, LofuvikConfig.to_model_spec),
+    replace=True,
+)
+
 __all__ = [
     "Architecture",
     "AttentionSpec",
+    "DeltaRuleSpec",
     "DenseMLPSpec",
     "DifferentialSpec",
     "EngineConfig",
@@ -69,6 +80,8 @@ __all__ = [
     "LayerNormSpec",
     "LayerSpec",
     "LinearRecurrenceSpec",
+    "LofuvikConfig",
+    "MatrixMemorySpec",
     "ModelSpec",
     "NoPositionSpec",
     "NormSpec",
@@ -80,8 +93,10 @@ __all__ = [
     "RunSpec",
     "SandwichConvSpec",
     "SchedulerConfig",
+    "SideBySideSpec",
     "StreamMixSpec",
     "TekilornConfig",
+    "WKVSpec",
     "ZabutarConfig",
     "ZofadraConfig",
     "architecture_of",

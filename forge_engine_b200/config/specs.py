@@ -70,6 +70,12 @@ class RotarySpec:
     # True: theta^(-2j / rotary_dim) is worked out in 64-bit and rounded once (always so with
     # ``interleaved`` or ``scaling``); False: in 32-bit throughout, as Qwen3's own code does.
     exact_frequencies: bool = False
+    # None, or (factor, original, fast, slow): frequency f_i becomes f_i / factor * r_i + f_i * (1 - r_i)
+    # with a ramp r_i = clamp((i - lo) / max(hi - lo, 0.001), 0, 1) between the dimensions that turn
+    # ``fast`` and ``slow`` times within ``original`` positions, dim(t) = rotary_dim *
+    # ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)),
+    # rotary_dim - 1); cosine and sine are multiplied by 0.1 ln(factor) + 1 ("YaRN").
+    yarn: tuple | None = None
 
 
 @dataclass(frozen=True)
@@ -137,6 +143,12 @@ class AttentionSpec:
     qk_norm_weight: bool = True
     # True (per-head ``qk_norm`` only): the norm is taken of the rotated head, not before the rotation.
     qk_norm_after_rotation: bool = False
+    # True: tensor ``sink`` [heads]; exp(sink_h) joins the denominator of head h's softmax once,
+    # with no key and no value, neither scaled nor capped.
+    sink: bool = False
+    # True: the heads' outputs are multiplied element by element by sigmoid(W x), x the mixer's input;
+    # the checkpoint holds ``gate_proj.weight`` [heads * v_head_dim, hidden].  (Not with ``head_gate``.)
+    output_gate: bool = False
 
 
 @dataclass(frozen=True)
@@ -216,6 +228,77 @@ class GatedRecurrenceSpec:
 
 
 @dataclass(frozen=True)
+class WKVSpec:
+    """Time mixing with a matrix state per head whose decay depends on the token, per key channel.
+    Every projection s of r, k, v, g, w reads h + (h' - h) mu_s, h' being the row of the token
+    before; w = exp(-exp(A tanh(B mix_w) + base)); o_t = (S + diag(u) k v^T)^T r, then
+    S <- diag(w) S + k v^T; each head's o is divided by its root mean square, the heads are
+    weighted, multiplied by silu(W_g mix_g) and projected.  ``rank``: rows of B (None: the stored
+    tensor says)."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    norm_eps: float
+    rank: int | None = None
+    kind: str = "wkv"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
+class DeltaRuleSpec:
+    """The gated delta rule: S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q per head.
+    q, k [num_kv_heads * head_dim] (shared by groups of heads) and v pass a causal convolution over
+    time with ``taps`` taps per channel and silu; q and k are unit vectors per head (q times
+    head_dim^(-1/2)); beta = sigmoid(W_b x), g = exp(-exp(A_log) softplus(W_a x + dt_bias)) per
+    head.  Each head's o is divided by its root mean square, weighted (one vector for all heads),
+    multiplied by silu(W_g x) and projected."""
+
+    hidden_size: int
+    num_heads: int
+    num_kv_heads: int
+    head_dim: int
+    v_head_dim: int
+    taps: int
+    norm_eps: float
+    kind: str = "delta_rule"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
+class MatrixMemorySpec:
+    """A matrix memory with exponential gates: per head a log input gate i = c tanh((W_i x + b_i) / c)
+    and a log forget gate f = logsigmoid(c tanh((W_f x + b_f) / c)), c = ``gate_cap``; with the running
+    maximum m_t = max(f + m_(t-1), i) (from zero on) S_t = e^(f + m_(t-1) - m_t) S_(t-1) + e^(i - m_t)
+    k v^T, n_t likewise with k alone, o = S^T q / (max(|n . q|, e^(-m_t)) + 1e-6), q times
+    head_dim^(-1/2).  Each head's o is divided by its root mean square, the heads are weighted,
+    multiplied by sigmoid(W_g x) and projected."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    gate_cap: float
+    norm_eps: float
+    kind: str = "matrix_memory"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
+class SideBySideSpec:
+    """Two mixers that read the same input; the result is half the sum of their outputs, each
+    divided by its root mean square over the width and weighted (tensors ``left.<name>`` and
+    ``right.<name>`` of the mixers, ``left.out`` and ``right.out`` [hidden] of the norms)."""
+
+    hidden_size: int
+    left: object
+    right: object
+    norm_eps: float
+    kind: str = "side_by_side"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
 class DenseMLPSpec:
     """down(act(up(x) + b_up)) + b_down, no gate.  ``activation`` "xielu": with two learned
     numbers p, q (tensor ``act`` [2]) act(z) = softplus(p) z^2 + z / 2 above zero and
@@ -283,13 +366,16 @@ class RoutedMLPSpec:
     # What a group is worth: "max" - its largest choice score; "top2" - the sum of its two
     # largest (of its one, where a group is a single expert).
     group_score: str = "max"
+    # True: tensor ``router.b`` [router outputs] is added to the router's logits (choice and weights).
+    router_bias: bool = False
 
 
 @dataclass(frozen=True)
 class LayerSpec:
     """One block: which norm, mixer and feed-forward it has and how they are wired.
 
-    ``arrangement`` "pre_norm": h += mixer(norm1(h)); h += ffn(norm2(h)).
+    ``arrangement`` "pre_norm": h += mixer(norm1(h)); h += ffn(norm2(h)).  "parallel": with
+    y = norm1(h), h += mixer(y) + ffn(y) (no ``post_norm``).
     ``names`` maps the roles (input_norm, mixer, post_norm, ffn) to the tensor-name
     prefix of this layer's weights in a checkpoint.
     """
@@ -359,6 +445,9 @@ class RunSpec:
     # None, or (tensor name, row): that row of a [rows, hidden] tensor of the checkpoint is
     # added to the residual stream right before this run.
     shift: tuple | None = None
+    # True: the embedding output (the stream before the first run) is added to the residual stream
+    # right before this run.
+    add_embedding: bool = False
 
 
 @dataclass(frozen=True)

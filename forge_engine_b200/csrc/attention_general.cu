@@ -231,6 +231,7 @@ struct GeneralAttn {
   long long o_part_stride;  //   o_part_stride * m elements further on
   const float* gate;        // or null: the row (token, head) is multiplied by sigmoid(gate[token * gate_stride + head])
   long long gate_stride;
+  int gate_dim;             // above zero: a gate per element, gate[token * gate_stride + head * gate_dim + element]
   int out_f32;              // the output is 32-bit whatever the cache holds
   const float* sinks;       // or null: per query head a number whose exponential joins the softmax's
                             //   denominator once (unscaled, uncapped), with no key and no value
@@ -395,7 +396,10 @@ attention_general_kernel(GeneralAttn a, int* status) {
       den = fmaf(part_l[w * RMAX + r], f, den);
     }
     float value = den > 0.f ? num / den : 0.f;
-    if (a.gate) value *= 1.f / (1.f + expf(-a.gate[(size_t)token * a.gate_stride + head0 + r]));
+    if (a.gate) {
+      const size_t g = (size_t)token * a.gate_stride + (a.gate_dim > 0 ? (size_t)(head0 + r) * a.gate_dim + d : (size_t)(head0 + r));
+      value *= 1.f / (1.f + expf(-a.gate[g]));
+    }
     const size_t at = (size_t)token * a.o_token_stride + (size_t)(head0 + r) * a.o_head_stride + (size_t)part * a.o_part_stride + d;
     if (a.out_f32) ((float*)a.out)[at] = value;
     else ((T*)a.out)[at] = from_float<T>(value);
@@ -462,7 +466,7 @@ FE_EXPORT int fe_attention_general(const void* q, long long q_token_stride, long
                                    const float* dist_bias, int dist_len, int window,
                                    float scale, int keep_first, float softcap, float temp_coef, int temp_every,
                                    int parts, long long q_part_stride, int k_part_stride, long long o_part_stride,
-                                   const float* gate, long long gate_stride, int out_f32, const float* sinks,
+                                   const float* gate, long long gate_stride, int gate_dim, int out_f32, const float* sinks,
                                    int n_tokens, int* status, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (parts < 1) parts = 1;
@@ -472,7 +476,7 @@ FE_EXPORT int fe_attention_general(const void* q, long long q_token_stride, long
   GeneralAttn a{q, q_token_stride, q_head_stride, k_cache, k_row, k_dim, v_cache, v_row, v_dim, out, o_token_stride,
                 o_head_stride, block_table, max_pages, page_size, num_pages, num_kv_heads, num_q_heads, positions,
                 token_entry, slopes, dist_bias, dist_len, window, scale, keep_first, softcap, temp_coef, temp_every, parts, q_part_stride,
-                k_part_stride, o_part_stride, gate, gate_stride, out_f32, sinks};
+                k_part_stride, o_part_stride, gate, gate_stride, gate_dim, out_f32, sinks};
   if (dtype == FE_DTYPE_F32) return dispatch_general<float>(a, n_tokens, status, stream);
   if (dtype == FE_DTYPE_BF16) return dispatch_general<bf16>(a, n_tokens, status, stream);
   return FE_ERR_BAD_DTYPE;

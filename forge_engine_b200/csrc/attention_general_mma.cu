@@ -54,7 +54,7 @@ struct Params {
   // what the plain layer does not have (off when zero / null); see GeneralAttn in attention_general.cu
   int keep_first; float softcap, temp_coef; int temp_every;
   int parts; long long q_ps; int k_ps; long long o_ps;
-  const float* gate; long long gate_stride; int out_f32;
+  const float* gate; long long gate_stride; int gate_dim; int out_f32;
   int row_hi;      // above zero: entries with more rows (new tokens x heads per kv head) are left to another kernel
   const float* sinks;   // or null: per query head a number whose exponential joins the denominator once
 };
@@ -342,7 +342,16 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
       // every score makes the sum infinite and the row zero, which is its limit
       const float l_all = p.sinks ? l_run[h] + exp2f(p.sinks[head] * LOG2E - m_run[h]) : l_run[h];
       float inv = l_all > 0.f ? 1.f / l_all : 0.f;
-      if (p.gate) inv *= sigmoidf(p.gate[(size_t)token * p.gate_stride + head]);
+      if (p.gate && p.gate_dim == 0) inv *= sigmoidf(p.gate[(size_t)token * p.gate_stride + head]);
+      if (p.gate && p.gate_dim > 0) {
+        // a gate per element
+        const float* gate = p.gate + (size_t)token * p.gate_stride + (size_t)head * p.gate_dim + vcol0 + pair * 2;
+#pragma unroll
+        for (int n = 0; n < DVW / 8; ++n) {
+          o[n][2 * h] *= sigmoidf(gate[n * 8]);
+          o[n][2 * h + 1] *= sigmoidf(gate[n * 8 + 1]);
+        }
+      }
       if (p.out_f32) {
         float* dst = reinterpret_cast<float*>(p.out) + at;
 #pragma unroll
@@ -423,7 +432,7 @@ __global__ void __launch_bounds__(128) attention_mma_merge_kernel(Params p) {
     const int rho = tile * BM + r;
     const int token = t_begin + rho / p.groups, head = kvh * p.groups + rho % p.groups;
     float value = num * inverse[lr];
-    if (p.gate) value *= sigmoidf(p.gate[(size_t)token * p.gate_stride + head]);
+    if (p.gate) value *= sigmoidf(p.gate[(size_t)token * p.gate_stride + (p.gate_dim > 0 ? (size_t)head * p.gate_dim + d : (size_t)head)]);
     const size_t at = (size_t)token * p.o_ts + (size_t)head * p.o_hs + (size_t)part * p.o_ps + d;
     if (p.out_f32) reinterpret_cast<float*>(p.out)[at] = value;
     else reinterpret_cast<bf16*>(p.out)[at] = __float2bfloat16_rn(value);
@@ -447,7 +456,7 @@ FE_EXPORT int GM_NAME(fe_attention_gmma_)(const void* q, long long q_ts, long lo
                                           int window, float scale, int splits,
                                           float* workspace, int keep_first, float softcap, float temp_coef,
                                           int temp_every, int parts, long long q_ps, int k_ps, long long o_ps,
-                                          const float* gate, long long gate_stride, int out_f32, int row_hi,
+                                          const float* gate, long long gate_stride, int gate_dim, int out_f32, int row_hi,
                                           const float* sinks, int* status, cudaStream_t stream) {
   if (entries <= 0 || max_new <= 0) return 0;
   if (parts < 1) parts = 1;
@@ -464,7 +473,7 @@ FE_EXPORT int GM_NAME(fe_attention_gmma_)(const void* q, long long q_ts, long lo
   Params p{(const bf16*)q, q_ts, q_hs, (const bf16*)k_cache, k_row, (const bf16*)v_cache, v_row, out, o_ts, o_hs,
            block_table, max_pages, page_size, num_pages, nkv, groups, cu_tokens, starts, slopes, dist_bias, dist_len, window, scale,
            splits, tiles, workspace, keep_first, softcap, temp_coef, temp_every, parts, q_ps, k_ps, o_ps, gate,
-           gate_stride, out_f32, row_hi, sinks};
+           gate_stride, gate_dim, out_f32, row_hi, sinks};
   static bool configured = false;
   if (!configured) {
     const cudaError_t rc = cudaFuncSetAttribute(attention_mma_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)SMEM_BYTES);

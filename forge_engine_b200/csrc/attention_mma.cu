@@ -69,10 +69,14 @@ struct AttnParams {
                          // 2: clusters of 8 splits do, and the clusters' results go through the workspace
   // The tcgen05 prefill kernel only (off when zero / null): with a window, keys below
   // keep_first stay visible to every query; row (token, head) of the output is multiplied by
-  // sigmoid(gate[token * gate_stride + head]).
+  // sigmoid(gate[token * gate_stride + head]), or with gate_dim above zero element d by
+  // sigmoid(gate[token * gate_stride + head * gate_dim + d]); exp(sinks[head]) joins the softmax's
+  // denominator once, with no key and no value.
   int keep_first = 0;
   const float* gate = nullptr;
   long long gate_stride = 0;
+  int gate_dim = 0;
+  const float* sinks = nullptr;
   // dist_bias[head * dist_len + min(query position - key position, dist_len - 1)] is added to
   // the score before it is scaled, so the table holds the bias divided by the scale.
   const float* dist_bias = nullptr;
@@ -1188,11 +1192,13 @@ FE_EXPORT int SYM(fe_attention_prefill_tc5_d)(const void* q, int q_stride, void*
                                               int num_pages, int num_kv_heads, int groups, const int* cu_tokens,
                                               const int* starts, int entries, int max_new, int total_tokens, int window,
                                               int keep_first, float scale, const float* gate, long long gate_stride,
-                                              int row_lo, const float* dist_bias, int dist_len, float softcap,
+                                              int gate_dim, int row_lo, const float* dist_bias, int dist_len, float softcap,
+                                              const float* sinks,
                                               int* status, cudaStream_t stream) {
   if (entries <= 0 || max_new * groups <= row_lo) return 0;
   if (dist_bias != nullptr && dist_len < 1) return FE_ERR_BAD_SHAPE;
   if (softcap < 0.f || (softcap > 0.f && dist_bias != nullptr)) return FE_ERR_BAD_SHAPE;
+  if (gate_dim > 0 && (gate_dim != D || ((uintptr_t)gate & 15) || gate_stride % 4)) return FE_ERR_BAD_ALIGN;
   if (entries > 65535 || num_kv_heads > 65535) return FE_ERR_TOO_LARGE;
   if (((uintptr_t)q | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)out) & 15) return FE_ERR_BAD_ALIGN;
   if ((q_stride % 8) != 0) return FE_ERR_BAD_ALIGN;
@@ -1207,7 +1213,7 @@ FE_EXPORT int SYM(fe_attention_prefill_tc5_d)(const void* q, int q_stride, void*
   p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.row_lo = row_lo; p.row_hi = 0x7fffffff;
   p.num_splits = 1; p.ws_acc = nullptr; p.ws_ml = nullptr; p.ws_count = nullptr; p.cluster_merge = 0;
-  p.keep_first = keep_first; p.gate = gate; p.gate_stride = gate_stride;
+  p.keep_first = keep_first; p.gate = gate; p.gate_stride = gate_stride; p.gate_dim = gate_dim; p.sinks = sinks;
   p.dist_bias = dist_bias; p.dist_len = dist_len;
   if (softcap > 0.f) { p.cap_over_scale = softcap / scale; p.scale_over_cap = scale / softcap; }
   CUtensorMap mk, mv, mq;

@@ -531,10 +531,14 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     if (ok) ok = mbar_wait(o_full, 0, abort_flag);
     asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
     if (ok) {
+      // a sink joins the sum in the units of the running maximum (log 2); one that dwarfs every
+      // score makes the sum infinite and the row zero, which is its limit
+      if (p.sinks != nullptr && row_valid)
+        l += exp2f(p.sinks[kvh * p.groups + row % p.groups] * 1.4426950408889634f - m_used);
       float inv = l > 0.f ? 1.f / l : 0.f;
       const int num_q_heads = p.nkv * p.groups;
       const int token = row / p.groups, g = row - token * p.groups;
-      if (p.gate != nullptr && row_valid)
+      if (p.gate != nullptr && p.gate_dim == 0 && row_valid)
         inv *= 1.f / (1.f + expf(-p.gate[(size_t)(tok0 + token) * p.gate_stride + kvh * p.groups + g]));
       bf16* dst = p.out + ((size_t)(tok0 + token) * num_q_heads + kvh * p.groups + g) * D;
 #pragma unroll 1
@@ -547,6 +551,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
             float v8[8];
 #pragma unroll
             for (int e = 0; e < 8; ++e) v8[e] = o[j + e] * inv;
+            if (p.gate != nullptr && p.gate_dim > 0) {
+              float g8[8];
+              load8(p.gate + (size_t)(tok0 + token) * p.gate_stride + (size_t)(kvh * p.groups + g) * p.gate_dim + c + j, g8);
+#pragma unroll
+              for (int e = 0; e < 8; ++e) v8[e] *= 1.f / (1.f + expf(-g8[e]));
+            }
             store8(dst + c + j, v8);
           }
         }

@@ -1,0 +1,436 @@
+// The gated delta rule: a state per head that is decayed and then corrected towards each key's value.
+//
+//     S <- g S;   u = beta (v - S^T k);   S <- S + k u^T;   o = S^T q
+//     beta = sigmoid(zb),  g = exp(-exp(A) softplus(za + b)),   per head
+//
+// q, k and v pass a short causal convolution over time and silu, q and k are made unit vectors per
+// head (q times dk^(-1/2)); groups of heads share a q/k head.  A head's o is divided by its root
+// mean square, weighted and gated.
+//
+//   delta_prepare   convolutions, silu, unit vectors, beta and log g of a token; the last taps - 1
+//                   rows of the convolution's input stay in the request's state.
+//   state_walk      (state_recurrence.cuh) short entries.
+//   delta_solve / delta_chain / state_out   long entries in chunks.  With c_t the sum of log g from the
+//                   chunk's first token up to t and S the state before the chunk, the u of a chunk solve
+//                     u_t + sum_(j < t) L_tj u_j = beta_t (v_t - e^(c_t) S^T k_t),
+//                     L_tj = beta_t e^(c_t - c_j) k_t . k_j,
+//                   a unit lower triangular system.  delta_solve solves it for all chunks side by side, once
+//                   for the right side beta v and once for beta e^c k, so that u = U - W S; delta_chain walks
+//                   the chunks with two products each (u, and the state it leads to); then
+//                     o_t = e^(c_t) S^T q_t + sum_(j <= t) e^(c_t - c_j) (q_t . k_j) u_j.
+#include "state_recurrence.cuh"
+
+// ---------------------------------------------------------------------------
+// delta_prepare
+// ---------------------------------------------------------------------------
+struct DeltaPrepare {
+  const float* proj;        // [tokens, ld]: q, k, v from column 0, zb and za at b_off, a_off
+  long long ld;
+  int b_off, a_off;
+  const float* conv;        // [taps, channels]
+  int taps;
+  float* state;             // [rows, taps - 1, channels], oldest first
+  const int *slots, *cu_tokens, *token_entry;
+  const float *a_log, *dt_bias;     // [heads]
+  int kv_heads, dk, heads, dv;
+  float* out;               // [tokens, channels]: q, k unit vectors, v
+  float* gates;             // [tokens, heads, 2]: beta, log g
+  int n_tokens;
+};
+
+// One token: its channels' convolution from `row(j)` (the input j tokens back, or a null pointer
+// before the start), then unit vectors and gates.
+template <typename F>
+__device__ __forceinline__ void delta_prepare_token(const DeltaPrepare& p, int t, float* buf, F row) {
+  const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv;
+  float* out = p.out + (size_t)t * channels;
+  for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+    float sum = 0.f;
+    for (int j = p.taps - 1; j >= 0; --j) sum = fmaf(p.conv[(size_t)(p.taps - 1 - j) * channels + c], row(j)[c], sum);
+    const float y = sum / (1.f + expf(-sum));
+    if (c < 2 * qk) buf[c] = y;
+    else out[c] = y;
+  }
+  __syncthreads();
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
+  const float q_scale = 1.f / sqrtf((float)p.dk);
+  for (int h = warp; h < 2 * p.kv_heads; h += warps) {
+    float ss = 0.f;
+    for (int d = lane; d < p.dk; d += 32) ss = fmaf(buf[h * p.dk + d], buf[h * p.dk + d], ss);
+    const float inv = (h < p.kv_heads ? q_scale : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+    for (int d = lane; d < p.dk; d += 32) out[h * p.dk + d] = buf[h * p.dk + d] * inv;
+  }
+  for (int h = threadIdx.x; h < p.heads; h += blockDim.x) {
+    const float* src = p.proj + (size_t)t * p.ld;
+    float* dst = p.gates + ((size_t)t * p.heads + h) * 2;
+    dst[0] = 1.f / (1.f + expf(-src[p.b_off + h]));
+    dst[1] = -expf(p.a_log[h]) * sr_softplus(src[p.a_off + h] + p.dt_bias[h]);
+  }
+  __syncthreads();
+}
+
+__global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepare p) {
+  extern __shared__ __align__(16) float buf[];      // q and k of a token
+  pdl_trigger();
+  pdl_wait();
+  const int back = p.taps - 1;
+  if ((int)blockIdx.x < p.n_tokens) {
+    // a token with all its taps inside the step
+    const int t = blockIdx.x;
+    if (t - p.cu_tokens[p.token_entry[t]] < back) return;
+    delta_prepare_token(p, t, buf, [&](int j) { return p.proj + (size_t)(t - j) * p.ld; });
+    return;
+  }
+  // an entry's edge: its first taps - 1 tokens, then the state for the next step
+  const int entry = blockIdx.x - p.n_tokens;
+  const int first = p.cu_tokens[entry], count = p.cu_tokens[entry + 1] - first;
+  if (count <= 0) return;
+  const int channels = 2 * p.kv_heads * p.dk + p.heads * p.dv;
+  float* st = p.state + (size_t)p.slots[entry] * back * channels;
+  for (int i = 0; i < min(count, back); ++i)
+    delta_prepare_token(p, first + i, buf, [&](int j) {
+      return j <= i ? p.proj + (size_t)(first + i - j) * p.ld : (const float*)st + (size_t)(back + i - j) * channels;
+    });
+  // the last taps - 1 rows of (state rows, the step's rows); a channel is one thread's, which reads
+  // a state row only before it overwrites it
+  for (int c = threadIdx.x; c < channels; c += blockDim.x)
+    for (int r = 0; r < back; ++r) {
+      const int at = count + r;
+      st[(size_t)r * channels + c] = at < back ? st[(size_t)at * channels + c] : p.proj[(size_t)(first + at - back) * p.ld + c];
+    }
+}
+
+FE_EXPORT int fe_delta_prepare(const float* proj, long long ld, int b_off, int a_off, const float* conv, int taps, float* state,
+                               const int* slots, const int* cu_tokens, const int* token_entry, const float* a_log,
+                               const float* dt_bias, int kv_heads, int dk, int heads, int dv, float* out, float* gates,
+                               int n_tokens, int n_entries, cudaStream_t stream) {
+  if (n_tokens <= 0) return 0;
+  if (taps < 1 || kv_heads < 1 || heads < 1 || dk < 1 || dv < 1 || heads % kv_heads || (taps > 1 && state == nullptr)) return FE_ERR_BAD_SHAPE;
+  DeltaPrepare p{proj, ld, b_off, a_off, conv, taps, state, slots, cu_tokens, token_entry, a_log, dt_bias, kv_heads, dk, heads, dv, out, gates, n_tokens};
+  const size_t smem = sizeof(float) * (size_t)2 * kv_heads * dk;
+  if (smem > 200 * 1024) return FE_ERR_TOO_LARGE;
+  if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const int rc = fe_launch_dependent(delta_prepare_kernel, dim3(n_tokens + (taps > 1 ? n_entries : 0)), dim3(256), smem, stream, p);
+  return rc ? rc : fe_last_error();
+}
+
+// ---------------------------------------------------------------------------
+// the recurrence
+// ---------------------------------------------------------------------------
+struct Delta {
+  const float* qkv;         // [tokens, channels]
+  long long ld;
+  int kv_heads, per;        // q/k heads; heads per q/k head
+  const float* gates;       // [tokens, heads, 2]
+  // chunk-parallel scratch, per (slot, head)
+  float* w;                 // [dk][SR_LONG]: W transposed
+  float* u;                 // [SR_LONG][dv]: U, then (chain) u
+  float* starts;            // [dk, dv]: the state before the chunk
+
+  static constexpr int VECS = 2, SCALARS = 2, EXTRA = 0;
+  static constexpr bool SCORES = true, NORMALISER = false;
+
+  __device__ __forceinline__ const float* q_row(const StateRun& p, int head, int token) const {
+    return qkv + (size_t)token * ld + (size_t)(head / per) * p.dk;
+  }
+  __device__ __forceinline__ const float* k_row(const StateRun& p, int head, int token) const {
+    return q_row(p, head, token) + (size_t)kv_heads * p.dk;
+  }
+  __device__ __forceinline__ float beta(const StateRun& p, int head, int token) const { return gates[((size_t)token * p.heads + head) * 2]; }
+  __device__ __forceinline__ float log_decay(const StateRun& p, int head, int token) const { return gates[((size_t)token * p.heads + head) * 2 + 1]; }
+
+  __device__ __forceinline__ float* column(const StateRun& p, int slot, int head, int col, size_t* step) const {
+    *step = p.dv;
+    return p.state + ((size_t)slot * p.heads + head) * p.dk * p.dv + col;
+  }
+  __device__ __forceinline__ void begin(const StateRun&, int, int, float*) const {}
+  __device__ __forceinline__ void end(const StateRun&, int, int, const float*) const {}
+  __device__ __forceinline__ void stage(const StateRun& p, int head, int first, int nt, float* vec, int pitch, float* sc) const {
+    for (int i = threadIdx.x; i < nt * p.dk; i += blockDim.x) {
+      const int t = i / p.dk, d = i - t * p.dk;
+      float* dst = vec + t * VECS * pitch + d;
+      dst[0] = q_row(p, head, first + t)[d], dst[pitch] = k_row(p, head, first + t)[d];
+    }
+    for (int t = threadIdx.x; t < nt; t += blockDim.x) {
+      sc[t * SCALARS] = beta(p, head, first + t);
+      sc[t * SCALARS + 1] = expf(log_decay(p, head, first + t));
+    }
+  }
+  template <int KPT>
+  __device__ __forceinline__ float step(float (&S)[KPT], const float* vec, int pitch, const float* sc, float value, int s, int ds) const {
+    const float *qs = vec + s, *ks = qs + pitch;
+    const float g = sc[1];
+    float have = 0.f;
+#pragma unroll
+    for (int i = 0; i < KPT; ++i) {
+      S[i] *= g;
+      have = fmaf(S[i], ks[i * ds], have);
+    }
+    const float u = sc[0] * (value - sr_column_sum(have, ds));
+    float acc = 0.f;
+#pragma unroll
+    for (int i = 0; i < KPT; ++i) {
+      S[i] = fmaf(ks[i * ds], u, S[i]);
+      acc = fmaf(S[i], qs[i * ds], acc);
+    }
+    return sr_column_sum(acc, ds);
+  }
+  __device__ __forceinline__ float scale(const float*, const float*, int) const { return 1.f; }
+
+  // -- chunk form --
+  // sums of log g up to every token of the chunk (tokens past the end keep the last sum)
+  __device__ __forceinline__ void chunk_sums(const StateRun& p, int head, const ChunkAt& at, double* c) const {
+    __shared__ float logs[SR_LONG];
+    if (threadIdx.x < SR_LONG) logs[threadIdx.x] = (int)threadIdx.x < at.count ? log_decay(p, head, at.first + threadIdx.x) : 0.f;
+    __syncthreads();
+    if (threadIdx.x == 0) {
+      double sum = 0.0;
+      for (int t = 0; t < SR_LONG; ++t) {
+        sum += (double)logs[t];
+        c[t] = sum;
+      }
+    }
+    __syncthreads();
+  }
+  __device__ __forceinline__ size_t cell(const StateRun& p, const ChunkAt& at, int head) const { return (size_t)at.slot * p.heads + head; }
+  __device__ __forceinline__ float query(const StateRun& p, int head, const ChunkAt& at, int t, int d) const { return q_row(p, head, at.first + t)[d]; }
+  __device__ __forceinline__ float key(const StateRun& p, int head, const ChunkAt& at, int t, int d) const { return k_row(p, head, at.first + t)[d]; }
+  __device__ __forceinline__ float other(const StateRun& p, int head, const ChunkAt& at, int t, int c) const {
+    return u[(cell(p, at, head) * SR_LONG + t) * p.dv + c];
+  }
+  __device__ __forceinline__ float start(const StateRun& p, int head, const ChunkAt& at, int d, int c) const {
+    return starts[(cell(p, at, head) * p.dk + d) * p.dv + c];
+  }
+  __device__ __forceinline__ void out_begin(const StateRun& p, int head, const ChunkAt& at, double* rt, double* ct, float* ea, float*) const {
+    chunk_sums(p, head, at, rt);
+    if (threadIdx.x < SR_LONG) {
+      const int t = threadIdx.x;
+      ct[t] = -rt[t];
+      ea[t] = t < at.count ? expf((float)rt[t]) : 0.f;
+    }
+  }
+};
+
+// W and U of one chunk of one head: the triangular system solved for the columns of beta e^c k
+// and beta v, a thread per column with the column in registers.
+__global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const StateRun p) {
+  extern __shared__ __align__(16) float smem[];
+  pdl_trigger();
+  pdl_wait();
+  ChunkAt at;
+  if (!sr_locate(p, &at)) return;
+  const int head = blockIdx.x, dk = p.dk, dv = p.dv, tid = threadIdx.x;
+  __shared__ double c[SR_LONG];
+  __shared__ float bt[SR_LONG], be[SR_LONG];
+  float* L = smem;                           // [SR_LONG rows t][SR_LONG]
+  float* kt = L + SR_LONG * SR_LONG;         // [dk][SR_TP]
+  sr_stage_transposed(kt, dk, at.count, [&](int t, int d) { return m.key(p, head, at, t, d); });
+  m.chunk_sums(p, head, at, c);
+  if (tid < SR_LONG) {
+    bt[tid] = tid < at.count ? m.beta(p, head, at.first + tid) : 0.f;
+    be[tid] = bt[tid] * expf((float)c[tid]);
+  }
+  __syncthreads();
+  for (int item = tid; item < 256; item += blockDim.x) {
+    const int row = 4 * (item & 15), col = 4 * (item >> 4);
+    float a[4][4] = {};
+    if (col <= row + 3) sr_mm44(a, kt, SR_TP, kt, SR_TP, dk, row, col);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const int t = row + e;
+      float l[4];
+#pragma unroll
+      for (int b = 0; b < 4; ++b) l[b] = col + b < t ? a[e][b] * bt[t] * expf((float)(c[t] - c[col + b])) : 0.f;
+      store4(L + t * SR_LONG + col, l);
+    }
+  }
+  __syncthreads();
+  const size_t cell = m.cell(p, at, head);
+  for (int i = tid; i < dk + dv; i += blockDim.x) {
+    float x[SR_LONG];
+    if (i < dk) {
+#pragma unroll
+      for (int t = 0; t < SR_LONG; ++t) x[t] = be[t] * kt[i * SR_TP + t];
+    } else {
+      const float* v = p.v + (size_t)at.first * p.v_ld + (size_t)head * dv + (i - dk);
+#pragma unroll
+      for (int t = 0; t < SR_LONG; ++t) x[t] = t < at.count ? bt[t] * v[(size_t)t * p.v_ld] : 0.f;
+    }
+#pragma unroll
+    for (int t = 1; t < SR_LONG; ++t) {
+      const float4* l4 = reinterpret_cast<const float4*>(L + t * SR_LONG);
+      float s0 = 0.f, s1 = 0.f;
+#pragma unroll
+      for (int j = 0; j < t; j += 4) {
+        const float4 l = l4[j >> 2];           // entries at and past the diagonal are zero
+        s0 = fmaf(l.x, x[j], s0);
+        s1 = fmaf(l.y, x[j + 1], s1);
+        s0 = fmaf(l.z, x[j + 2], s0);
+        s1 = fmaf(l.w, x[j + 3], s1);
+      }
+      x[t] -= s0 + s1;
+    }
+    if (i < dk) {
+      float* dst = m.w + (cell * dk + i) * SR_LONG;
+#pragma unroll
+      for (int t = 0; t < SR_LONG; t += 4) store4(dst + t, x + t);
+    } else {
+      float* dst = m.u + cell * SR_LONG * dv + (i - dk);
+#pragma unroll
+      for (int t = 0; t < SR_LONG; ++t) dst[(size_t)t * dv] = x[t];
+    }
+  }
+}
+
+// The chain over an entry's chunks for one head and 32 value columns: u = U - W S, then
+// S <- e^(c_end) S + sum_j e^(c_end - c_j) k_j u_j^T.  The state's columns stay in shared memory.
+// Thread (rg, cg) owns four rows and two columns of a product.
+#define DC_COLS 32
+__device__ __forceinline__ void dc_mm42(float (&acc)[4][2], const float* xt, int ldx, const float* y, int depth, int row, int col) {
+#pragma unroll 8
+  for (int k = 0; k < depth; ++k) {
+    const float4 x = *reinterpret_cast<const float4*>(xt + k * ldx + row);
+    const float2 b = *reinterpret_cast<const float2*>(y + k * DC_COLS + col);
+    acc[0][0] = fmaf(x.x, b.x, acc[0][0]), acc[0][1] = fmaf(x.x, b.y, acc[0][1]);
+    acc[1][0] = fmaf(x.y, b.x, acc[1][0]), acc[1][1] = fmaf(x.y, b.y, acc[1][1]);
+    acc[2][0] = fmaf(x.z, b.x, acc[2][0]), acc[2][1] = fmaf(x.z, b.y, acc[2][1]);
+    acc[3][0] = fmaf(x.w, b.x, acc[3][0]), acc[3][1] = fmaf(x.w, b.y, acc[3][1]);
+  }
+}
+
+__global__ void __launch_bounds__(256) delta_chain_kernel(const Delta m, const StateRun p, int* status) {
+  extern __shared__ __align__(16) float smem[];
+  pdl_trigger();
+  pdl_wait();
+  const int head = blockIdx.x, entry = blockIdx.y, col0 = blockIdx.z * DC_COLS, tid = threadIdx.x;
+  const int first = p.cu_tokens[entry], count = p.cu_tokens[entry + 1] - first;
+  if (count < p.long_from) return;
+  const int slot = p.slots[entry];
+  if (slot < 0 || slot >= p.state_rows) {
+    if (tid == 0 && blockIdx.z == 0) atomicOr(status, FE_STATUS_BAD_PAGE);
+    return;
+  }
+  const int dk = p.dk, dv = p.dv, kp = (dk + 63) / 64 * 64;
+  const int cols = min(DC_COLS, dv - col0);
+  __shared__ float w[SR_LONG], logs[SR_LONG];
+  __shared__ float keep;
+  float* S = smem;                           // [kp][DC_COLS]
+  float* wt = S + kp * DC_COLS;              // [dk][SR_LONG]
+  float* ks = wt + dk * SR_LONG;             // [SR_LONG][kp], weighted
+  float* us = ks + SR_LONG * kp;             // [SR_LONG][DC_COLS]
+  const int row = 4 * (tid & 15), col = 2 * (tid >> 4);
+  float* st = p.state + ((size_t)slot * p.heads + head) * dk * dv + col0;
+  for (int i = tid; i < kp * DC_COLS; i += blockDim.x) {
+    const int d = i / DC_COLS, c = i - d * DC_COLS;
+    S[i] = (d < dk && c < cols) ? st[(size_t)d * dv + c] : 0.f;
+  }
+  const int chunks = (count + SR_LONG - 1) / SR_LONG;
+  for (int chunk = 0; chunk < chunks; ++chunk) {
+    ChunkAt at;
+    at.entry_first = first, at.first = first + chunk * SR_LONG, at.count = min(SR_LONG, count - chunk * SR_LONG);
+    at.slot = sr_slot(first, entry, chunk), at.chunks = chunks;
+    const size_t cell = m.cell(p, at, head);
+    __syncthreads();
+    if (tid < SR_LONG) logs[tid] = tid < at.count ? m.log_decay(p, head, at.first + tid) : 0.f;
+    const float4* wsrc = reinterpret_cast<const float4*>(m.w + cell * dk * SR_LONG);
+    for (int i = tid; i < dk * SR_LONG / 4; i += blockDim.x) reinterpret_cast<float4*>(wt)[i] = wsrc[i];
+    __syncthreads();
+    if (tid < SR_LONG) {
+      // e^(sum of the later logs): summed from the end, so that late tokens keep their precision
+      float after = 0.f;
+      for (int j = at.count - 1; j > tid; --j) after += logs[j];
+      w[tid] = tid < at.count ? expf(after) : 0.f;
+      if (tid == 0) keep = expf(after + logs[0]);
+    }
+    __syncthreads();
+    for (int i = tid; i < SR_LONG * kp; i += blockDim.x) {
+      const int t = i / kp, d = i - t * kp;
+      ks[i] = (t < at.count && d < dk) ? m.key(p, head, at, t, d) * w[t] : 0.f;
+    }
+    float a[4][2] = {};
+    dc_mm42(a, wt, SR_LONG, S, dk, row, col);
+    float* u = m.u + cell * SR_LONG * dv + col0;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+#pragma unroll
+      for (int b = 0; b < 2; ++b) {
+        float x = 0.f;
+        if (col + b < cols) {
+          x = u[(size_t)(row + e) * dv + col + b] - a[e][b];
+          u[(size_t)(row + e) * dv + col + b] = x;
+        }
+        us[(row + e) * DC_COLS + col + b] = x;
+      }
+    // the state before the chunk, for state_out
+    float* dst = m.starts + cell * dk * dv + col0;
+    for (int i = tid; i < dk * DC_COLS; i += blockDim.x) {
+      const int d = i / DC_COLS, c = i - d * DC_COLS;
+      if (c < cols) dst[(size_t)d * dv + c] = S[i];
+    }
+    __syncthreads();
+    for (int d0 = 0; d0 < kp; d0 += 64) {
+      float b[4][2] = {};
+      dc_mm42(b, ks + d0, kp, us, at.count, row, col);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * DC_COLS + col);
+        const float2 old = *s2;
+        *s2 = make_float2(fmaf(keep, old.x, b[e][0]), fmaf(keep, old.y, b[e][1]));
+      }
+    }
+  }
+  __syncthreads();
+  for (int i = tid; i < dk * DC_COLS; i += blockDim.x) {
+    const int d = i / DC_COLS, c = i - d * DC_COLS;
+    if (c < cols) st[(size_t)d * dv + c] = S[i];
+  }
+}
+
+static size_t delta_solve_smem(int dk) { return sizeof(float) * ((size_t)SR_LONG * SR_LONG + (size_t)dk * SR_TP); }
+static size_t delta_chain_smem(int dk) {
+  const size_t kp = (size_t)(dk + 63) / 64 * 64;
+  return sizeof(float) * (kp * DC_COLS + (size_t)dk * SR_LONG + SR_LONG * kp + SR_LONG * DC_COLS);
+}
+static bool delta_chunk_takes(int dk, int dv) {
+  return chunk_takes(dk, dv, true) && delta_solve_smem(dk) <= 200 * 1024 && delta_chain_smem(dk) <= 200 * 1024;
+}
+
+FE_EXPORT long long fe_delta_rule_scratch(int tokens, int entries, int heads, int dk, int dv, int max_new) {
+  const long long need = walk_in_stretches(dk, dv, 0) ? (long long)tokens * heads * dv : 0;
+  if (max_new < SR_LONG_FROM || !delta_chunk_takes(dk, dv)) return need;
+  return (need + 3) / 4 * 4 + sr_slots(tokens, entries) * heads * ((long long)dk * SR_LONG + (long long)SR_LONG * dv + (long long)dk * dv);
+}
+
+FE_EXPORT int fe_delta_rule(const float* qkv, long long ld, const float* gates, const float* gate, long long gate_ld,
+                            const float* norm_w, float eps, float* state, int state_rows, const int* slots,
+                            const int* cu_tokens, void* out, int out_dtype, int entries, int kv_heads, int heads, int dk, int dv,
+                            int tokens, int max_new, float* scratch, int* status, cudaStream_t stream) {
+  if (entries <= 0 || tokens <= 0) return 0;
+  if (heads < 1 || kv_heads < 1 || heads % kv_heads || dk < 1 || dv < 1 || heads > 65535 || entries > 65535) return FE_ERR_BAD_SHAPE;
+  StateRun p{state, state_rows, slots, cu_tokens, heads, dk, dv, 0, qkv + 2 * kv_heads * dk, ld, norm_w, 0, gate, gate_ld, 0, eps, out, nullptr, 0};
+  Delta m{qkv, ld, kv_heads, heads / kv_heads, gates, nullptr, nullptr, nullptr};
+  if (walk_in_stretches(dk, dv, 0)) {
+    p.raw = scratch;
+    scratch = scratch ? scratch + ((size_t)tokens * heads * dv + 3) / 4 * 4 : nullptr;
+  }
+  const bool chunked = max_new >= SR_LONG_FROM && scratch != nullptr && delta_chunk_takes(dk, dv);
+  if (chunked) p.long_from = SR_LONG_FROM;
+  int rc = launch_walk(m, p, out_dtype, entries, tokens, status, stream);
+  if (rc || !chunked) return rc ? rc : fe_last_error();
+  const int chunks = (max_new + SR_LONG - 1) / SR_LONG;
+  if (chunks > 65535) return FE_ERR_TOO_LARGE;
+  const size_t cells = (size_t)sr_slots(tokens, entries) * heads;
+  m.w = scratch;
+  m.u = m.w + cells * dk * SR_LONG;
+  m.starts = m.u + cells * SR_LONG * dv;
+  size_t smem = delta_solve_smem(dk);
+  cudaFuncSetAttribute(delta_solve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  rc = fe_launch_dependent(delta_solve_kernel, dim3(heads, entries, chunks), dim3(128), smem, stream, m, p);
+  if (rc) return rc;
+  smem = delta_chain_smem(dk);
+  cudaFuncSetAttribute(delta_chain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  rc = fe_launch_dependent(delta_chain_kernel, dim3(heads, entries, (dv + DC_COLS - 1) / DC_COLS), dim3(256), smem, stream, m, p, status);
+  if (rc) return rc;
+  rc = launch_out(m, p, out_dtype, entries, chunks, stream);
+  return rc ? rc : fe_last_error();
+}

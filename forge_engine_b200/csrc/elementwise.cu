@@ -58,14 +58,14 @@ FE_EXPORT int fe_embedding(const int* ids, const void* table, int table_dtype, f
 }
 
 // ---------------------------------------------------------------------------
-// x = residual[src] + update[src] (+ shift, one vector for all rows);  residual[src] = x (optional);
+// x = residual[src] + update[src] (+ shift[src], rows shift_stride apart; 0: one vector for all rows);  residual[src] = x (optional);
 // out[r] = x * rsqrt(mean(x^2) + eps) * weight       -- all in 32-bit, one rounding
 // src = row_map ? row_map[r] : r
 // ---------------------------------------------------------------------------
 template <typename TU, typename TO, int PER>
 __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TU* __restrict__ update,
                                    const float* __restrict__ weight, TO* __restrict__ out,
-                                   const int* __restrict__ row_map, const float* __restrict__ shift, int size, float eps,
+                                   const int* __restrict__ row_map, const float* __restrict__ shift, long long shift_stride, int size, float eps,
                                    int write_residual) {
   // PER > 0: every thread keeps its PER elements (strided by blockDim) in registers between
   // the two passes; PER == 0: rows too long for that are read twice.
@@ -77,6 +77,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TU* __res
   float* res = residual + (size_t)src * size;
   const TU* upd = update ? update + (size_t)src * size : nullptr;
   TO* dst = out + (size_t)r * size;
+  if (shift) shift += (size_t)src * shift_stride;
   float ss = 0.f;
   if constexpr (PER > 0) {
     float x[PER > 0 ? PER : 1];
@@ -122,7 +123,7 @@ __global__ void add_rmsnorm_kernel(float* __restrict__ residual, const TU* __res
 template <typename TU, typename TO, int PER>
 __global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const TU* __restrict__ update,
                                        const float* __restrict__ weight, TO* __restrict__ out,
-                                       const int* __restrict__ row_map, const float* __restrict__ shift, int size, float eps,
+                                       const int* __restrict__ row_map, const float* __restrict__ shift, long long shift_stride, int size, float eps,
                                        int write_residual) {
   __shared__ float scratch[33];
   pdl_trigger();
@@ -132,6 +133,7 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const TU* _
   float* res = residual + (size_t)src * size;
   const TU* upd = update ? update + (size_t)src * size : nullptr;
   TO* dst = out + (size_t)r * size;
+  if (shift) shift += (size_t)src * shift_stride;
   const int groups = size >> 2;
   float x[PER][4];
   float ss = 0.f;
@@ -173,13 +175,13 @@ __global__ void add_rmsnorm_vec_kernel(float* __restrict__ residual, const TU* _
 
 FE_EXPORT int fe_add_rmsnorm(float* residual, const void* update, int update_dtype,
                              const float* weight, void* out, int out_dtype, const int* row_map,
-                             const float* shift, int rows, int size, float eps, int write_residual,
+                             const float* shift, long long shift_stride, int rows, int size, float eps, int write_residual,
                              cudaStream_t stream) {
   if (rows <= 0) return 0;
   int rc = 0;
   const int update_bytes = update_dtype == FE_DTYPE_F32 ? 16 : 8, out_bytes = out_dtype == FE_DTYPE_F32 ? 16 : 8;
   if ((size % 4) == 0 && size <= 16384 && ((uintptr_t)residual % 16) == 0 && ((uintptr_t)weight % 16) == 0 &&
-      ((uintptr_t)update % update_bytes) == 0 && ((uintptr_t)out % out_bytes) == 0 && ((uintptr_t)shift % 16) == 0) {
+      ((uintptr_t)update % update_bytes) == 0 && ((uintptr_t)out % out_bytes) == 0 && ((uintptr_t)shift % 16) == 0 && (shift_stride % 4) == 0) {
     const int groups = size / 4;
     const int per = groups <= 1024 ? 1 : groups <= 2048 ? 2 : 4;
     const int vthreads = (((groups + per - 1) / per) + 31) / 32 * 32;
@@ -187,13 +189,13 @@ FE_EXPORT int fe_add_rmsnorm(float* residual, const void* update, int update_dty
     do {                                                                                                          \
       if (per == 1)                                                                                               \
         rc = fe_launch_dependent(add_rmsnorm_vec_kernel<TU, TO, 1>, dim3(rows), dim3(vthreads), 0, stream, residual, \
-            (const TU*)update, weight, (TO*)out, row_map, shift, size, eps, write_residual);                             \
+            (const TU*)update, weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                             \
       else if (per == 2)                                                                                          \
         rc = fe_launch_dependent(add_rmsnorm_vec_kernel<TU, TO, 2>, dim3(rows), dim3(vthreads), 0, stream, residual, \
-            (const TU*)update, weight, (TO*)out, row_map, shift, size, eps, write_residual);                             \
+            (const TU*)update, weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                             \
       else                                                                                                        \
         rc = fe_launch_dependent(add_rmsnorm_vec_kernel<TU, TO, 4>, dim3(rows), dim3(vthreads), 0, stream, residual, \
-            (const TU*)update, weight, (TO*)out, row_map, shift, size, eps, write_residual);                             \
+            (const TU*)update, weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                             \
     } while (0)
     if (update_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_F32) LAUNCH_VEC(float, float);
     else if (update_dtype == FE_DTYPE_BF16 && out_dtype == FE_DTYPE_BF16) LAUNCH_VEC(bf16, bf16);
@@ -210,13 +212,13 @@ FE_EXPORT int fe_add_rmsnorm(float* residual, const void* update, int update_dty
   do {                                                                                               \
     if (per <= 4)                                                                                    \
       rc = fe_launch_dependent(add_rmsnorm_kernel<TU, TO, 4>, dim3(rows), dim3(threads), 0, stream, residual, (const TU*)update,      \
-          weight, (TO*)out, row_map, shift, size, eps, write_residual);                                     \
+          weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                                     \
     else if (per <= 16)                                                                              \
       rc = fe_launch_dependent(add_rmsnorm_kernel<TU, TO, 16>, dim3(rows), dim3(threads), 0, stream, residual, (const TU*)update,     \
-          weight, (TO*)out, row_map, shift, size, eps, write_residual);                                     \
+          weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                                     \
     else                                                                                             \
       rc = fe_launch_dependent(add_rmsnorm_kernel<TU, TO, 0>, dim3(rows), dim3(threads), 0, stream, residual, (const TU*)update,      \
-          weight, (TO*)out, row_map, shift, size, eps, write_residual);                                     \
+          weight, (TO*)out, row_map, shift, shift_stride, size, eps, write_residual);                                     \
   } while (0)
   if (update_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_F32) LAUNCH(float, float);
   else if (update_dtype == FE_DTYPE_BF16 && out_dtype == FE_DTYPE_BF16) LAUNCH(bf16, bf16);
@@ -394,5 +396,35 @@ FE_EXPORT int fe_scale_cap(float* x, long long total, float scale, float cap, cu
   long long blocks = (total + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   const int rc = fe_launch_dependent(scale_cap_kernel, dim3((unsigned)blocks), dim3(256), 0, stream, x, total, scale, cap);
+  return rc ? rc : fe_last_error();
+}
+
+// ---------------------------------------------------------------------------
+// norm_pair: out = scale * (a / rms(a) * w_a + b / rms(b) * w_b) per row, rms over the row with
+// eps inside the root; everything 32-bit (two mixers side by side, each normalised)
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(256)
+norm_pair_kernel(const float* __restrict__ a, const float* __restrict__ b, const float* __restrict__ w_a,
+                 const float* __restrict__ w_b, float* __restrict__ out, int size, float eps, float scale) {
+  __shared__ float scratch[33];
+  pdl_trigger();
+  pdl_wait();
+  const size_t at = (size_t)blockIdx.x * size;
+  float sa = 0.f, sb = 0.f;
+  for (int i = threadIdx.x; i < size; i += blockDim.x) {
+    const float x = a[at + i], y = b[at + i];
+    sa = fmaf(x, x, sa);
+    sb = fmaf(y, y, sb);
+  }
+  const float ia = scale / sqrtf(block_sum(sa, scratch) / (float)size + eps);
+  const float ib = scale / sqrtf(block_sum(sb, scratch) / (float)size + eps);
+  for (int i = threadIdx.x; i < size; i += blockDim.x) out[at + i] = a[at + i] * ia * w_a[i] + b[at + i] * ib * w_b[i];
+}
+
+FE_EXPORT int fe_norm_pair(const float* a, const float* b, const float* w_a, const float* w_b, float* out, int rows, int size,
+                           float eps, float scale, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (size < 1) return FE_ERR_BAD_SHAPE;
+  const int rc = fe_launch_dependent(norm_pair_kernel, dim3(rows), dim3(256), 0, stream, a, b, w_a, w_b, out, size, eps, scale);
   return rc ? rc : fe_last_error();
 }

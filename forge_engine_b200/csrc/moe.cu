@@ -25,7 +25,8 @@
 //                64 (any dtype), or mma.sync tiles for bfloat16; each output element is summed
 //                over k in a fixed order, so a row's result does not depend on its neighbours.
 //   moe_combine  a token's update = the sum of its slots' rows (times the weight where it
-//                scales the output) + gate * the shared unit's output, in slot order.
+//                scales the output) + gate * the shared unit's output, in slot order (+ a 32-bit row
+//                of another sublayer that joins the stream in the same sum).
 #include "common.cuh"
 
 #define MOE_BM 64
@@ -56,14 +57,15 @@ __device__ __forceinline__ float moe_act(float z, float u, const MoeAct& a) {
 }
 
 // ---------------------------------------------------------------------------
-// router logits: out[n, r] = sum_k x[n, k] * w[r, k] for a handful of rows r, in plain 32-bit
+// router logits: out[n, r] = sum_k x[n, k] * w[r, k] (+ bias[r]) for a handful of rows r, in plain 32-bit
 // FMAs.  A block takes one token (its activations in shared memory as floats) and eight rows,
 // a warp one row: lanes stride over k, the 32 partial sums meet in a butterfly.  The order of
 // additions depends on k alone, so a token's logits do not depend on the batch.
 // ---------------------------------------------------------------------------
 template <typename TX>
 __global__ void __launch_bounds__(256)
-moe_logits_kernel(const TX* __restrict__ x, const float* __restrict__ w, float* __restrict__ out, int rows, int k) {
+moe_logits_kernel(const TX* __restrict__ x, const float* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out,
+                  int rows, int k) {
   extern __shared__ float xs[];
   pdl_trigger();
   pdl_wait();
@@ -88,11 +90,11 @@ moe_logits_kernel(const TX* __restrict__ x, const float* __restrict__ w, float* 
     for (int i = lane; i < k; i += 32) sum = fmaf(xs[i], wr[i], sum);
   }
   sum = warp_sum(sum);
-  if (lane == 0) out[(size_t)token * rows + row] = sum;
+  if (lane == 0) out[(size_t)token * rows + row] = bias != nullptr ? sum + bias[row] : sum;
 }
 
-// x [n, k] (bfloat16 or 32-bit), w [rows, k] 32-bit, out [n, rows] 32-bit
-FE_EXPORT int fe_moe_logits(const void* x, int x_dtype, const float* w, float* out, int n, int rows, int k, cudaStream_t stream) {
+// x [n, k] (bfloat16 or 32-bit), w [rows, k] and bias [rows] (or null) 32-bit, out [n, rows] 32-bit
+FE_EXPORT int fe_moe_logits(const void* x, int x_dtype, const float* w, const float* bias, float* out, int n, int rows, int k, cudaStream_t stream) {
   if (n <= 0 || rows <= 0) return 0;
   if (k <= 0 || (size_t)k * sizeof(float) > 200 * 1024 || ((uintptr_t)w & 15)) return FE_ERR_BAD_SHAPE;
   const size_t smem = (size_t)k * sizeof(float);
@@ -100,10 +102,10 @@ FE_EXPORT int fe_moe_logits(const void* x, int x_dtype, const float* w, float* o
   int rc;
   if (x_dtype == FE_DTYPE_BF16) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_logits_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    rc = fe_launch_dependent(moe_logits_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)x, w, out, rows, k);
+    rc = fe_launch_dependent(moe_logits_kernel<bf16>, grid, dim3(256), smem, stream, (const bf16*)x, w, bias, out, rows, k);
   } else if (x_dtype == FE_DTYPE_F32) {
     if (smem > 48 * 1024) cudaFuncSetAttribute(moe_logits_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    rc = fe_launch_dependent(moe_logits_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, w, out, rows, k);
+    rc = fe_launch_dependent(moe_logits_kernel<float>, grid, dim3(256), smem, stream, (const float*)x, w, bias, out, rows, k);
   } else return FE_ERR_BAD_DTYPE;
   return rc ? rc : fe_last_error();
 }
@@ -542,7 +544,7 @@ __global__ void __launch_bounds__(256)
 moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ slot_row, const float* __restrict__ slot_weight,
                    int top, int width, const TS* __restrict__ shared, const float* __restrict__ shared_logit,
                    long long shared_ld, const int* __restrict__ slot_expert, int experts, const void* __restrict__ input,
-                   int input_bf16, TO* __restrict__ out) {
+                   int input_bf16, const float* __restrict__ add, TO* __restrict__ out) {
   pdl_trigger();
   pdl_wait();
   const int token = blockIdx.x;
@@ -572,6 +574,12 @@ moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ slot_
 #pragma unroll
         for (int e = 0; e < 4; ++e) sum[e] = fmaf(gate, v[e], sum[e]);
       }
+      if (add != nullptr) {
+        float v[4];
+        load4(add + (size_t)token * width + c, v);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) sum[e] += v[e];
+      }
       store4(out + (size_t)token * width + c, sum);
     }
     return;
@@ -588,6 +596,7 @@ moe_combine_kernel(const float* __restrict__ rows, const int* __restrict__ slot_
       sum += slot_weight ? v * slot_weight[slot] : v;
     }
     if (shared != nullptr) sum = fmaf(gate, to_float(shared[(size_t)token * width + c]), sum);
+    if (add != nullptr) sum += add[(size_t)token * width + c];
     out[(size_t)token * width + c] = from_float<TO>(sum);
   }
 }
@@ -672,7 +681,7 @@ FE_EXPORT int fe_moe_grouped(const void* a, int a_dtype, long long lda, const vo
 FE_EXPORT int fe_moe_combine(const float* rows, const int* slot_row, const float* slot_weight, int top, int width,
                              const void* shared, int shared_dtype, const float* shared_logit, long long shared_ld,
                              void* out, int out_dtype, int n_tokens, const int* slot_expert, int experts,
-                             const void* input, int input_dtype, cudaStream_t stream) {
+                             const void* input, int input_dtype, const float* add, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (input != nullptr && (slot_expert == nullptr || (input_dtype != FE_DTYPE_F32 && input_dtype != FE_DTYPE_BF16)))
     return FE_ERR_BAD_DTYPE;
@@ -683,7 +692,7 @@ FE_EXPORT int fe_moe_combine(const float* rows, const int* slot_row, const float
   int rc = FE_ERR_BAD_DTYPE;
 #define MOE_COMBINE(TS, TO)                                                                                           \
   rc = fe_launch_dependent(moe_combine_kernel<TS, TO>, grid, dim3(256), 0, stream, rows, slot_row, slot_weight, top, \
-                           width, (const TS*)shared, shared_logit, shared_ld, slot_expert, experts, input, input_bf16, (TO*)out)
+                           width, (const TS*)shared, shared_logit, shared_ld, slot_expert, experts, input, input_bf16, add, (TO*)out)
   if (shared == nullptr) shared_dtype = FE_DTYPE_F32;
   if (shared_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_F32) MOE_COMBINE(float, float);
   else if (shared_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_BF16) MOE_COMBINE(float, bf16);

@@ -296,23 +296,25 @@ __global__ void qk_rope_cache_sums_kernel(float* __restrict__ sums, bf16* __rest
 }
 
 // cos and sin of float(position) * inv_freq[j] for every token and pair j, taken once per
-// step: table [n, half] of (cos, sin).  The angles are the same in every layer.
+// step: table [n, half] of (cos, sin), both times `amplitude` (1 for a plain rotation).  The angles
+// are the same in every layer.
 __global__ void rope_table_kernel(const int* __restrict__ positions, const float* __restrict__ inv_freq, int half, int n,
-                                  float2* __restrict__ table) {
+                                  float amplitude, float2* __restrict__ table) {
   pdl_trigger();
   pdl_wait();
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
   if (i >= n * half) return;
   const int token = i / half, j = i - token * half;
   const float angle = (float)positions[token] * inv_freq[j];
-  table[i] = make_float2(cosf(angle), sinf(angle));
+  table[i] = make_float2(cosf(angle) * amplitude, sinf(angle) * amplitude);
 }
 
-FE_EXPORT int fe_rope_table(const int* positions, const float* inv_freq, int half, int n, void* table, cudaStream_t stream) {
+FE_EXPORT int fe_rope_table(const int* positions, const float* inv_freq, int half, int n, float amplitude, void* table,
+                            cudaStream_t stream) {
   if (n <= 0 || half <= 0) return 0;
   const int threads = 128;
   return fe_launch_dependent(rope_table_kernel, dim3((n * half + threads - 1) / threads), dim3(threads), 0, stream, positions,
-                             inv_freq, half, n, (float2*)table);
+                             inv_freq, half, n, amplitude, (float2*)table);
 }
 
 // `table` (optional): the output of fe_rope_table for these tokens and inv_freq; without it

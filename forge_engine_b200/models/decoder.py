@@ -90,7 +90,10 @@ class DecoderModel:
             if shift is not None and shift not in self.shifts:
                 name, row = shift
                 self.shifts[shift] = weights[name][row].to(device=ctx.device, dtype=torch.float32).contiguous()
+        self.reuses_embedding = any(getattr(run, "add_embedding", False) for run in spec.schedule)
         for index, run in enumerate(spec.schedule):
+            if getattr(run, "add_embedding", False) and getattr(run, "shift", None) is not None:
+                raise ValueError(f"run {index} adds both the embedding output and a vector")
             if not 0 <= run.layer < len(self.blocks):
                 raise ValueError(f"run {index} names layer {run.layer}, which does not exist")
             if run.cache_of is not None and not 0 <= run.cache_of < index:
@@ -161,12 +164,15 @@ class DecoderModel:
                              scale=getattr(self.spec, "embedding_scale", 1.0), positions=batch.positions,
                              position_table=self.position_table)
         pending = None
+        start = h.clone() if self.reuses_embedding else None      # the embedding output
         for index, run in enumerate(self.spec.schedule):
             shift = getattr(run, "shift", None)
-            if shift is None:
+            extra = start if getattr(run, "add_embedding", False) else None if shift is None else self.shifts[shift]
+            if extra is None:
                 pending = self.blocks[run.layer].forward(h, pending, batch, cache.view(index))
             else:
-                pending = self.blocks[run.layer].forward(h, pending, batch, cache.view(index), shift=self.shifts[shift])
+                # a vector for all rows, or a row each, that the block's first norm adds to the stream
+                pending = self.blocks[run.layer].forward(h, pending, batch, cache.view(index), shift=extra)
         if batch.n_want == 0:
             return torch.empty((0, self.spec.vocab_size), dtype=torch.float32, device=self.ctx.device)
         # an arrangement whose pending update is more than a tensor folds it into the final norm itself

@@ -63,7 +63,7 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_qkv_prepare": [p, i, i, i, i, i, i, p, i, p, i, i, i, i, i, p, i, p, i, i, i, f, p, i, i, p, ll, ll, i,
                            p, p, i, p, i, i, i, p, p, i, p, p],
         "fe_attention_general": [p, ll, ll, p, i, i, p, i, i, p, ll, ll, i, p, i, i, i, i, i, p, p, p, p, i, i, f,
-                                 i, f, f, i, i, ll, i, ll, p, ll, i, p, i, p, p],
+                                 i, f, f, i, i, ll, i, ll, p, ll, i, i, p, i, p, p],
         "fe_differential_combine": [p, p, i, ll, i, f, f, f, p],
         "fe_bias_xielu": [p, i, p, p, i, ll, i, f, f, p],
         "fe_bias_act": [p, i, p, p, i, ll, i, i, p],
@@ -75,31 +75,43 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_causal_conv_state": [p, p, p, ll, p, p, p, p, i, i, i, i, i, p],
         "fe_moe_route": [p, ll, i, i, i, i, i, p, p, p, p, p, p, p, p, p, i, i, i, p, i, i, f, f, i, p],
         "fe_moe_grouped": [p, i, ll, p, p, i, p, i, i, i, i, i, p, p, p, p, p, i, f, f, i, p],
-        "fe_moe_combine": [p, p, p, i, i, p, i, p, ll, p, i, i, p, i, p, i, p],
+        "fe_moe_combine": [p, p, p, i, i, p, i, p, ll, p, i, i, p, i, p, i, p, p],
         "fe_moe_max_tiles": [i, i, i],
         "fe_linear_recurrence": [p, i, i, i, i, i, i, p, p, p, p, p, i, i, i, i, i, p],
         "fe_linear_recurrence_chunked": [p, i, i, i, i, i, i, p, p, p, p, p, p, i, i, i, i, i, i, p],
         "fe_linear_recurrence_chunks": [i, i],
         "fe_gemm_simt_batched": [p, i, p, i, p, i, i, i, i, i, ll, ll, ll, ll, ll, p],
-        "fe_add_rmsnorm": [p, p, i, p, p, i, p, p, i, i, f, i, p],
+        "fe_add_rmsnorm": [p, p, i, p, p, i, p, p, ll, i, i, f, i, p],
+        "fe_norm_pair": [p, p, p, p, p, i, i, f, f, p],
         "fe_silu_mul": [p, p, i, i, i, i, p],
         "fe_qk_rope_cache": [p, i, p, p, f, p, p, i, p, p, p, p, p, i, i, i, i, i, i, i, i, p, p],
         "fe_qk_rope_cache_sums": [p, p, p, p, f, p, p, p, p, p, p, p, i, i, i, i, i, i, i, i, p, p],
-        "fe_rope_table": [p, p, i, i, p, p],
+        "fe_rope_table": [p, p, i, i, f, p, p],
         "fe_attention_simt": [p, i, i, p, p, p, i, i, i, p, p, i, f, p, i, i, i, i, p, p],
         "fe_gemm_simt": [p, i, p, i, p, p, i, i, i, i, i, p],
         "fe_sample": [p, i, i, p, p, p, p, p, p, p, p, p],
         "fe_gemm_tc5": [p, p, p, p, i, i, i, i, i, p, p, p, f, f, p],
         "fe_gemm_tc5_grouped": [p, p, p, i, i, i, i, i, i, i, p, p, p, f, f, p, p],
         "fe_moe_gather": [p, i, i, i, i, p, p, p, p],
-        "fe_moe_logits": [p, i, p, p, i, i, i, p],
+        "fe_moe_logits": [p, i, p, p, p, i, i, i, p],
+        "fe_token_shift": [p, p, p, i, p, ll, p, f, p, i, p, p, p, p, p, p, i, i, i, p],
+        "fe_wkv_decay": [p, p, p, p, i, i, i, p],
+        "fe_wkv": [p, p, p, p, ll, p, p, p, ll, f, p, i, p, p, p, i, i, i, i, i, i, p, p, p],
+        "fe_wkv_scratch": [i, i, i, i, i],
+        "fe_state_long_from": [],
+        "fe_delta_prepare": [p, ll, i, i, p, i, p, p, p, p, p, p, i, i, i, i, p, p, i, i, p],
+        "fe_delta_rule": [p, ll, p, p, ll, p, f, p, i, p, p, p, i, i, i, i, i, i, i, i, p, p, p],
+        "fe_delta_rule_scratch": [i, i, i, i, i, i],
+        "fe_matrix_memory": [p, ll, i, i, i, i, i, i, p, p, f, f, p, f, p, p, p, i, p, p, p, i, i, i, i, i, i, i, p, p, p],
+        "fe_matrix_memory_scratch": [i, i, i, i, i, i],
         "fe_gemm_tc5_qkv_rope": [p, p, p, p, i, i, i, p, p, f, p, p, p, p, p, p, i, i, i, i, i, i, p, p],
     }
     for name, argtypes in signatures.items():
         fn = getattr(handle, name)
         fn.argtypes = argtypes
         fn.restype = c_int
-    handle.fe_gated_recurrence_scratch.restype = ctypes.c_longlong
+    for name in ("fe_gated_recurrence_scratch", "fe_wkv_scratch", "fe_delta_rule_scratch", "fe_matrix_memory_scratch"):
+        getattr(handle, name).restype = ctypes.c_longlong
     handle.fe_uniform_host.argtypes = [c_ulonglong, c_ulonglong]
     handle.fe_uniform_host.restype = c_float
 
@@ -143,25 +155,30 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
                           block_table: torch.Tensor, cu_tokens: torch.Tensor, starts: torch.Tensor, n_entries: int,
                           max_new: int, num_q_heads: int, window: int | None, keep_first: int, scale: float,
                           gate: torch.Tensor | None, row_lo: int, status: torch.Tensor,
-                          distance_bias: torch.Tensor | None = None, softcap: float | None = None) -> None:
+                          distance_bias: torch.Tensor | None = None, softcap: float | None = None,
+                          sinks: torch.Tensor | None = None, gate_per_element: bool = False) -> None:
     """The tcgen05 prefill attention for the entries of a step with more than ``row_lo`` rows
     (new tokens x heads per kv head): ``q`` [N, heads * D] and ``out`` [N, heads * D] bfloat16,
     caches [pages, kv_heads, page_size, D].  ``window`` with ``keep_first``: keys below it
     stay visible; ``gate`` (32-bit [N, >= heads]): sigmoid gates per (token, head);
     ``distance_bias`` (32-bit [heads, L]): entry min(query position - key position, L - 1) of the
     head's row is added to the score before the scale, so it holds the bias over the scale;
-    ``softcap`` c (not together with the bias): scaled scores become c tanh(score / c)."""
+    ``softcap`` c (not together with the bias): scaled scores become c tanh(score / c);
+    ``sinks`` (32-bit, per query head): exp(sink) joins the denominator once; ``gate_per_element``:
+    ``gate`` is [N, heads * D], one sigmoid gate per element of the output."""
     _dense(q, "q"), _dense(out, "out"), _dense(k_cache, "k_cache"), _dense(v_cache, "v_cache"), _dense(block_table, "block_table")
     num_pages, nkv, page_size, d = k_cache.shape
     n = q.shape[0]
     assert q.dtype == out.dtype == k_cache.dtype == v_cache.dtype == torch.bfloat16 and v_cache.shape == k_cache.shape
     assert q.shape == out.shape == (n, num_q_heads * d) and num_q_heads % nkv == 0
-    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == n)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == n
+                            and gate.shape[1] >= num_q_heads * (d if gate_per_element else 1))
+    assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_cuda and sinks.is_contiguous() and sinks.numel() == num_q_heads)
     handle = _attention_handle(d)
     fn = getattr(handle, f"fe_attention_prefill_tc5_d{d}")
     if not getattr(fn, "_declared", False):
         p, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
-        fn.argtypes = [p, i, p, p, p, p, i, i, i, i, i, p, p, i, i, i, i, i, f, p, ll, i, p, i, f, p, p]
+        fn.argtypes = [p, i, p, p, p, p, i, i, i, i, i, p, p, i, i, i, i, i, f, p, ll, i, i, p, i, f, p, p, p]
         fn.restype = c_int
         fn._declared = True
     assert not (softcap and distance_bias is not None)
@@ -170,9 +187,9 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     gate_stride = 0 if gate is None else (int(gate.stride(0)) if n > 1 else int(gate.shape[1]))
     check(fn(ptr(q), int(q.shape[1]), ptr(out), ptr(k_cache), ptr(v_cache), ptr(block_table), block_table.shape[1],
              page_size, num_pages, nkv, num_q_heads // nkv, ptr(cu_tokens), ptr(starts), int(n_entries), int(max_new), n,
-             int(window or 0), int(keep_first or 0), float(scale), ptr(gate), gate_stride, int(row_lo),
+             int(window or 0), int(keep_first or 0), float(scale), ptr(gate), gate_stride, d if gate_per_element else 0, int(row_lo),
              ptr(distance_bias), 0 if distance_bias is None else int(distance_bias.shape[1]), float(softcap or 0.0),
-             ptr(status), stream()), "attention_prefill_tc5")
+             ptr(sinks), ptr(status), stream()), "attention_prefill_tc5")
 
 
 def _attention_handle(head_dim: int):
@@ -413,13 +430,14 @@ def moe_max_tiles(slots: int, experts: int, tile_rows: int = 0) -> int:
     return int(lib().fe_moe_max_tiles(int(slots), int(experts), int(tile_rows)))
 
 
-def moe_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
-    """out[n, r] = x[n] . w[r] for a handful of 32-bit rows ``w`` (a router), in plain 32-bit
+def moe_logits(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, bias: torch.Tensor | None = None) -> None:
+    """out[n, r] = x[n] . w[r] (+ bias[r], 32-bit) for a handful of 32-bit rows ``w`` (a router), in plain 32-bit
     FMAs whatever the dtype of ``x``."""
     _dense(x, "x"), _dense(w, "w"), _dense(out, "out")
     n, k = x.shape
     assert w.dtype == torch.float32 and out.dtype == torch.float32 and w.shape[1] == k and out.shape == (n, w.shape[0])
-    check(lib().fe_moe_logits(ptr(x), code(x), ptr(w), ptr(out), n, int(w.shape[0]), int(k), stream()), "moe_logits")
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == w.shape[0])
+    check(lib().fe_moe_logits(ptr(x), code(x), ptr(w), ptr(bias), ptr(out), n, int(w.shape[0]), int(k), stream()), "moe_logits")
 
 
 def moe_gather(x: torch.Tensor, plan: dict, top: int, slot_weight: torch.Tensor | None, out: torch.Tensor) -> None:
@@ -516,22 +534,24 @@ def moe_grouped(a: torch.Tensor, w1: torch.Tensor, w2: torch.Tensor | None, out:
 
 def moe_combine(rows: torch.Tensor, plan: dict, top: int, out: torch.Tensor, *, slot_weight: torch.Tensor | None = None,
                 shared: torch.Tensor | None = None, shared_logit: torch.Tensor | None = None,
-                identity_input: torch.Tensor | None = None, experts: int = 0) -> None:
+                identity_input: torch.Tensor | None = None, experts: int = 0, add: torch.Tensor | None = None) -> None:
     """out[token] = sum over the token's slots of rows[slot's row] (times ``slot_weight``) +
     sigmoid(shared_logit[token]) * shared[token] (the gate 1 without a logit); 32-bit sums.
     With ``identity_input`` [N, width] a slot whose expert number is ``experts`` or above
-    contributes the token's row of it instead of a row of ``rows``."""
+    contributes the token's row of it instead of a row of ``rows``.  ``add`` (32-bit [N, width])
+    is added to the result (another sublayer's update that joins the stream in the same sum)."""
     _dense(rows, "rows"), _dense(out, "out")
     n, width = out.shape
     assert rows.dtype == torch.float32 and rows.shape == (n * top, width)
     assert shared is None or (shared.shape == out.shape and shared.is_contiguous())
     assert shared_logit is None or (shared_logit.dtype == torch.float32 and shared_logit.shape[0] == n)
     assert identity_input is None or (identity_input.shape == out.shape and identity_input.is_contiguous())
+    assert add is None or (add.shape == out.shape and add.is_contiguous() and add.dtype == torch.float32)
     check(lib().fe_moe_combine(ptr(rows), ptr(plan["slot_row"]), ptr(slot_weight), int(top), int(width), ptr(shared),
                                code(shared) if shared is not None else F32, ptr(shared_logit),
                                int(shared_logit.stride(0)) if shared_logit is not None and n > 1 else 1,
                                ptr(out), code(out), n, ptr(plan["slot_expert"]), int(experts), ptr(identity_input),
-                               code(identity_input) if identity_input is not None else F32, stream()), "moe_combine")
+                               code(identity_input) if identity_input is not None else F32, ptr(add), stream()), "moe_combine")
 
 
 CONV_MAX_TAPS = 8      # what causal_conv_state takes
@@ -783,7 +803,7 @@ def general_attention_lib(key_dim: int, value_dim: int, value_in_key: bool):
         run = getattr(handle, f"fe_attention_gmma_{suffix}")
         p, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
         run.argtypes = [p, ll, ll, p, i, p, i, p, ll, ll, p, i, i, i, i, i, p, p, i, i, p, p, i, i, f, i, p,
-                        i, f, f, i, i, ll, i, ll, p, ll, i, i, p, p, p]
+                        i, f, f, i, i, ll, i, ll, p, ll, i, i, i, p, p, p]
         run.restype = c_int
         space = getattr(handle, f"fe_attention_gmma_workspace_{suffix}")
         space.argtypes = [i, i, i, i, i]
@@ -844,6 +864,7 @@ def attention_general(
     row_hi: int = 0,
     distance_bias: torch.Tensor | None = None,
     sinks: torch.Tensor | None = None,
+    gate_per_element: bool = False,
 ) -> None:
     """Paged causal attention for any key and value size: scores, softmax and sums in 32-bit.
 
@@ -868,7 +889,8 @@ def attention_general(
     elements after the head's first, its key ``part_strides[1]`` * m elements into the cached
     row, and writes ``part_strides[2]`` * m elements after the head's first output.  ``gate``
     (32-bit [N, >= heads], a column slice is fine): row (token, head) is multiplied by
-    sigmoid(gate[token, head]).  ``out`` may be 32-bit whatever the cache holds.  ``row_hi`` > 0
+    sigmoid(gate[token, head]); ``gate_per_element``: it is [N, heads * v_dim] and every element
+    of the output has a gate of its own (plain heads only: ``parts`` 1).  ``out`` may be 32-bit whatever the cache holds.  ``row_hi`` > 0
     (tensor-core kernel only): entries with more rows (new tokens x heads per kv head) are
     skipped - another kernel serves them."""
     num_pages, nkv, page_size, k_row = k_cache.shape
@@ -876,7 +898,9 @@ def attention_general(
     n = positions.numel()
     assert q.dtype == k_cache.dtype == v_cache.dtype and out.dtype in (q.dtype, torch.float32)
     assert slopes is None or (slopes.dtype == torch.float32 and slopes.numel() == num_q_heads and slopes.is_cuda)
-    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == n and gate.shape[1] >= num_q_heads)
+    assert gate is None or (gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == n
+                            and gate.shape[1] >= num_q_heads * (v_dim if gate_per_element else 1))
+    assert not gate_per_element or parts == 1
     assert distance_bias is None or (distance_bias.dtype == torch.float32 and distance_bias.is_cuda and distance_bias.is_contiguous()
                                      and distance_bias.dim() == 2 and distance_bias.shape[0] == num_q_heads)
     assert sinks is None or (sinks.dtype == torch.float32 and sinks.is_cuda and sinks.is_contiguous() and sinks.numel() == num_q_heads)
@@ -885,7 +909,7 @@ def attention_general(
     coef, every = query_temperature or (0.0, 0)
     gate_stride = 0 if gate is None else (int(gate.stride(0)) if n > 1 else int(gate.shape[1]))
     extras = (int(keep_first or 0), float(softcap or 0.0), float(coef), int(every), int(parts), int(part_strides[0]),
-              int(part_strides[1]), int(part_strides[2]), ptr(gate), gate_stride, out_f32)
+              int(part_strides[1]), int(part_strides[2]), ptr(gate), gate_stride, v_dim if gate_per_element else 0, out_f32)
     value_in_key = v_cache.data_ptr() == k_cache.data_ptr()
     if (entries is not None and general_mma_takes(q.dtype, k_dim, v_dim)
             and (k_dim == k_row if parts == 1 else (not value_in_key and part_strides[1] * (parts - 1) + k_dim <= k_row))
@@ -996,7 +1020,8 @@ def add_rmsnorm(
     write_residual: bool = True,
     shift: torch.Tensor | None = None,
 ) -> None:
-    """residual += update (+ ``shift``, one 32-bit vector added to every row) (32-bit, in
+    """residual += update (+ ``shift``: one 32-bit vector added to every row, or [N, size] a row
+    each) (32-bit, in
     place unless ``write_residual`` is false); out = rmsnorm(residual) * weight.  With
     ``row_map`` row r of ``out`` comes from row ``row_map[r]`` of ``residual`` and ``update``."""
     _dense(residual, "residual"), _dense(weight, "weight"), _dense(out, "out")
@@ -1010,15 +1035,181 @@ def add_rmsnorm(
         assert row_map.dtype == torch.int32 and row_map.numel() == rows
     else:
         assert residual.shape[0] == rows
-    assert shift is None or (shift.dtype == torch.float32 and shift.numel() == size and shift.is_contiguous())
+    assert shift is None or (shift.dtype == torch.float32 and shift.is_contiguous() and shift.shape in ((size,), tuple(residual.shape)))
     check(
         lib().fe_add_rmsnorm(
             ptr(residual), ptr(update), code(update) if update is not None else code(out),
-            ptr(weight), ptr(out), code(out), ptr(row_map), ptr(shift), rows, size, float(eps),
+            ptr(weight), ptr(out), code(out), ptr(row_map), ptr(shift), size if shift is not None and shift.dim() == 2 else 0,
+            rows, size, float(eps),
             1 if write_residual else 0, stream(),
         ),
         "add_rmsnorm",
     )
+
+
+def norm_pair(a: torch.Tensor, b: torch.Tensor, w_a: torch.Tensor, w_b: torch.Tensor, out: torch.Tensor, eps: float,
+              scale: float) -> None:
+    """out = scale * (a / rms(a) * w_a + b / rms(b) * w_b) per row of 32-bit [N, C], eps inside the roots."""
+    _dense(a, "a"), _dense(b, "b"), _dense(out, "out")
+    rows, size = out.shape
+    assert a.shape == b.shape == out.shape and a.dtype == b.dtype == out.dtype == torch.float32
+    assert w_a.dtype == w_b.dtype == torch.float32 and w_a.numel() == w_b.numel() == size
+    check(lib().fe_norm_pair(ptr(a), ptr(b), ptr(w_a), ptr(w_b), ptr(out), rows, size, float(eps), float(scale), stream()),
+          "norm_pair")
+
+
+# ---------------------------------------------------------------------------
+# recurrences with a matrix state per head
+# ---------------------------------------------------------------------------
+
+
+def state_long_from() -> int:
+    """Tokens from which on an entry of these recurrences runs chunk by chunk."""
+    return int(lib().fe_state_long_from())
+
+
+def _state_checks(state: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor, norm: torch.Tensor, out: torch.Tensor) -> tuple:
+    _dense(state, "state"), _dense(out, "out")
+    assert state.dtype == torch.float32 and norm.dtype == torch.float32 and norm.is_contiguous()
+    assert slots.dtype == torch.int32 and cu_tokens.dtype == torch.int32
+    rows, heads, dk, dv = state.shape
+    assert out.shape[1] == heads * dv
+    return rows, heads, dk, dv
+
+
+def _state_scratch(device, floats: int) -> torch.Tensor | None:
+    return None if floats <= 0 else _scratch.get("state recurrence chunks", device, floats, torch.float32, 1 << 20)
+
+
+def _columns(t: torch.Tensor, width: int) -> int:
+    """Row stride of 32-bit ``t`` [N, >= width], which may be a column slice of a contiguous tensor."""
+    assert t.dtype == torch.float32 and t.is_cuda and t.dim() == 2 and t.stride(1) == 1 and t.shape[1] >= width
+    return int(t.stride(0)) if t.shape[0] > 1 else int(t.shape[1])
+
+
+def token_shift(mu: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor, token_entry: torch.Tensor,
+                mixed: torch.Tensor, plain: torch.Tensor | None, *, y: torch.Tensor | None = None,
+                residual: torch.Tensor | None = None, update: torch.Tensor | None = None, shift: torch.Tensor | None = None,
+                weight: torch.Tensor | None = None, eps: float = 0.0) -> None:
+    """mixed[j, t] = h_t + (h_(t-1) - h_t) mu[j] for every row j of 32-bit ``mu`` [mixes, C], and
+    plain[t] = h_t, both rounded on store.  h: the rows ``y`` (32-bit [N, C]); or, for steps in
+    which every entry brings one token, the norm of ``residual`` after ``update`` and ``shift`` have
+    been added to it in place (as ``add_rmsnorm``).  ``state`` (32-bit [rows, C]) holds the row
+    before an entry's first token and gets its last."""
+    mixes, width = mu.shape
+    n = mixed.shape[1]
+    _dense(mu, "mu"), _dense(state, "state"), _dense(mixed, "mixed")
+    assert mu.dtype == state.dtype == torch.float32 and mixed.shape == (mixes, n, width) and state.shape[1] == width
+    assert plain is None or (plain.shape == (n, width) and plain.dtype == mixed.dtype and plain.is_contiguous())
+    assert (y is None) != (residual is None)
+    for t in (y, residual, update):
+        assert t is None or (t.shape == (n, width) and t.is_contiguous())
+    assert y is None or y.dtype == torch.float32
+    assert residual is None or (residual.dtype == torch.float32 and weight.dtype == torch.float32 and slots.numel() >= n)
+    assert shift is None or (shift.dtype == torch.float32 and shift.is_contiguous() and shift.shape in ((width,), (n, width)))
+    check(lib().fe_token_shift(ptr(y), ptr(residual), ptr(update), code(update) if update is not None else F32, ptr(shift),
+                               width if shift is not None and shift.dim() == 2 else 0, ptr(weight), float(eps), ptr(mu), int(mixes),
+                               ptr(state), ptr(slots), ptr(cu_tokens), ptr(token_entry), ptr(mixed), ptr(plain), code(mixed), int(n),
+                               int(width), stream()), "token_shift")
+
+
+def wkv_decay(low: torch.Tensor, up: torch.Tensor, base: torch.Tensor, out: torch.Tensor) -> None:
+    """out[t, c] = exp(-exp(base[c] + sum_j tanh(low[t, j]) up[j, c])), all 32-bit."""
+    for name, t in (("low", low), ("up", up), ("base", base), ("out", out)):
+        _dense(t, name)
+        assert t.dtype == torch.float32, name
+    n, rank = low.shape
+    assert up.shape[0] == rank and out.shape == (n, up.shape[1]) and base.numel() == up.shape[1]
+    check(lib().fe_wkv_decay(ptr(low), ptr(up), ptr(base), ptr(out), int(n), int(rank), int(up.shape[1]), stream()), "wkv_decay")
+
+
+def wkv(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, decay: torch.Tensor, bonus: torch.Tensor, norm: torch.Tensor,
+        gate: torch.Tensor, eps: float, state: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor, out: torch.Tensor,
+        n_entries: int, max_new: int, status: torch.Tensor) -> None:
+    """o_t = (S + diag(bonus) k v^T)^T r, S <- diag(decay) S + k v^T over the tokens of every entry,
+    from and to the 32-bit state [rows, heads, d, d]; ``out`` [N, heads * d] gets o divided by its root
+    mean square per head, times ``norm`` [heads * d] and silu(gate).  r, k, v, decay 32-bit
+    [N, heads * d] with one row stride, ``bonus`` 32-bit [heads, d]."""
+    rows, heads, dk, dv = _state_checks(state, slots, cu_tokens, norm, out)
+    assert dk == dv and norm.numel() == heads * dv and bonus.dtype == torch.float32 and bonus.numel() == heads * dk
+    n, size = int(out.shape[0]), heads * dk
+    ld = _columns(r, size)
+    assert all(_columns(t, size) == ld and t.shape[0] == n for t in (k, v, decay))
+    scratch = _state_scratch(out.device, int(lib().fe_wkv_scratch(n, int(n_entries), heads, dk, int(max_new))))
+    check(lib().fe_wkv(ptr(r), ptr(k), ptr(v), ptr(decay), ld, ptr(bonus), ptr(norm), ptr(gate), _columns(gate, size), float(eps),
+                       ptr(state), rows, ptr(slots), ptr(cu_tokens), ptr(out), code(out), int(n_entries), heads, dk, n, int(max_new),
+                       ptr(scratch), ptr(status), stream()), "wkv")
+    _count_chunked(max_new)
+
+
+def _count_chunked(max_new: int) -> None:
+    global LAUNCHES
+    if max_new >= state_long_from():
+        LAUNCHES += 3
+
+
+def delta_prepare(proj: torch.Tensor, b_off: int, a_off: int, conv: torch.Tensor, state: torch.Tensor | None, slots: torch.Tensor,
+                  cu_tokens: torch.Tensor, token_entry: torch.Tensor, a_log: torch.Tensor, dt_bias: torch.Tensor, kv_heads: int,
+                  dk: int, heads: int, dv: int, out: torch.Tensor, gates: torch.Tensor, n_entries: int) -> None:
+    """From 32-bit ``proj`` [N, C] (q, k, v from column 0, the gates' logits at ``b_off`` and
+    ``a_off``): ``out`` [N, channels] = silu of the causal convolution of q, k, v over time (``conv``
+    [taps, channels], the last tap weighing the token itself), q and k made unit vectors per head (q
+    times dk^(-1/2)); ``gates`` [N, heads, 2] = sigmoid(b) and -exp(a_log) softplus(a + dt_bias).
+    ``state`` 32-bit [rows, taps - 1, channels]: the convolution's last inputs."""
+    taps, channels = conv.shape
+    n = int(out.shape[0])
+    for name, t in (("conv", conv), ("a_log", a_log), ("dt_bias", dt_bias), ("out", out), ("gates", gates)):
+        _dense(t, name)
+        assert t.dtype == torch.float32, name
+    assert channels == 2 * kv_heads * dk + heads * dv and out.shape == (n, channels) and gates.shape == (n, heads, 2)
+    assert a_log.numel() == dt_bias.numel() == heads
+    assert taps == 1 or (state.dtype == torch.float32 and state.is_contiguous() and state.shape[1:] == (taps - 1, channels))
+    check(lib().fe_delta_prepare(ptr(proj), _columns(proj, max(a_off, b_off) + heads), int(b_off), int(a_off), ptr(conv), int(taps),
+                                 ptr(state), ptr(slots), ptr(cu_tokens), ptr(token_entry), ptr(a_log), ptr(dt_bias), int(kv_heads),
+                                 int(dk), int(heads), int(dv), ptr(out), ptr(gates), n, int(n_entries), stream()), "delta_prepare")
+
+
+def delta_rule(qkv: torch.Tensor, gates: torch.Tensor, gate: torch.Tensor, norm: torch.Tensor, eps: float, state: torch.Tensor,
+               slots: torch.Tensor, cu_tokens: torch.Tensor, out: torch.Tensor, kv_heads: int, n_entries: int, max_new: int,
+               status: torch.Tensor) -> None:
+    """S <- g S; u = beta (v - S^T k); S <- S + k u^T; o = S^T q over the tokens of every entry, from
+    and to the 32-bit state [rows, heads, dk, dv]; ``out`` [N, heads * dv] gets o divided by its root
+    mean square per head, times ``norm`` [dv] and silu(gate).  ``qkv`` and ``gates`` (beta, log g) as
+    ``delta_prepare`` leaves them."""
+    rows, heads, dk, dv = _state_checks(state, slots, cu_tokens, norm, out)
+    _dense(qkv, "qkv"), _dense(gates, "gates")
+    n = int(out.shape[0])
+    assert qkv.shape == (n, 2 * kv_heads * dk + heads * dv) and gates.shape == (n, heads, 2) and norm.numel() == dv
+    assert qkv.dtype == gates.dtype == torch.float32
+    scratch = _state_scratch(out.device, int(lib().fe_delta_rule_scratch(n, int(n_entries), heads, dk, dv, int(max_new))))
+    check(lib().fe_delta_rule(ptr(qkv), int(qkv.shape[1]), ptr(gates), ptr(gate), _columns(gate, heads * dv), ptr(norm), float(eps),
+                              ptr(state), rows, ptr(slots), ptr(cu_tokens), ptr(out), code(out), int(n_entries), int(kv_heads), heads,
+                              dk, dv, n, int(max_new), ptr(scratch), ptr(status), stream()), "delta_rule")
+    _count_chunked(max_new)
+
+
+def matrix_memory(proj: torch.Tensor, offsets: tuple, i_bias: torch.Tensor, f_bias: torch.Tensor, cap: float, q_scale: float,
+                  norm: torch.Tensor, eps: float, state: torch.Tensor, normaliser: torch.Tensor, top: torch.Tensor,
+                  slots: torch.Tensor, cu_tokens: torch.Tensor, out: torch.Tensor, n_entries: int, max_new: int,
+                  status: torch.Tensor) -> None:
+    """The exponentially gated matrix memory over the tokens of every entry.  ``proj`` 32-bit [N, C]
+    with q, k, v, the output gate and the two gates' logits from columns ``offsets`` on; state 32-bit
+    [rows, heads, dk, dv], ``normaliser`` [rows, heads, dk], ``top`` [rows, heads] (the running
+    maximum).  ``out`` [N, heads * dv] gets o divided by its root mean square per head, times ``norm``
+    [heads * dv] and sigmoid(gate)."""
+    rows, heads, dk, dv = _state_checks(state, slots, cu_tokens, norm, out)
+    q_off, k_off, v_off, g_off, i_off, f_off = (int(o) for o in offsets)
+    n = int(out.shape[0])
+    _dense(normaliser, "normaliser"), _dense(top, "top")
+    assert normaliser.shape == (rows, heads, dk) and top.shape == (rows, heads) and normaliser.dtype == top.dtype == torch.float32
+    assert i_bias.dtype == f_bias.dtype == torch.float32 and i_bias.numel() == f_bias.numel() == heads and norm.numel() == heads * dv
+    ld = _columns(proj, max(q_off + heads * dk, k_off + heads * dk, v_off + heads * dv, g_off + heads * dv, i_off + heads, f_off + heads))
+    scratch = _state_scratch(out.device, int(lib().fe_matrix_memory_scratch(n, int(n_entries), heads, dk, dv, int(max_new))))
+    check(lib().fe_matrix_memory(ptr(proj), ld, q_off, k_off, v_off, g_off, i_off, f_off, ptr(i_bias), ptr(f_bias), float(cap),
+                                 float(q_scale), ptr(norm), float(eps), ptr(state), ptr(normaliser), ptr(top), rows, ptr(slots),
+                                 ptr(cu_tokens), ptr(out), code(out), int(n_entries), heads, dk, dv, n, int(max_new), ptr(scratch),
+                                 ptr(status), stream()), "matrix_memory")
+    _count_chunked(max_new)
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:
@@ -1030,13 +1221,13 @@ def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:
     check(lib().fe_silu_mul(ptr(gate_up), ptr(out), code(out), rows, inter, int(block), stream()), "silu_mul")
 
 
-def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, table: torch.Tensor) -> None:
-    """table[t, j] = (cos, sin) of float(positions[t]) * inv_freq[j], in 32-bit."""
+def rope_table(positions: torch.Tensor, inv_freq: torch.Tensor, table: torch.Tensor, amplitude: float = 1.0) -> None:
+    """table[t, j] = (cos, sin) of float(positions[t]) * inv_freq[j], both times ``amplitude``, in 32-bit."""
     _dense(positions, "positions"), _dense(inv_freq, "inv_freq"), _dense(table, "table")
     n, half = positions.numel(), inv_freq.numel()
     assert positions.dtype == torch.int32 and inv_freq.dtype == torch.float32
     assert table.dtype == torch.float32 and table.shape == (n, half, 2)
-    check(lib().fe_rope_table(ptr(positions), ptr(inv_freq), half, n, ptr(table), stream()), "rope_table")
+    check(lib().fe_rope_table(ptr(positions), ptr(inv_freq), half, n, float(amplitude), ptr(table), stream()), "rope_table")
 
 
 def qk_rope_cache(

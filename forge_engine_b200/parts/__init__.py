@@ -1,6 +1,20 @@
 """Parts of a layer: norms, position encodings, mixers, feed-forwards, blocks."""
 
-from . import attention, block, ffn, gated_recurrence, latent_attention, linear_recurrence, moe, norms, positions  # noqa: F401  (registers the kinds)
+from . import (  # noqa: F401  (registers the kinds)
+    attention,
+    block,
+    delta_rule,
+    ffn,
+    gated_recurrence,
+    latent_attention,
+    linear_recurrence,
+    matrix_memory,
+    moe,
+    norms,
+    positions,
+    side_by_side,
+    wkv,
+)
 from .base import (
     BuildContext,
     CacheView,

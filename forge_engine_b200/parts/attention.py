@@ -133,14 +133,15 @@ class GQAttention(Mixer):
     def _is_general(spec) -> bool:
         """Whether the layer needs what only the general kernels do: values of another size
         than keys, q and k normalised over the whole projection, a bias on the distance, kept
-        first tokens, capped scores, a query temperature, a gate per head, two maps per head, q and
-        k normalised without a weight or after the rotation."""
+        first tokens, capped scores, a query temperature, a gate per head or per element, sinks, two
+        maps per head, q and k normalised without a weight or after the rotation."""
         return (getattr(spec, "v_head_dim", None) not in (None, spec.head_dim)
                 or (spec.qk_norm and getattr(spec, "qk_norm_scope", "head") == "whole")
                 or getattr(spec, "distance_bias_base", None) is not None
                 or getattr(spec, "distance_bias_table", None) is not None or not getattr(spec, "kv_projection", True)
                 or bool(getattr(spec, "keep_first", 0)) or getattr(spec, "softcap", None) is not None
                 or getattr(spec, "query_temperature", None) is not None or bool(getattr(spec, "head_gate", False))
+                or bool(getattr(spec, "sink", False)) or bool(getattr(spec, "output_gate", False))
                 or getattr(spec, "differential", None) is not None
                 or (spec.qk_norm and (not getattr(spec, "qk_norm_weight", True) or getattr(spec, "qk_norm_after_rotation", False))))
 
@@ -163,6 +164,14 @@ class GQAttention(Mixer):
         self.differential = getattr(spec, "differential", None)
         self.parts = 1 if self.differential is None else 2
         self.head_gate = bool(getattr(spec, "head_gate", False))
+        self.output_gate = bool(getattr(spec, "output_gate", False))
+        if self.output_gate and (self.head_gate or self.parts > 1 or spec.bias or not getattr(spec, "kv_projection", True)):
+            raise ConfigError("a gate per element goes with a plain layer: no gate per head, no second map, no biases, keys of its own")
+        self.sinks = None
+        if getattr(spec, "sink", False):
+            if self.parts > 1:
+                raise ConfigError("a differential layer takes no sinks")
+            self.sinks = weights[name("sink")].to(device=ctx.device, dtype=torch.float32).contiguous()
         self.keep_first = int(getattr(spec, "keep_first", 0) or 0) if spec.window else 0
         self.softcap = getattr(spec, "softcap", None)
         self.query_temperature = getattr(spec, "query_temperature", None)
@@ -180,6 +189,9 @@ class GQAttention(Mixer):
         if self.head_gate:
             # the gates' logits are further columns of the same product
             rows.append(self.nq)
+            names.append(name("gate_proj.weight"))
+        if self.output_gate:
+            rows.append(self.nq * self.dv)
             names.append(name("gate_proj.weight"))
         if spec.bias:
             if self.head_gate:
@@ -265,6 +277,10 @@ class GQAttention(Mixer):
             shapes[name("rel")] = WeightInfo((spec.distance_bias_table[0], spec.num_heads), "bias")
         if getattr(spec, "head_gate", False):
             shapes[name("gate_proj.weight")] = WeightInfo((spec.num_heads, h))
+        if getattr(spec, "output_gate", False):
+            shapes[name("gate_proj.weight")] = WeightInfo((spec.num_heads * dv, h))
+        if getattr(spec, "sink", False):
+            shapes[name("sink")] = WeightInfo((spec.num_heads,), "bias")
         if parts > 1:
             for vector in ("lambda_q1", "lambda_k1", "lambda_q2", "lambda_k2"):
                 shapes[name(vector)] = WeightInfo((spec.head_dim,), "bias")
@@ -370,14 +386,14 @@ class GQAttention(Mixer):
         if self.plan_key not in batch.plans:
             self.plan_step(batch.entries, k_cache.shape[2], batch.plans)
         splits, long_entries, short_entries = batch.plans[self.plan_key]
-        gate = qkv[:, k_end + nkv * dv :] if self.head_gate else None
+        gate = qkv[:, k_end + nkv * dv :] if self.head_gate or self.output_gate else None
         with self.ctx.section("mixer.attention"):
             if long_entries:
                 # prompt portions of a plain softmax layer with heads of 64 or 128: the tcgen05 kernel
                 native.attention_prefill_tc5(q, k_cache, v_cache, out, table, batch.cu_tokens, batch.starts, batch.n_entries,
                                              batch.max_new, nq, self.spec.window, self.keep_first, self.spec.scale, gate,
                                              SHORT_ENTRY_ROWS, self.ctx.status, distance_bias=self.distance_bias_unscaled,
-                                             softcap=self.softcap)
+                                             softcap=self.softcap, sinks=self.sinks, gate_per_element=self.output_gate)
             if short_entries:
                 native.attention_general(q, (nq * d, d), k_cache, self.d, v_cache, dv, out, (nq * parts * dv, parts * dv), table,
                                          batch.positions, batch.token_entry, nq, self.slopes, self.spec.window,
@@ -387,7 +403,8 @@ class GQAttention(Mixer):
                                          softcap=self.softcap, query_temperature=self.query_temperature, parts=parts,
                                          part_strides=(self.d, self.d, dv) if parts > 1 else (0, 0, 0),
                                          gate=gate, row_hi=SHORT_ENTRY_ROWS if long_entries else 0,
-                                         distance_bias=self.distance_bias)
+                                         distance_bias=self.distance_bias, sinks=self.sinks,
+                                         gate_per_element=self.output_gate)
             if parts > 1:
                 maps = out
                 out = torch.empty((n, nq * dv), dtype=k_cache.dtype, device=x.device)
@@ -446,8 +463,8 @@ class GQAttention(Mixer):
 
     def _prefill_tc5(self, page_size: int) -> bool:
         """Whether prompt portions of this (general) layer run on the tcgen05 prefill kernel:
-        a plain softmax over one map per head (a window, kept first tokens, a gate per head and
-        either a bias by distance or capped scores it has), keys and values of 64 or 128."""
+        a plain softmax over one map per head (a window, kept first tokens, gates, sinks and either a
+        bias by distance or capped scores it has), keys and values of 64 or 128."""
         return (self.parts == 1 and self.slopes is None and (self.softcap is None or self.distance_bias is None)
                 and self.query_temperature is None
                 and self.spec.scale > 0 and native.prefill_tc5_takes(self.ctx.dtype, self.d, self.dv, self.nq // self.nkv, page_size)

@@ -16,7 +16,7 @@ the package needs to change; an architecture then names the kind in its LayerSpe
 
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, field
 
 from ..cache.manager import CacheNeeds
 from ..errors import ConfigError
@@ -73,6 +73,8 @@ class CacheView:
     owns: bool
     state: object = None
     own_state: object = None
+    # further states of the run by name (``CacheNeeds.states``), each [max_requests + 1, *shape]
+    states: dict = field(default_factory=dict)
 
 
 class Part:
@@ -135,7 +137,10 @@ class Mixer(Part):
 
 
 class FeedForward(Part):
-    """Token-wise ``forward(x) -> update`` [N, hidden]."""
+    """Token-wise ``forward(x) -> update`` [N, hidden].  A feed-forward with ``takes_add`` also takes
+    ``forward(x, add=...)``: a 32-bit [N, hidden] that is added to its update."""
+
+    takes_add = False
 
     def forward(self, x):
         raise NotImplementedError

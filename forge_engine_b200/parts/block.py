@@ -8,7 +8,8 @@ block's first norm (or the final norm) adds it in the same kernel that normalise
 "stream_mix" is the same pre-norm block over several copies of the residual stream that
 learned weights mix (or over one, with the update scaled by a constant).  "sandwich_conv" has
 a norm on both sides of every sublayer and a short convolution on its input; "output_norm" a
-norm on the sublayer's output only, the sublayer reading the stream itself.
+norm on the sublayer's output only, the sublayer reading the stream itself.  "parallel" has one norm
+that mixer and feed-forward both read, and one sum of both updates.
 """
 
 from __future__ import annotations
@@ -443,3 +444,60 @@ class OutputNormBlock:
 
 
 register_arrangement("output_norm", OutputNormBlock, replace=True)
+
+
+class ParallelBlock:
+    """Mixer and feed-forward side by side on one norm: with y = norm1(h), h += mixer(y) + ff(y).
+
+    The residual stream ``h`` is 32-bit.  The mixer's update (32-bit sums of its last projection)
+    joins the feed-forward's in that part's own last kernel where it takes one (``takes_add``), so
+    that the block hands a single update on, unadded, as the "pre_norm" block does.  A mixer with
+    ``enter`` reads more of the stream than the normalised row and makes its input itself, together
+    with the rounded row the feed-forward reads."""
+
+    roles = ("input_norm", "mixer", "ffn")
+
+    def __init__(self, spec, weights: dict, ctx: BuildContext) -> None:
+        self.ctx = ctx
+        self.input_norm = build_part(spec.input_norm, weights["input_norm"], ctx)
+        self.mixer = build_part(spec.mixer, weights["mixer"], ctx)
+        self.ffn = None if spec.ffn is None else build_part(spec.ffn, weights["ffn"], ctx)
+
+    @classmethod
+    def weight_shapes(cls, spec) -> dict:
+        """role -> {local name -> WeightInfo}"""
+        return {role: part_class(getattr(spec, role)).weight_shapes(getattr(spec, role)) for role in cls.roles
+                if getattr(spec, role) is not None}
+
+    def cache_needs(self):
+        return self.mixer.cache_needs()
+
+    def plan_step(self, entries: list, page_size: int, plans: dict) -> None:
+        planner = getattr(self.mixer, "plan_step", None)
+        if planner is not None:
+            planner(entries, page_size, plans)
+
+    @property
+    def graph_safe(self) -> bool:
+        return all(getattr(part, "graph_safe", False) for part in (self.input_norm, self.mixer, self.ffn) if part is not None)
+
+    def forward(self, h, pending, batch, cache: CacheView, shift=None):
+        """``shift``: None, a 32-bit vector, or 32-bit [N, hidden], added to ``h`` before anything else."""
+        with self.ctx.section("input_norm"):
+            enter = getattr(self.mixer, "enter", None)
+            if enter is None:
+                u = normed = self.input_norm.add_forward(h, pending) if shift is None else \
+                    self.input_norm.add_forward(h, pending, shift=shift)
+            else:
+                u, normed = enter(h, pending, shift, self.input_norm, batch, cache, self.ffn is not None)
+        with self.ctx.section("mixer"):
+            update = self.mixer.forward(u, batch, cache)
+        if self.ffn is None:
+            return update
+        with self.ctx.section("ffn"):
+            if self.ffn.takes_add and update.dtype == torch.float32:
+                return self.ffn.forward(normed, add=update)
+            return self.ffn.forward(normed).float().add_(update)
+
+
+register_arrangement("parallel", ParallelBlock, replace=True)

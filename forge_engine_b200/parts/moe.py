@@ -36,6 +36,7 @@ def _shared_spec(spec):
 
 class RoutedMLP(FeedForward):
     graph_safe = True
+    takes_add = True      # another sublayer's update joins in the kernel that sums a token's rows
 
     def __init__(self, spec, weights: dict, ctx: BuildContext) -> None:
         if spec.score not in ("sigmoid", "softmax"):
@@ -81,6 +82,10 @@ class RoutedMLP(FeedForward):
                 rows.append(weights["shared.sg"].reshape(1, -1))
         self.router = torch.cat([r.float() for r in rows], dim=0).contiguous()
         del rows
+        self.router_bias = None
+        if getattr(spec, "router_bias", False):
+            self.router_bias = torch.zeros(self.router.shape[0], dtype=torch.float32, device=self.router.device)
+            self.router_bias[: self.experts + self.identity].copy_(weights["router.b"])
         names = [local_name(unit, n) for n in self._unit_names(unit)]
         # bfloat16 with sizes in sixteens: the products run on the tcgen05 kernel in its grouped
         # form, gate and up as one matrix per expert whose rows alternate 16 gate and 16 up features
@@ -130,6 +135,8 @@ class RoutedMLP(FeedForward):
         h, unit = spec.hidden_size, spec.expert
         outputs = spec.experts + int(getattr(spec, "identity", 0) or 0)
         shapes = {"router": WeightInfo((outputs, h))}
+        if getattr(spec, "router_bias", False):
+            shapes["router.b"] = WeightInfo((outputs,), "bias")
         if getattr(spec, "correction", False):
             shapes["correction"] = WeightInfo((outputs,), "bias")
         names = [local_name(unit, n) for n in cls._unit_names(unit)]
@@ -153,7 +160,8 @@ class RoutedMLP(FeedForward):
         per_expert = slots / self.experts
         return 16 if per_expert <= 16 else 32 if per_expert <= 32 else 64 if per_expert <= 96 else 128
 
-    def forward(self, x):
+    def forward(self, x, add=None):
+        """``add`` (32-bit [N, width]) is added to the update, in the kernel that sums a token's rows."""
         n = x.shape[0]
         slots = n * self.top
         device = x.device
@@ -161,9 +169,9 @@ class RoutedMLP(FeedForward):
         with section("ffn.router"):
             logits = torch.empty((n, self.router.shape[0]), dtype=torch.float32, device=device)
             if self.width <= 48 * 1024:
-                native.moe_logits(x, self.router, logits)
+                native.moe_logits(x, self.router, logits, self.router_bias)
             else:
-                native.gemm_simt(x, self.router, logits)
+                native.gemm_simt(x, self.router, logits, self.router_bias)
         tile_rows = self.tile_rows(slots) if self.fused else 0
         max_tiles = native.moe_max_tiles(slots, self.experts, tile_rows)
         with section("ffn.route"):
@@ -204,7 +212,7 @@ class RoutedMLP(FeedForward):
             native.moe_combine(rows, plan, self.top, out, slot_weight=None if self.weight_on_input else weight,
                                shared=shared,
                                shared_logit=logits[:, self.experts + self.identity] if self.shared_gate else None,
-                               identity_input=x if self.identity else None, experts=self.experts)
+                               identity_input=x if self.identity else None, experts=self.experts, add=add)
         return out
 
 

@@ -7,6 +7,8 @@ are the same in every layer: ``table`` takes them once per step (in 32-bit, not 
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ..ops import native
@@ -33,20 +35,36 @@ class RotaryEncoding(PositionEncoding):
             self.inv_freq = (1.0 / (spec.theta**exponent)).to(ctx.device).contiguous()
         self.scaling = getattr(spec, "scaling", None)
         self.exact = bool(getattr(spec, "exact_frequencies", False))
-        if self.scaling is not None or getattr(spec, "exact_frequencies", False):
+        self.yarn = getattr(spec, "yarn", None)
+        self.amplitude = 1.0         # what cosine and sine are multiplied by
+        if self.scaling is not None or self.exact or self.yarn is not None:
             exponent = torch.arange(0, spec.rotary_dim, 2, dtype=torch.float64) / spec.rotary_dim
             freq = self.theta ** -exponent
             if self.scaling is not None:
                 freq = self.stretch(freq, self.scaling)
+            if self.yarn is not None:
+                freq, self.amplitude = self.ramp(freq, self.theta, spec.rotary_dim, self.yarn)
             self.inv_freq = freq.float().to(ctx.device).contiguous()
+
+    @staticmethod
+    def ramp(freq: torch.Tensor, theta: float, dims: int, yarn: tuple) -> tuple:
+        """(frequencies, factor of cosine and sine) after blending every frequency with its
+        ``factor``-th part by a ramp between the dimensions that turn ``fast`` and ``slow`` times
+        within ``original`` positions (64-bit)."""
+        factor, original, fast, slow = (float(v) for v in yarn)
+        if min(factor, original, fast, slow) <= 0 or theta <= 0 or theta == 1:
+            raise ValueError("frequency scaling needs positive numbers and a base other than 1")
+        place = lambda turns: dims * math.log(original / (2.0 * math.pi * turns)) / (2.0 * math.log(theta))  # noqa: E731
+        low, high = max(math.floor(place(fast)), 0), min(math.ceil(place(slow)), dims - 1)
+        index = torch.arange(freq.numel(), dtype=torch.float64)
+        part = ((index - low) / max(high - low, 0.001)).clamp(0.0, 1.0)
+        return freq / factor * part + freq * (1.0 - part), 0.1 * math.log(factor) + 1.0
 
     @staticmethod
     def stretch(freq: torch.Tensor, scaling: tuple) -> torch.Tensor:
         """Frequencies stretched by wavelength l = 2 pi / f (64-bit in, 64-bit out): kept below
         original / high, divided by ``factor`` above original / low, and blended in between with
         s = (original / l - low) / (high - low) as (1 - s) f / factor + s f."""
-        import math
-
         factor, low, high, original = (float(v) for v in scaling)
         if factor <= 0 or high <= low or original <= 0:
             raise ValueError("frequency scaling needs factor > 0, original > 0 and high > low")
@@ -61,11 +79,11 @@ class RotaryEncoding(PositionEncoding):
     def table(self, batch) -> torch.Tensor:
         """[tokens, rotary_dim / 2, 2] (cos, sin) of this step's angles; worked out by the
         first layer that asks and shared through the batch."""
-        key = ("rotary", self.theta, self.rotary_dim, self.interleaved, self.scaling, self.exact)
+        key = ("rotary", self.theta, self.rotary_dim, self.interleaved, self.scaling, self.exact, self.yarn)
         table = batch.shared.get(key)
         if table is None:
             table = torch.empty((batch.n_tokens, self.rotary_dim // 2, 2), dtype=torch.float32, device=self.inv_freq.device)
-            native.rope_table(batch.positions, self.inv_freq, table)
+            native.rope_table(batch.positions, self.inv_freq, table, self.amplitude)
             batch.shared[key] = table
         return table
 
