@@ -538,7 +538,8 @@ def design_compare(args) -> int:
     of `--layers` (4) layers of one kind: the Qwen3 layer, the Zofadra attention, latent
     attention and linear-recurrence layers, the Tekilorn differential, gated window and
     routed layers, the Zabutar gated-recurrence, biased-attention and routed layers and the Nuvivik
-    attention, latent and routed layers at the same sizes, plus a model of each design that mixes its layers.
+    attention, latent and routed layers and the Lofuvik time-mixing, delta-rule and side-by-side
+    layers at the same sizes, plus a model of each design that mixes its layers.
     One JSON line per model: tokens/s, ms per step, the median device time of every part of a
     step (CUDA events round each part, in a second runner) and, for the token-mixing kernel,
     its share of the measured peaks (prefill: its flops over the library GEMM's burst rate;
@@ -659,6 +660,34 @@ def design_compare(args) -> int:
             "nuvivik-routed": nuvivik([dict(n_attention, mlp=n_routed)] * layers),
             "nuvivik-mixed": nuvivik([n_latent, dict(n_latent, mlp=n_routed), n_latent, dict(n_attention, mlp=n_routed)]),
         })
+        # Lofuvik at the same sizes: time mixing and the matrix memory with the state sizes of the other
+        # recurrences, the delta rule with half as many query/key heads, attention at Qwen3's head sizes
+        # without a window (capped, sinks, a gate per element, half the head rotated); every
+        # feed-forward is routed, 2 of 16 gated experts of ff / 2: as many active weights per token as
+        # the dense one.  "-mixers" leave the feed-forward out.
+        l_routed = {"kind": "moe", "expert": {"ff": z["ff"] // 2}, "router": {"experts": 16, "top": 2}}
+        l_wkv = {"type": "wkv", "mlp": l_routed, "mixer": {"heads": H, "dim": rec["dim"], "rank": 64}}
+        l_delta = {"type": "delta", "mlp": l_routed, "mixer": {
+            "heads": H, "kv_heads": H // 2, "dim": rec["dim"], "vdim": rec["vdim"], "conv": 4}}
+        l_parallel = {"type": "parallel", "mlp": l_routed, "mixer": {
+            "left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "softcap": 30.0,
+                     "rot": {"base": 1e6, "dims": D // 2, "scaling": {"factor": 4.0, "original": 8192, "fast": 32.0, "slow": 1.0}}},
+            "right": {"heads": H, "dim": rec["dim"], "vdim": rec["vdim"], "gate_cap": 15.0}}}
+
+        def lofuvik(kinds, loop=None):
+            raw = {"architecture": "Lofuvik", "vocab": vocab, "width": W, "norm": {"eps": 1e-5}, "layers": kinds}
+            if loop:
+                raw["loop"] = loop
+            return raw
+
+        bare = lambda layer: dict(layer, mlp=None)                                 # noqa: E731
+        models.update({
+            "lofuvik-wkv": lofuvik([bare(l_wkv)] * layers),
+            "lofuvik-delta": lofuvik([bare(l_delta)] * layers),
+            "lofuvik-parallel": lofuvik([bare(l_parallel)] * layers),
+            "lofuvik-routed": lofuvik([l_delta] * layers),
+            "lofuvik-mixed": lofuvik([l_wkv, l_delta, l_parallel, l_wkv], loop={"start": 1, "stop": 3, "times": 2}),
+        })
         if args.design_models:
             wanted = [w for w in args.design_models.split(",") if w]
             models = {name: raw for name, raw in models.items() if any(name.startswith(w) for w in wanted)}
@@ -680,13 +709,21 @@ def design_compare(args) -> int:
         mixer_cost["zabutar-attention"] = mixer_cost["qwen3"]
         mixer_cost["nuvivik-attention"] = mixer_cost["nuvivik-routed"] = mixer_cost["qwen3-window"]
         mixer_cost["nuvivik-latent"] = (2 * H * (2 * rank + rot) * seen(window), batch * window * (rank + rot) * 2)
+        # time mixing also reads a decay per key channel; the delta rule has two more products per token
+        mixer_cost["lofuvik-wkv"] = (6 * H * rec["dim"] * rec["vdim"] * CONTEXT, mixer_cost["zofadra-recurrence"][1])
+        mixer_cost["lofuvik-delta"] = mixer_cost["lofuvik-routed"] = (
+            8 * H * rec["dim"] * rec["vdim"] * CONTEXT, mixer_cost["zofadra-recurrence"][1])
+        mixer_cost["lofuvik-parallel"] = mixer_cost["qwen3"]
+        second_cost = {"lofuvik-parallel": ("mixer.recurrence", *mixer_cost["zofadra-recurrence"])}
         mixer_part = {"qwen3": "mixer.attention", "qwen3-window": "mixer.attention", "zofadra-attention": "mixer.attention",
                       "zofadra-latent": "mixer.attention", "zofadra-recurrence": "mixer.recurrence",
                       "tekilorn-differential": "mixer.attention", "tekilorn-window": "mixer.attention",
                       "tekilorn-routed": "mixer.attention", "zabutar-recurrence": "mixer.recurrence",
                       "zabutar-routed": "mixer.recurrence", "zabutar-attention": "mixer.attention",
                       "nuvivik-attention": "mixer.attention", "nuvivik-routed": "mixer.attention",
-                      "nuvivik-latent": "mixer.attention"}
+                      "nuvivik-latent": "mixer.attention", "lofuvik-wkv": "mixer.recurrence",
+                      "lofuvik-delta": "mixer.recurrence", "lofuvik-routed": "mixer.recurrence",
+                      "lofuvik-parallel": "mixer.attention"}
         for name, raw in models.items():
             n_layers = len(raw["layers"]) if "layers" in raw else raw["num_hidden_layers"]
             pages = batch * (-(-(CONTEXT + 64) // PAGE) + 1) + -(-CONTEXT // PAGE) + 8
@@ -751,10 +788,13 @@ def design_compare(args) -> int:
                 else:
                     parts = runner.timings(reset=True)["parts"]
                     result["decode_parts_ms"] = {k: round(v["median"], 4) for k, v in parts.items()}
+            timed_parts = []
             if name in mixer_cost:
-                flops, moved = mixer_cost[name]
-                part = mixer_part[name]
-                result["mixer_kernel"] = {
+                timed_parts.append(("mixer_kernel", mixer_part[name], *mixer_cost[name]))
+            if name in second_cost:
+                timed_parts.append(("second_mixer_kernel", *second_cost[name]))
+            for key, part, flops, moved in timed_parts:
+                result[key] = {
                     "part": part,
                     "prefill_ms": result["prefill_parts_ms"].get(part),
                     "prefill_frac_of_gemm_peak": round(flops / (result["prefill_parts_ms"][part] * 1e-3) / (bf16_tflops * 1e12), 4),
