@@ -38,65 +38,77 @@ struct DeltaPrepare {
   int n_tokens;
 };
 
-// One token: its channels' convolution from `row(j)` (the input j tokens back, or a null pointer
-// before the start), then unit vectors and gates.
+#define DP_WARPS 4
+
+// One token's channels of one row - a q, k or v head - by a warp: convolution from `input(j)` (the
+// inputs j tokens back), silu, and for q and k the unit vector.  `buf` is the warp's own; a lane reads
+// back only what it wrote.
 template <typename F>
-__device__ __forceinline__ void delta_prepare_token(const DeltaPrepare& p, int t, float* buf, F row) {
-  const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv;
-  float* out = p.out + (size_t)t * channels;
-  for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+__device__ __forceinline__ void delta_prepare_row(const DeltaPrepare& p, int t, int r, float* buf, F input) {
+  const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv, lane = threadIdx.x & 31;
+  const bool unit = r < 2 * p.kv_heads;
+  const int base = unit ? r * p.dk : 2 * qk + (r - 2 * p.kv_heads) * p.dv, size = unit ? p.dk : p.dv;
+  float* out = p.out + (size_t)t * channels + base;
+  float ss = 0.f;
+  for (int d = lane; d < size; d += 32) {
     float sum = 0.f;
-    for (int j = p.taps - 1; j >= 0; --j) sum = fmaf(p.conv[(size_t)(p.taps - 1 - j) * channels + c], row(j)[c], sum);
+#pragma unroll 4
+    for (int j = p.taps - 1; j >= 0; --j) sum = fmaf(p.conv[(size_t)(p.taps - 1 - j) * channels + base + d], input(j)[base + d], sum);
     const float y = sum / (1.f + expf(-sum));
-    if (c < 2 * qk) buf[c] = y;
-    else out[c] = y;
+    if (unit) buf[d] = y;
+    else out[d] = y;
+    ss = fmaf(y, y, ss);
   }
-  __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = blockDim.x >> 5;
-  const float q_scale = 1.f / sqrtf((float)p.dk);
-  for (int h = warp; h < 2 * p.kv_heads; h += warps) {
-    float ss = 0.f;
-    for (int d = lane; d < p.dk; d += 32) ss = fmaf(buf[h * p.dk + d], buf[h * p.dk + d], ss);
-    const float inv = (h < p.kv_heads ? q_scale : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
-    for (int d = lane; d < p.dk; d += 32) out[h * p.dk + d] = buf[h * p.dk + d] * inv;
-  }
+  if (!unit) return;
+  const float inv = (r < p.kv_heads ? 1.f / sqrtf((float)p.dk) : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
+  for (int d = lane; d < size; d += 32) out[d] = buf[d] * inv;
+}
+
+__device__ __forceinline__ void delta_prepare_gates(const DeltaPrepare& p, int t) {
+  const float* src = p.proj + (size_t)t * p.ld;
   for (int h = threadIdx.x; h < p.heads; h += blockDim.x) {
-    const float* src = p.proj + (size_t)t * p.ld;
     float* dst = p.gates + ((size_t)t * p.heads + h) * 2;
     dst[0] = 1.f / (1.f + expf(-src[p.b_off + h]));
     dst[1] = -expf(p.a_log[h]) * sr_softplus(src[p.a_off + h] + p.dt_bias[h]);
   }
-  __syncthreads();
 }
 
-__global__ void __launch_bounds__(256) delta_prepare_kernel(DeltaPrepare p) {
-  extern __shared__ __align__(16) float buf[];      // q and k of a token
+__global__ void __launch_bounds__(32 * DP_WARPS) delta_prepare_kernel(DeltaPrepare p) {
+  extern __shared__ __align__(16) float smem[];      // [DP_WARPS][dk]
   pdl_trigger();
   pdl_wait();
-  const int back = p.taps - 1;
+  const int back = p.taps - 1, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int r = blockIdx.y * DP_WARPS + warp, rows = 2 * p.kv_heads + p.heads;
+  float* buf = smem + warp * p.dk;
   if ((int)blockIdx.x < p.n_tokens) {
     // a token with all its taps inside the step
     const int t = blockIdx.x;
     if (t - p.cu_tokens[p.token_entry[t]] < back) return;
-    delta_prepare_token(p, t, buf, [&](int j) { return p.proj + (size_t)(t - j) * p.ld; });
+    if (r < rows) delta_prepare_row(p, t, r, buf, [&](int j) { return p.proj + (size_t)(t - j) * p.ld; });
+    if (blockIdx.y == 0) delta_prepare_gates(p, t);
     return;
   }
   // an entry's edge: its first taps - 1 tokens, then the state for the next step
   const int entry = blockIdx.x - p.n_tokens;
-  const int first = p.cu_tokens[entry], count = p.cu_tokens[entry + 1] - first;
+  const int first = p.cu_tokens[entry], count = p.cu_tokens[entry + 1] - first, edge = min(count, back);
   if (count <= 0) return;
-  const int channels = 2 * p.kv_heads * p.dk + p.heads * p.dv;
+  if (blockIdx.y == 0)
+    for (int i = 0; i < edge; ++i) delta_prepare_gates(p, first + i);
+  if (r >= rows) return;
+  const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv;
   float* st = p.state + (size_t)p.slots[entry] * back * channels;
-  for (int i = 0; i < min(count, back); ++i)
-    delta_prepare_token(p, first + i, buf, [&](int j) {
+  for (int i = 0; i < edge; ++i)
+    delta_prepare_row(p, first + i, r, buf, [&](int j) {
       return j <= i ? p.proj + (size_t)(first + i - j) * p.ld : (const float*)st + (size_t)(back + i - j) * channels;
     });
-  // the last taps - 1 rows of (state rows, the step's rows); a channel is one thread's, which reads
-  // a state row only before it overwrites it
-  for (int c = threadIdx.x; c < channels; c += blockDim.x)
-    for (int r = 0; r < back; ++r) {
-      const int at = count + r;
-      st[(size_t)r * channels + c] = at < back ? st[(size_t)at * channels + c] : p.proj[(size_t)(first + at - back) * p.ld + c];
+  // the last taps - 1 rows of (state rows, the step's rows); a channel is one lane's, which reads a
+  // state row only before it overwrites it
+  const int base = r < 2 * p.kv_heads ? r * p.dk : 2 * qk + (r - 2 * p.kv_heads) * p.dv;
+  for (int d = lane; d < (r < 2 * p.kv_heads ? p.dk : p.dv); d += 32)
+    for (int k = 0; k < back; ++k) {
+      const int at = count + k;
+      st[(size_t)k * channels + base + d] =
+          at < back ? st[(size_t)at * channels + base + d] : p.proj[(size_t)(first + at - back) * p.ld + base + d];
     }
 }
 
@@ -107,10 +119,11 @@ FE_EXPORT int fe_delta_prepare(const float* proj, long long ld, int b_off, int a
   if (n_tokens <= 0) return 0;
   if (taps < 1 || kv_heads < 1 || heads < 1 || dk < 1 || dv < 1 || heads % kv_heads || (taps > 1 && state == nullptr)) return FE_ERR_BAD_SHAPE;
   DeltaPrepare p{proj, ld, b_off, a_off, conv, taps, state, slots, cu_tokens, token_entry, a_log, dt_bias, kv_heads, dk, heads, dv, out, gates, n_tokens};
-  const size_t smem = sizeof(float) * (size_t)2 * kv_heads * dk;
-  if (smem > 200 * 1024) return FE_ERR_TOO_LARGE;
-  if (smem > 48 * 1024) cudaFuncSetAttribute(delta_prepare_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const int rc = fe_launch_dependent(delta_prepare_kernel, dim3(n_tokens + (taps > 1 ? n_entries : 0)), dim3(256), smem, stream, p);
+  const size_t smem = sizeof(float) * (size_t)DP_WARPS * dk;
+  const int pieces = (2 * kv_heads + heads + DP_WARPS - 1) / DP_WARPS;
+  if (smem > 48 * 1024 || pieces > 65535) return FE_ERR_TOO_LARGE;
+  const int rc = fe_launch_dependent(delta_prepare_kernel, dim3(n_tokens + (taps > 1 ? n_entries : 0), pieces), dim3(32 * DP_WARPS), smem,
+                                     stream, p);
   return rc ? rc : fe_last_error();
 }
 
@@ -125,7 +138,8 @@ struct Delta {
   // chunk-parallel scratch, per (slot, head)
   float* w;                 // [dk][SR_LONG]: W transposed
   float* u;                 // [SR_LONG][dv]: U, then (chain) u
-  float* starts;            // [dk, dv]: the state before the chunk
+  float* before;            // [dk, dv]: the state before the chunk
+  float* decays;            // [SR_LONG + 4]: e^(c_end - c_t) per token, then e^(c_end)
 
   static constexpr int VECS = 2, SCALARS = 2, EXTRA = 0;
   static constexpr bool SCORES = true, NORMALISER = false;
@@ -178,35 +192,33 @@ struct Delta {
   __device__ __forceinline__ float scale(const float*, const float*, int) const { return 1.f; }
 
   // -- chunk form --
-  // sums of log g up to every token of the chunk (tokens past the end keep the last sum)
+  // sums of log g up to the chunk's tokens lane and 32 + lane, by one warp (tokens past the end keep
+  // the last sum)
   __device__ __forceinline__ void chunk_sums(const StateRun& p, int head, const ChunkAt& at, double* c) const {
-    __shared__ float logs[SR_LONG];
-    if (threadIdx.x < SR_LONG) logs[threadIdx.x] = (int)threadIdx.x < at.count ? log_decay(p, head, at.first + threadIdx.x) : 0.f;
-    __syncthreads();
-    if (threadIdx.x == 0) {
-      double sum = 0.0;
-      for (int t = 0; t < SR_LONG; ++t) {
-        sum += (double)logs[t];
-        c[t] = sum;
-      }
-    }
-    __syncthreads();
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) c[h] = lane + 32 * h < at.count ? (double)log_decay(p, head, at.first + lane + 32 * h) : 0.0;
+    sr_running_sum(c[0], c[1]);
   }
   __device__ __forceinline__ size_t cell(const StateRun& p, const ChunkAt& at, int head) const { return (size_t)at.slot * p.heads + head; }
-  __device__ __forceinline__ float query(const StateRun& p, int head, const ChunkAt& at, int t, int d) const { return q_row(p, head, at.first + t)[d]; }
-  __device__ __forceinline__ float key(const StateRun& p, int head, const ChunkAt& at, int t, int d) const { return k_row(p, head, at.first + t)[d]; }
-  __device__ __forceinline__ float other(const StateRun& p, int head, const ChunkAt& at, int t, int c) const {
-    return u[(cell(p, at, head) * SR_LONG + t) * p.dv + c];
+  __device__ __forceinline__ Rows queries(const StateRun& p, int head, const ChunkAt& at) const { return Rows{q_row(p, head, at.first), ld}; }
+  __device__ __forceinline__ float query_mul() const { return 1.f; }
+  __device__ __forceinline__ Rows keys(const StateRun& p, int head, const ChunkAt& at) const { return Rows{k_row(p, head, at.first), ld}; }
+  __device__ __forceinline__ Rows others(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{u + cell(p, at, head) * SR_LONG * p.dv, p.dv};
   }
-  __device__ __forceinline__ float start(const StateRun& p, int head, const ChunkAt& at, int d, int c) const {
-    return starts[(cell(p, at, head) * p.dk + d) * p.dv + c];
+  __device__ __forceinline__ Rows starts(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{before + cell(p, at, head) * p.dk * p.dv, p.dv};
   }
   __device__ __forceinline__ void out_begin(const StateRun& p, int head, const ChunkAt& at, double* rt, double* ct, float* ea, float*) const {
-    chunk_sums(p, head, at, rt);
-    if (threadIdx.x < SR_LONG) {
-      const int t = threadIdx.x;
-      ct[t] = -rt[t];
-      ea[t] = t < at.count ? expf((float)rt[t]) : 0.f;
+    double c[2];
+    chunk_sums(p, head, at, c);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = (threadIdx.x & 31) + 32 * h;
+      rt[t] = c[h];
+      ct[t] = -c[h];
+      ea[t] = t < at.count ? expf((float)c[h]) : 0.f;
     }
   }
 };
@@ -224,12 +236,23 @@ __global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const S
   __shared__ float bt[SR_LONG], be[SR_LONG];
   float* L = smem;                           // [SR_LONG rows t][SR_LONG]
   float* kt = L + SR_LONG * SR_LONG;         // [dk][SR_TP]
-  sr_stage_transposed(kt, dk, at.count, [&](int t, int d) { return m.key(p, head, at, t, d); });
-  m.chunk_sums(p, head, at, c);
-  if (tid < SR_LONG) {
-    bt[tid] = tid < at.count ? m.beta(p, head, at.first + tid) : 0.f;
-    be[tid] = bt[tid] * expf((float)c[tid]);
+  if (tid < 32) {
+    double sums[2];
+    m.chunk_sums(p, head, at, sums);
+    const double end = __shfl_sync(0xffffffffu, sums[1], 31);
+    float* decays = m.decays + m.cell(p, at, head) * (SR_LONG + 4);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = tid + 32 * h;
+      const float beta = t < at.count ? m.beta(p, head, at.first + t) : 0.f;
+      c[t] = sums[h];
+      bt[t] = beta;
+      be[t] = beta * expf((float)sums[h]);
+      decays[t] = t < at.count ? expf((float)(end - sums[h])) : 0.f;
+    }
+    if (tid == 0) decays[SR_LONG] = expf((float)end);
   }
+  sr_stage_transposed(kt, m.keys(p, head, at), dk, at.count);
   __syncthreads();
   for (int item = tid; item < 256; item += blockDim.x) {
     const int row = 4 * (item & 15), col = 4 * (item >> 4);
@@ -259,16 +282,16 @@ __global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const S
 #pragma unroll
     for (int t = 1; t < SR_LONG; ++t) {
       const float4* l4 = reinterpret_cast<const float4*>(L + t * SR_LONG);
-      float s0 = 0.f, s1 = 0.f;
+      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
 #pragma unroll
       for (int j = 0; j < t; j += 4) {
         const float4 l = l4[j >> 2];           // entries at and past the diagonal are zero
         s0 = fmaf(l.x, x[j], s0);
         s1 = fmaf(l.y, x[j + 1], s1);
-        s0 = fmaf(l.z, x[j + 2], s0);
-        s1 = fmaf(l.w, x[j + 3], s1);
+        s2 = fmaf(l.z, x[j + 2], s2);
+        s3 = fmaf(l.w, x[j + 3], s3);
       }
-      x[t] -= s0 + s1;
+      x[t] -= (s0 + s1) + (s2 + s3);
     }
     if (i < dk) {
       float* dst = m.w + (cell * dk + i) * SR_LONG;
@@ -282,15 +305,16 @@ __global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const S
   }
 }
 
-// The chain over an entry's chunks for one head and 32 value columns: u = U - W S, then
-// S <- e^(c_end) S + sum_j e^(c_end - c_j) k_j u_j^T.  The state's columns stay in shared memory.
-// Thread (rg, cg) owns four rows and two columns of a product.
-#define DC_COLS 32
+// The chain over an entry's chunks for one head and COLS value columns: u = U - W S, then
+// S <- e^(c_end) S + sum_j k_j (e^(c_end - c_j) u_j)^T.  The state's columns stay in shared memory;
+// the next chunk's W and keys are on their way while a chunk is worked on.  Thread (rg, cg) of
+// 16 x COLS / 2 owns four rows and two columns of a product.
+template <int COLS>
 __device__ __forceinline__ void dc_mm42(float (&acc)[4][2], const float* xt, int ldx, const float* y, int depth, int row, int col) {
 #pragma unroll 8
   for (int k = 0; k < depth; ++k) {
     const float4 x = *reinterpret_cast<const float4*>(xt + k * ldx + row);
-    const float2 b = *reinterpret_cast<const float2*>(y + k * DC_COLS + col);
+    const float2 b = *reinterpret_cast<const float2*>(y + k * COLS + col);
     acc[0][0] = fmaf(x.x, b.x, acc[0][0]), acc[0][1] = fmaf(x.x, b.y, acc[0][1]);
     acc[1][0] = fmaf(x.y, b.x, acc[1][0]), acc[1][1] = fmaf(x.y, b.y, acc[1][1]);
     acc[2][0] = fmaf(x.z, b.x, acc[2][0]), acc[2][1] = fmaf(x.z, b.y, acc[2][1]);
@@ -298,11 +322,12 @@ __device__ __forceinline__ void dc_mm42(float (&acc)[4][2], const float* xt, int
   }
 }
 
-__global__ void __launch_bounds__(256) delta_chain_kernel(const Delta m, const StateRun p, int* status) {
+template <int COLS>
+__global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, const StateRun p, int* status) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
-  const int head = blockIdx.x, entry = blockIdx.y, col0 = blockIdx.z * DC_COLS, tid = threadIdx.x;
+  const int head = blockIdx.x, entry = blockIdx.y, col0 = blockIdx.z * COLS, tid = threadIdx.x;
   const int first = p.cu_tokens[entry], count = p.cu_tokens[entry + 1] - first;
   if (count < p.long_from) return;
   const int slot = p.slots[entry];
@@ -311,94 +336,109 @@ __global__ void __launch_bounds__(256) delta_chain_kernel(const Delta m, const S
     return;
   }
   const int dk = p.dk, dv = p.dv, kp = (dk + 63) / 64 * 64;
-  const int cols = min(DC_COLS, dv - col0);
-  __shared__ float w[SR_LONG], logs[SR_LONG];
-  __shared__ float keep;
-  float* S = smem;                           // [kp][DC_COLS]
-  float* wt = S + kp * DC_COLS;              // [dk][SR_LONG]
-  float* ks = wt + dk * SR_LONG;             // [SR_LONG][kp], weighted
-  float* us = ks + SR_LONG * kp;             // [SR_LONG][DC_COLS]
+  const int cols = min(COLS, dv - col0), half = dk * SR_LONG + SR_LONG * kp;
+  float* S = smem;                           // [kp][COLS]
+  float* us = S + kp * COLS;                 // [SR_LONG][COLS], weighted
+  float* buffers = us + SR_LONG * COLS;      // 2 x (W transposed [dk][SR_LONG], keys [SR_LONG][kp])
   const int row = 4 * (tid & 15), col = 2 * (tid >> 4);
   float* st = p.state + ((size_t)slot * p.heads + head) * dk * dv + col0;
-  for (int i = tid; i < kp * DC_COLS; i += blockDim.x) {
-    const int d = i / DC_COLS, c = i - d * DC_COLS;
+  for (int i = tid; i < kp * COLS; i += blockDim.x) {
+    const int d = i / COLS, c = i - d * COLS;
     S[i] = (d < dk && c < cols) ? st[(size_t)d * dv + c] : 0.f;
   }
+  for (int i = tid; i < 2 * half; i += blockDim.x) buffers[i] = 0.f;      // key channels past dk stay zero
+  __syncthreads();
   const int chunks = (count + SR_LONG - 1) / SR_LONG;
+  const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
+  const size_t cell0 = (size_t)sr_slot(first, entry, 0) * p.heads + head;
+  const Rows keys{m.k_row(p, head, first), m.ld};
+  const bool wide = keys.wide(dk);
+  auto fetch = [&](int chunk, float* buf) {
+    const float* w = m.w + (cell0 + (size_t)chunk * p.heads) * dk * SR_LONG;
+    for (int i = 4 * tid; i < dk * SR_LONG; i += 4 * blockDim.x) sr_copy16(buf + i, w + i);
+    const int have = min(SR_LONG, count - chunk * SR_LONG);
+    float* ks = buf + dk * SR_LONG;
+    for (int t = warp; t < SR_LONG; t += warps) {
+      float* dst = ks + t * kp;
+      if (t >= have) {
+        for (int d = lane; d < dk; d += 32) dst[d] = 0.f;
+      } else if (wide) {
+        for (int d = 4 * lane; d < dk; d += 128) sr_copy16(dst + d, keys.row(chunk * SR_LONG + t) + d);
+      } else {
+        for (int d = lane; d < dk; d += 32) sr_copy4(dst + d, keys.row(chunk * SR_LONG + t) + d);
+      }
+    }
+    sr_copy_commit();
+  };
+  fetch(0, buffers);
   for (int chunk = 0; chunk < chunks; ++chunk) {
-    ChunkAt at;
-    at.entry_first = first, at.first = first + chunk * SR_LONG, at.count = min(SR_LONG, count - chunk * SR_LONG);
-    at.slot = sr_slot(first, entry, chunk), at.chunks = chunks;
-    const size_t cell = m.cell(p, at, head);
-    __syncthreads();
-    if (tid < SR_LONG) logs[tid] = tid < at.count ? m.log_decay(p, head, at.first + tid) : 0.f;
-    const float4* wsrc = reinterpret_cast<const float4*>(m.w + cell * dk * SR_LONG);
-    for (int i = tid; i < dk * SR_LONG / 4; i += blockDim.x) reinterpret_cast<float4*>(wt)[i] = wsrc[i];
-    __syncthreads();
-    if (tid < SR_LONG) {
-      // e^(sum of the later logs): summed from the end, so that late tokens keep their precision
-      float after = 0.f;
-      for (int j = at.count - 1; j > tid; --j) after += logs[j];
-      w[tid] = tid < at.count ? expf(after) : 0.f;
-      if (tid == 0) keep = expf(after + logs[0]);
-    }
-    __syncthreads();
-    for (int i = tid; i < SR_LONG * kp; i += blockDim.x) {
-      const int t = i / kp, d = i - t * kp;
-      ks[i] = (t < at.count && d < dk) ? m.key(p, head, at, t, d) * w[t] : 0.f;
-    }
-    float a[4][2] = {};
-    dc_mm42(a, wt, SR_LONG, S, dk, row, col);
-    float* u = m.u + cell * SR_LONG * dv + col0;
+    const size_t cell = cell0 + (size_t)chunk * p.heads;
+    const float* buf = buffers + (chunk & 1) * half;
+    float* u = m.u + (cell * SR_LONG + row) * dv + col0 + col;
+    const float* decays = m.decays + cell * (SR_LONG + 4);
+    float x[4][2], w[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e)
+    for (int e = 0; e < 4; ++e) {
+      w[e] = decays[row + e];
+#pragma unroll
+      for (int b = 0; b < 2; ++b) x[e][b] = col + b < cols ? u[(size_t)e * dv + b] : 0.f;
+    }
+    const float keep = decays[SR_LONG];
+    sr_copy_wait<0>();
+    __syncthreads();
+    if (chunk + 1 < chunks) fetch(chunk + 1, buffers + ((chunk + 1) & 1) * half);
+    float a[4][2] = {};
+    dc_mm42<COLS>(a, buf, SR_LONG, S, dk, row, col);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
 #pragma unroll
       for (int b = 0; b < 2; ++b) {
-        float x = 0.f;
-        if (col + b < cols) {
-          x = u[(size_t)(row + e) * dv + col + b] - a[e][b];
-          u[(size_t)(row + e) * dv + col + b] = x;
-        }
-        us[(row + e) * DC_COLS + col + b] = x;
+        x[e][b] -= a[e][b];
+        if (col + b < cols) u[(size_t)e * dv + b] = x[e][b];
       }
+      *reinterpret_cast<float2*>(us + (row + e) * COLS + col) = make_float2(x[e][0] * w[e], x[e][1] * w[e]);
+    }
     // the state before the chunk, for state_out
-    float* dst = m.starts + cell * dk * dv + col0;
-    for (int i = tid; i < dk * DC_COLS; i += blockDim.x) {
-      const int d = i / DC_COLS, c = i - d * DC_COLS;
+    float* dst = m.before + cell * dk * dv + col0;
+    for (int i = tid; i < dk * COLS; i += blockDim.x) {
+      const int d = i / COLS, c = i - d * COLS;
       if (c < cols) dst[(size_t)d * dv + c] = S[i];
     }
     __syncthreads();
+    const float* ks = buf + dk * SR_LONG;
     for (int d0 = 0; d0 < kp; d0 += 64) {
       float b[4][2] = {};
-      dc_mm42(b, ks + d0, kp, us, at.count, row, col);
+      dc_mm42<COLS>(b, ks + d0, kp, us, SR_LONG, row, col);
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * DC_COLS + col);
+        float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * COLS + col);
         const float2 old = *s2;
         *s2 = make_float2(fmaf(keep, old.x, b[e][0]), fmaf(keep, old.y, b[e][1]));
       }
     }
   }
   __syncthreads();
-  for (int i = tid; i < dk * DC_COLS; i += blockDim.x) {
-    const int d = i / DC_COLS, c = i - d * DC_COLS;
+  for (int i = tid; i < dk * COLS; i += blockDim.x) {
+    const int d = i / COLS, c = i - d * COLS;
     if (c < cols) st[(size_t)d * dv + c] = S[i];
   }
 }
 
 static size_t delta_solve_smem(int dk) { return sizeof(float) * ((size_t)SR_LONG * SR_LONG + (size_t)dk * SR_TP); }
-static size_t delta_chain_smem(int dk) {
+// Value columns of a block of delta_chain: few where the heads are small, so that there are more blocks.
+static int delta_chain_cols(int dv) { return dv <= 64 ? 16 : 32; }
+static size_t delta_chain_smem(int dk, int cols) {
   const size_t kp = (size_t)(dk + 63) / 64 * 64;
-  return sizeof(float) * (kp * DC_COLS + (size_t)dk * SR_LONG + SR_LONG * kp + SR_LONG * DC_COLS);
+  return sizeof(float) * (kp * cols + (size_t)SR_LONG * cols + 2 * ((size_t)dk * SR_LONG + SR_LONG * kp));
 }
 static bool delta_chunk_takes(int dk, int dv) {
-  return chunk_takes(dk, dv, true) && delta_solve_smem(dk) <= 200 * 1024 && delta_chain_smem(dk) <= 200 * 1024;
+  return chunk_takes(dk, dv, true) && delta_solve_smem(dk) <= 200 * 1024 && delta_chain_smem(dk, delta_chain_cols(dv)) <= 200 * 1024;
 }
 
 FE_EXPORT long long fe_delta_rule_scratch(int tokens, int entries, int heads, int dk, int dv, int max_new) {
   const long long need = walk_in_stretches(dk, dv, 0) ? (long long)tokens * heads * dv : 0;
   if (max_new < SR_LONG_FROM || !delta_chunk_takes(dk, dv)) return need;
-  return (need + 3) / 4 * 4 + sr_slots(tokens, entries) * heads * ((long long)dk * SR_LONG + (long long)SR_LONG * dv + (long long)dk * dv);
+  return (need + 3) / 4 * 4 + sr_slots(tokens, entries) * heads * ((long long)dk * SR_LONG + (long long)SR_LONG * dv + (long long)dk * dv + SR_LONG + 4);
 }
 
 FE_EXPORT int fe_delta_rule(const float* qkv, long long ld, const float* gates, const float* gate, long long gate_ld,
@@ -408,7 +448,7 @@ FE_EXPORT int fe_delta_rule(const float* qkv, long long ld, const float* gates, 
   if (entries <= 0 || tokens <= 0) return 0;
   if (heads < 1 || kv_heads < 1 || heads % kv_heads || dk < 1 || dv < 1 || heads > 65535 || entries > 65535) return FE_ERR_BAD_SHAPE;
   StateRun p{state, state_rows, slots, cu_tokens, heads, dk, dv, 0, qkv + 2 * kv_heads * dk, ld, norm_w, 0, gate, gate_ld, 0, eps, out, nullptr, 0};
-  Delta m{qkv, ld, kv_heads, heads / kv_heads, gates, nullptr, nullptr, nullptr};
+  Delta m{qkv, ld, kv_heads, heads / kv_heads, gates, nullptr, nullptr, nullptr, nullptr};
   if (walk_in_stretches(dk, dv, 0)) {
     p.raw = scratch;
     scratch = scratch ? scratch + ((size_t)tokens * heads * dv + 3) / 4 * 4 : nullptr;
@@ -422,14 +462,22 @@ FE_EXPORT int fe_delta_rule(const float* qkv, long long ld, const float* gates, 
   const size_t cells = (size_t)sr_slots(tokens, entries) * heads;
   m.w = scratch;
   m.u = m.w + cells * dk * SR_LONG;
-  m.starts = m.u + cells * SR_LONG * dv;
+  m.decays = m.u + cells * SR_LONG * dv;
+  m.before = m.decays + cells * (SR_LONG + 4);
   size_t smem = delta_solve_smem(dk);
   cudaFuncSetAttribute(delta_solve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
   rc = fe_launch_dependent(delta_solve_kernel, dim3(heads, entries, chunks), dim3(128), smem, stream, m, p);
   if (rc) return rc;
-  smem = delta_chain_smem(dk);
-  cudaFuncSetAttribute(delta_chain_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  rc = fe_launch_dependent(delta_chain_kernel, dim3(heads, entries, (dv + DC_COLS - 1) / DC_COLS), dim3(256), smem, stream, m, p, status);
+  const int cols = delta_chain_cols(dv);
+  smem = delta_chain_smem(dk, cols);
+  const dim3 chain(heads, entries, (dv + cols - 1) / cols);
+  if (cols == 16) {
+    cudaFuncSetAttribute(delta_chain_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    rc = fe_launch_dependent(delta_chain_kernel<16>, chain, dim3(128), smem, stream, m, p, status);
+  } else {
+    cudaFuncSetAttribute(delta_chain_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    rc = fe_launch_dependent(delta_chain_kernel<32>, chain, dim3(256), smem, stream, m, p, status);
+  }
   if (rc) return rc;
   rc = launch_out(m, p, out_dtype, entries, chunks, stream);
   return rc ? rc : fe_last_error();

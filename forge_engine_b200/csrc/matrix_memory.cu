@@ -92,60 +92,58 @@ struct Memory {
   }
 
   // -- chunk form --
-  // F (sums of f up to every token) and i of a chunk in shared memory, by one warp; tokens past
-  // the end keep F and have i = 0
-  __device__ __forceinline__ void chunk_gates(const ChunkAt& at, int head, double* F, float* i_log, float* f_log) const {
-    const int tid = threadIdx.x;
-    if (tid < SR_LONG) {
-      float i = 0.f, f = 0.f;
-      if (tid < at.count) gates(at.first + tid, head, &i, &f);
-      i_log[tid] = i, f_log[tid] = f;
+  // i, f and the running sum F of f for a chunk's tokens lane and 32 + lane, by one warp; tokens
+  // past the end have f = 0 and i = minus infinity
+  struct Gates { double F[2]; float i[2]; };
+  __device__ __forceinline__ Gates chunk_gates(const ChunkAt& at, int head) const {
+    Gates g;
+    const int lane = threadIdx.x & 31;
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = lane + 32 * h;
+      float i = -INFINITY, f = 0.f;
+      if (t < at.count) gates(at.first + t, head, &i, &f);
+      g.i[h] = i, g.F[h] = (double)f;
     }
-    __syncthreads();
-    if (tid == 0) {
-      double sum = 0.0;
-      for (int t = 0; t < SR_LONG; ++t) {
-        sum += (double)f_log[t];
-        F[t] = sum;
-      }
-    }
-    __syncthreads();
+    sr_running_sum(g.F[0], g.F[1]);
+    return g;
   }
   __device__ __forceinline__ const float* chunk(const StateRun& p, const ChunkAt& at, int head) const {
     return sums + ((size_t)at.slot * p.heads + head) * ((size_t)p.dk * p.dv + p.dk);
   }
-  __device__ __forceinline__ float query(const StateRun& p, int head, const ChunkAt& at, int t, int d) const {
-    return q[(size_t)(at.first + t) * ld + (size_t)head * p.dk + d] * q_scale;
+  __device__ __forceinline__ Rows queries(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{q + (size_t)at.first * ld + (size_t)head * p.dk, ld};
   }
-  __device__ __forceinline__ float key(const StateRun& p, int head, const ChunkAt& at, int t, int d) const {
-    return k[(size_t)(at.first + t) * ld + (size_t)head * p.dk + d];
+  __device__ __forceinline__ float query_mul() const { return q_scale; }
+  __device__ __forceinline__ Rows keys(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{k + (size_t)at.first * ld + (size_t)head * p.dk, ld};
   }
-  __device__ __forceinline__ float other(const StateRun& p, int head, const ChunkAt& at, int t, int c) const {
-    return p.v[(size_t)(at.first + t) * p.v_ld + (size_t)head * p.dv + c];
+  __device__ __forceinline__ Rows others(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{p.v + (size_t)at.first * p.v_ld + (size_t)head * p.dv, p.v_ld};
   }
-  __device__ __forceinline__ float start(const StateRun& p, int head, const ChunkAt& at, int d, int c) const {
-    return chunk(p, at, head)[(size_t)d * p.dv + c];
+  __device__ __forceinline__ Rows starts(const StateRun& p, int head, const ChunkAt& at) const { return Rows{chunk(p, at, head), p.dv}; }
+  __device__ __forceinline__ const float* start_norm(const StateRun& p, int head, const ChunkAt& at) const {
+    return chunk(p, at, head) + (size_t)p.dk * p.dv;
   }
-  __device__ __forceinline__ float start_norm(const StateRun& p, int head, const ChunkAt& at, int d) const {
-    return chunk(p, at, head)[(size_t)p.dk * p.dv + d];
-  }
+  // m_t = F_t + max(m before the chunk, the largest i_j - F_j up to t): the recurrence's maximum
   __device__ __forceinline__ void out_begin(const StateRun& p, int head, const ChunkAt& at, double* rt, double* ct, float* ea,
                                             float* fl) const {
-    __shared__ float i_log[SR_LONG], f_log[SR_LONG];
-    chunk_gates(at, head, rt, i_log, f_log);          // rt holds F for now
-    if (threadIdx.x == 0) {
-      if (at.first == at.entry_first)      // m after the entry's last token, now that nobody reads the one before its first
-        top[(size_t)p.slots[blockIdx.y] * p.heads + head] = marks[((size_t)at.slot * p.heads + head) * 4 + 3];
-      const float m_start = marks[((size_t)at.slot * p.heads + head) * 4 + 2];
-      float m = m_start;
-      for (int t = 0; t < SR_LONG; ++t) {
-        m = fmaxf(f_log[t] + m, i_log[t]);
-        const double F = rt[t];
-        ct[t] = (double)i_log[t] - F;
-        ea[t] = t < at.count ? expf((float)(F + (double)m_start - (double)m)) : 0.f;
-        fl[t] = expf(-m);
-        rt[t] = F - (double)m;
-      }
+    const int lane = threadIdx.x & 31;
+    const size_t cell = (size_t)at.slot * p.heads + head;
+    if (lane == 0 && at.first == at.entry_first)      // m after the entry's last token, now that nobody reads the one before its first
+      top[(size_t)p.slots[blockIdx.y] * p.heads + head] = marks[cell * 4 + 3];
+    const double m_start = (double)marks[cell * 4 + 2];
+    const Gates g = chunk_gates(at, head);
+    double big[2] = {(double)g.i[0] - g.F[0], (double)g.i[1] - g.F[1]};
+    sr_running_max(big[0], big[1]);
+#pragma unroll
+    for (int h = 0; h < 2; ++h) {
+      const int t = lane + 32 * h;
+      const double F = g.F[h], m = F + fmax(m_start, big[h]);
+      rt[t] = F - m;
+      ct[t] = (double)g.i[h] - F;
+      ea[t] = t < at.count ? expf((float)(F + m_start - m)) : 0.f;
+      fl[t] = expf((float)-m);
     }
   }
 };
@@ -158,55 +156,57 @@ __global__ void __launch_bounds__(256) memory_sums_kernel(const Memory m, const 
   ChunkAt at;
   if (!sr_locate(p, &at)) return;
   const int head = blockIdx.x, dk = p.dk, dv = p.dv, tid = threadIdx.x;
-  __shared__ double F[SR_LONG];
-  __shared__ float i_log[SR_LONG], f_log[SR_LONG], w[SR_LONG];
-  const int kp = (dk + 63) / 64 * 64;
-  float* ks = smem;                       // [SR_LONG][kp], weighted
-  float* tile = ks + SR_LONG * kp;        // [SR_LONG][64]
-  m.chunk_gates(at, head, F, i_log, f_log);
+  __shared__ float w[SR_LONG];
+  float* ks = smem;                       // [SR_LONG][64]: 64 channels of the keys, weighted
+  float* tile = ks + SR_LONG * 64;        // [SR_LONG][64]
   if (tid < 32) {
-    const double end = F[at.count - 1];
-    float big = -INFINITY;
-    for (int t = tid; t < at.count; t += 32) big = fmaxf(big, (float)(end - F[t] + (double)i_log[t]));
-    big = warp_max(big);
-    for (int t = tid; t < SR_LONG; t += 32)
-      w[t] = t < at.count ? expf((float)(end - F[t] + (double)i_log[t] - (double)big)) : 0.f;
+    const Memory::Gates g = m.chunk_gates(at, head);
+    const double end = __shfl_sync(0xffffffffu, g.F[1], 31);
+    float x[2];
+#pragma unroll
+    for (int h = 0; h < 2; ++h) x[h] = (float)(end - g.F[h] + (double)g.i[h]);      // minus infinity past the end
+    const float big = warp_max(fmaxf(x[0], x[1]));
+#pragma unroll
+    for (int h = 0; h < 2; ++h) w[tid + 32 * h] = expf((float)(end - g.F[h] + (double)g.i[h] - (double)big));
     if (tid == 0) {
       float* mark = m.marks + ((size_t)at.slot * p.heads + head) * 4;
       mark[0] = big;
       mark[1] = (float)end;
     }
   }
-  __syncthreads();
-  for (int i = tid; i < SR_LONG * kp; i += blockDim.x) {
-    const int t = i / kp, d = i - t * kp;
-    ks[i] = (t < at.count && d < dk) ? m.key(p, head, at, t, d) * w[t] : 0.f;
-  }
-  __syncthreads();
   float* sum = m.sums + ((size_t)at.slot * p.heads + head) * ((size_t)dk * dv + dk);
-  for (int d = tid; d < dk; d += blockDim.x) {
-    float s = 0.f;
-    for (int t = 0; t < at.count; ++t) s += ks[t * kp + d];
-    sum[(size_t)dk * dv + d] = s;
-  }
+  const bool wide = (dv & 3) == 0 && ((uintptr_t)sum & 15) == 0;
   const int row = 4 * (tid & 15), col = 4 * (tid >> 4);
-  for (int c0 = 0; c0 < dv; c0 += 64) {
+  const Rows keys = m.keys(p, head, at), values = m.others(p, head, at);
+  for (int d0 = 0; d0 < dk; d0 += 64) {
     __syncthreads();
-    for (int i = tid; i < SR_LONG * 64; i += blockDim.x) {
-      const int t = i >> 6, c = c0 + (i & 63);
-      tile[i] = (t < at.count && c < dv) ? m.other(p, head, at, t, c) : 0.f;
-    }
+    sr_stage_columns(ks, keys, SR_LONG, at.count, d0, dk);
     __syncthreads();
-    for (int d0 = 0; d0 < dk; d0 += 64) {
+    for (int i = tid; i < SR_LONG * 64; i += blockDim.x) ks[i] *= w[i >> 6];
+    for (int c0 = 0; c0 < dv; c0 += 64) {
+      __syncthreads();
+      sr_stage_columns(tile, values, SR_LONG, at.count, c0, dv);
+      __syncthreads();
+      if (c0 == 0 && tid < 64 && d0 + tid < dk) {
+        float s = 0.f;
+#pragma unroll 8
+        for (int t = 0; t < SR_LONG; ++t) s += ks[t * 64 + tid];
+        sum[(size_t)dk * dv + d0 + tid] = s;
+      }
       float acc[4][4] = {};
-      sr_mm44(acc, ks + d0, kp, tile, 64, at.count, row, col);
+      sr_mm44(acc, ks, 64, tile, 64, at.count, row, col);
 #pragma unroll
       for (int a = 0; a < 4; ++a) {
         const int d = d0 + row + a;
         if (d >= dk) continue;
+        float* dst = sum + (size_t)d * dv + c0 + col;
+        if (wide && c0 + col < dv) {
+          store4(dst, acc[a]);
+        } else if (!wide) {
 #pragma unroll
-        for (int b = 0; b < 4; ++b)
-          if (c0 + col + b < dv) sum[(size_t)d * dv + c0 + col + b] = acc[a][b];
+          for (int b = 0; b < 4; ++b)
+            if (c0 + col + b < dv) dst[b] = acc[a][b];
+        }
       }
     }
   }
@@ -259,11 +259,9 @@ __global__ void __launch_bounds__(256) memory_scan_kernel(const Memory m, const 
   if (cell == 0) marks[3] = top;
 }
 
-static size_t memory_sums_smem(int dk) { return sizeof(float) * (size_t)SR_LONG * ((dk + 63) / 64 * 64 + 64); }
-
 FE_EXPORT long long fe_matrix_memory_scratch(int tokens, int entries, int heads, int dk, int dv, int max_new) {
   const long long need = walk_in_stretches(dk, dv, 1) ? (long long)tokens * heads * dv : 0;
-  if (max_new < SR_LONG_FROM || !chunk_takes(dk, dv, true) || memory_sums_smem(dk) > 200 * 1024) return need;
+  if (max_new < SR_LONG_FROM || !chunk_takes(dk, dv, true)) return need;
   return need + sr_slots(tokens, entries) * heads * ((long long)dk * dv + dk + 4);
 }
 
@@ -280,7 +278,7 @@ FE_EXPORT int fe_matrix_memory(const float* proj, long long ld, int q_off, int k
     p.raw = scratch;
     scratch = scratch ? scratch + (size_t)tokens * heads * dv : nullptr;
   }
-  const bool chunked = max_new >= SR_LONG_FROM && scratch != nullptr && chunk_takes(dk, dv, true) && memory_sums_smem(dk) <= 200 * 1024;
+  const bool chunked = max_new >= SR_LONG_FROM && scratch != nullptr && chunk_takes(dk, dv, true);
   if (chunked) p.long_from = SR_LONG_FROM;
   int rc = launch_walk(m, p, out_dtype, entries, tokens, status, stream);
   if (rc || !chunked) return rc ? rc : fe_last_error();
@@ -288,8 +286,7 @@ FE_EXPORT int fe_matrix_memory(const float* proj, long long ld, int q_off, int k
   if (chunks > 65535) return FE_ERR_TOO_LARGE;
   m.sums = scratch;
   m.marks = m.sums + (size_t)sr_slots(tokens, entries) * heads * ((size_t)dk * dv + dk);
-  const size_t smem = memory_sums_smem(dk);
-  cudaFuncSetAttribute(memory_sums_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const size_t smem = sizeof(float) * 2 * SR_LONG * 64;
   rc = fe_launch_dependent(memory_sums_kernel, dim3(heads, entries, chunks), dim3(256), smem, stream, m, p);
   if (rc) return rc;
   rc = fe_launch_dependent(memory_scan_kernel, dim3(heads, entries, (unsigned)(((long long)dk * dv + dk + 255) / 256)), dim3(256), 0, stream, m, p, status);

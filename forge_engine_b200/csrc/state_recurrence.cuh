@@ -277,24 +277,135 @@ __device__ __forceinline__ void sr_mm44(float (&acc)[4][4], const float* xt, int
   }
 }
 
-// Rows of `src` (token t at src + t * ld, `width` channels) as a transposed tile
-// dst[channel * SR_TP + t], zero past `count` tokens.
-template <typename F>
-__device__ __forceinline__ void sr_stage_transposed(float* dst, int width, int count, F value) {
-  for (int i = threadIdx.x; i < SR_LONG * width; i += blockDim.x) {
-    const int t = i / width, d = i - t * width;
-    dst[d * SR_TP + t] = t < count ? value(t, d) : 0.f;
+// Copies of 16 or 4 bytes into shared memory that complete in the background.
+__device__ __forceinline__ void sr_copy16(float* dst, const float* src) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void sr_copy4(float* dst, const float* src) {
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"((unsigned)__cvta_generic_to_shared(dst)), "l"(src) : "memory");
+}
+__device__ __forceinline__ void sr_copy_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N> __device__ __forceinline__ void sr_copy_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+
+// Rows of 32-bit numbers `ld` apart.
+struct Rows {
+  const float* base;
+  long long ld;
+  __device__ __forceinline__ const float* row(int r) const { return base + (size_t)r * ld; }
+  __device__ __forceinline__ bool wide(int width) const {
+    return (width & 3) == 0 && (ld & 3) == 0 && ((uintptr_t)base & 15) == 0;
+  }
+};
+
+// The first `width` numbers of `count` rows (tokens), times `mul`, as a transposed tile
+// dst[channel * SR_TP + t]; zero past the last row.  A thread's loads are issued four at a time
+// before any is stored; neighbouring lanes take neighbouring rows, so that the stores fall into
+// different banks.
+__device__ __forceinline__ void sr_stage_transposed(float* dst, const Rows& src, int width, int count, float mul = 1.f) {
+  const int step = blockDim.x;
+  if (src.wide(width)) {
+    const int items = SR_LONG * (width >> 2);
+    for (int i0 = threadIdx.x; i0 < items; i0 += 4 * step) {
+      float4 x[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int i = i0 + j * step, t = i & (SR_LONG - 1), d = (i / SR_LONG) * 4;
+        x[j] = (i < items && t < count) ? *reinterpret_cast<const float4*>(src.row(t) + d) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int i = i0 + j * step, t = i & (SR_LONG - 1), d = (i / SR_LONG) * 4;
+        if (i < items) {
+          float* to = dst + d * SR_TP + t;
+          to[0] = x[j].x * mul, to[SR_TP] = x[j].y * mul, to[2 * SR_TP] = x[j].z * mul, to[3 * SR_TP] = x[j].w * mul;
+        }
+      }
+    }
+    return;
+  }
+  const int items = SR_LONG * width;
+  for (int i0 = threadIdx.x; i0 < items; i0 += 4 * step) {
+    float x[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = i0 + j * step, t = i & (SR_LONG - 1), d = i / SR_LONG;
+      x[j] = (i < items && t < count) ? src.row(t)[d] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = i0 + j * step;
+      if (i < items) dst[(i / SR_LONG) * SR_TP + (i & (SR_LONG - 1))] = x[j] * mul;
+    }
   }
 }
 
+// Columns c0 .. c0 + 63 of `count` of `rows` rows of `width` numbers as a tile dst[row * 64 + column];
+// zero past the last row and the last column.
+__device__ __forceinline__ void sr_stage_columns(float* dst, const Rows& src, int rows, int count, int c0, int width) {
+  const int step = blockDim.x;
+  if (src.wide(width)) {
+    const int items = rows * 16;
+    for (int i0 = threadIdx.x; i0 < items; i0 += 4 * step) {
+      float4 x[4];
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int i = i0 + j * step, r = i >> 4, c = c0 + (i & 15) * 4;
+        x[j] = (r < count && c < width) ? *reinterpret_cast<const float4*>(src.row(r) + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int j = 0; j < 4; ++j) {
+        const int i = i0 + j * step;
+        if (i < items) reinterpret_cast<float4*>(dst)[i] = x[j];
+      }
+    }
+    return;
+  }
+  const int items = rows * 64;
+  for (int i0 = threadIdx.x; i0 < items; i0 += 4 * step) {
+    float x[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = i0 + j * step, r = i >> 6, c = c0 + (i & 63);
+      x[j] = (r < count && c < width) ? src.row(r)[c] : 0.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      const int i = i0 + j * step;
+      if (i < items) dst[i] = x[j];
+    }
+  }
+}
+
+// Inclusive running sum / maximum over 64 numbers held by a warp: element lane in `a`, element
+// 32 + lane in `b`.
+__device__ __forceinline__ void sr_running_sum(double& a, double& b) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double x = __shfl_up_sync(0xffffffffu, a, o), y = __shfl_up_sync(0xffffffffu, b, o);
+    if (lane >= o) a += x, b += y;
+  }
+  b += __shfl_sync(0xffffffffu, a, 31);
+}
+__device__ __forceinline__ void sr_running_max(double& a, double& b) {
+  const int lane = threadIdx.x & 31;
+#pragma unroll
+  for (int o = 1; o < 32; o <<= 1) {
+    const double x = __shfl_up_sync(0xffffffffu, a, o), y = __shfl_up_sync(0xffffffffu, b, o);
+    if (lane >= o) a = fmax(a, x), b = fmax(b, y);
+  }
+  b = fmax(b, __shfl_sync(0xffffffffu, a, 31));
+}
+
 // state_out: the outputs of one chunk of one head.  A mechanism M has
-//   SCORES            whether the chunk's own tokens join through scores (else M's `local_row` does)
+//   SCORES            whether the chunk's own tokens join through scores (else M's `local` rows do)
 //   out_begin(...)    per token: row term rt, column term ct (64-bit; the weight of token j in token
-//                     t's output is exp(rt[t] + ct[j])) and the factor ea[t] of the start state's
-//                     share; called by all threads, followed by a barrier
-//   query(t, d), key(t, d), other(t, c)   the chunk's queries, keys and what the scores weigh
-//   start(d, c)       the state before the chunk
-//   NORMALISER        whether rows are divided by max(|sum|, floor_t) + 1e-6 (M's `start_norm(d)`)
+//                     t's output is exp(rt[t] + ct[j])), the factor ea[t] of the start state's
+//                     share and (NORMALISER) the floor fl[t]; called by warp 0
+//   queries, keys, others, starts, locals   rows of the chunk: its queries (times query_mul()) and keys
+//                     per token, what the scores weigh, the state before the chunk per key channel,
+//                     what the chunk's own tokens give (without SCORES)
+//   NORMALISER        whether rows are divided by max(|sum|, floor_t) + 1e-6 (M's `start_norm`)
 // 256 threads: thread (rg, cg) owns rows 4 rg .. and, in pass n, columns 64 n + 4 cg ..
 template <class M, typename TO, int NP>
 __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRun p) {
@@ -311,10 +422,9 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
   float* as = qt + dk * SR_TP;                   // [SR_LONG tokens j][SR_TP tokens t] (SCORES only)
   float* tile = as + (M::SCORES ? SR_LONG * SR_TP : 0);   // keys [dk][SR_TP], then tiles of 64 columns
   const int rg = tid & 15, cg = tid >> 4, row = 4 * rg;
-  sr_stage_transposed(qt, dk, at.count, [&](int t, int d) { return m.query(p, head, at, t, d); });
-  if constexpr (M::SCORES)
-    sr_stage_transposed(tile, dk, at.count, [&](int t, int d) { return m.key(p, head, at, t, d); });
-  m.out_begin(p, head, at, rt, ct, ea, fl);
+  sr_stage_transposed(qt, m.queries(p, head, at), dk, at.count, m.query_mul());
+  if constexpr (M::SCORES) sr_stage_transposed(tile, m.keys(p, head, at), dk, at.count);
+  if (tid < 32) m.out_begin(p, head, at, rt, ct, ea, fl);
   __syncthreads();
   if constexpr (M::SCORES) {
     float a[4][4] = {};
@@ -334,9 +444,12 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
     if constexpr (M::NORMALISER) {
       // four threads a token: the sum of its weights and its query against the start normaliser
       const int t = tid >> 2, g = tid & 3;
+      const float* n0 = m.start_norm(p, head, at);
       float own = 0.f, old = 0.f;
+#pragma unroll 4
       for (int j = g; j < SR_LONG; j += 4) own += as[j * SR_TP + t];
-      for (int d = g; d < dk; d += 4) old = fmaf(qt[d * SR_TP + t], m.start_norm(p, head, at, d), old);
+#pragma unroll 4
+      for (int d = g; d < dk; d += 4) old = fmaf(qt[d * SR_TP + t], n0[d], old);
       own = sr_column_sum(fmaf(ea[t], old, own), 4);
       if (g == 0) den[t] = 1.f / (fmaxf(fabsf(own), fl[t]) + 1e-6f);
     }
@@ -349,18 +462,12 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
     float own[4][4] = {}, old[4][4] = {};
     if constexpr (M::SCORES) {
       __syncthreads();
-      for (int i = tid; i < SR_LONG * 64; i += blockDim.x) {
-        const int t = i >> 6, c = c0 + (i & 63);
-        tile[i] = (t < at.count && c < dv) ? m.other(p, head, at, t, c) : 0.f;
-      }
+      sr_stage_columns(tile, m.others(p, head, at), SR_LONG, at.count, c0, dv);
       __syncthreads();
       sr_mm44(own, as, SR_TP, tile, 64, min(at.count, row + 4), row, 4 * cg);
     }
     __syncthreads();
-    for (int i = tid; i < dk * 64; i += blockDim.x) {
-      const int d = i >> 6, c = c0 + (i & 63);
-      tile[i] = c < dv ? m.start(p, head, at, d, c) : 0.f;
-    }
+    sr_stage_columns(tile, m.starts(p, head, at), dk, dk, c0, dv);
     __syncthreads();
     sr_mm44(old, qt, SR_TP, tile, 64, dk, row, 4 * cg);
 #pragma unroll
@@ -369,7 +476,7 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
 #pragma unroll
       for (int b = 0; b < 4; ++b) {
         float x = fmaf(ea[t], old[a][b], own[a][b]);
-        if constexpr (!M::SCORES) x += (t < at.count && col + b < dv) ? m.local_row(p, head, at, t, col + b) : 0.f;
+        if constexpr (!M::SCORES) x += (t < at.count && col + b < dv) ? m.locals(p, head, at).row(t)[col + b] : 0.f;
         if constexpr (M::NORMALISER) x *= den[t];
         acc[n][a][b] = x;
         ss[a] = fmaf(x, x, ss[a]);
@@ -380,6 +487,8 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
   for (int a = 0; a < 4; ++a) part[cg][row + a] = ss[a];
   __syncthreads();
   const float* w = p.norm_w + (size_t)head * p.norm_stride;
+  const bool wide = (dv & 3) == 0 && (p.norm_stride & 3) == 0 && (p.gate_ld & 3) == 0 &&
+                    (((uintptr_t)p.norm_w | (uintptr_t)p.gate | (uintptr_t)p.out) & 15) == 0;
 #pragma unroll
   for (int a = 0; a < 4; ++a) {
     const int t = row + a;
@@ -392,10 +501,18 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
     TO* dst = (TO*)p.out + ((size_t)(at.first + t) * p.heads + head) * dv;
 #pragma unroll
     for (int n = 0; n < NP; ++n) {
+      const int c = 64 * n + 4 * cg;
+      if (wide) {
+        if (c >= dv) continue;
+        float wv[4], gv[4], y[4];
+        load4(w + c, wv), load4(g + c, gv);
 #pragma unroll
-      for (int b = 0; b < 4; ++b) {
-        const int c = 64 * n + 4 * cg + b;
-        if (c < dv) dst[c] = from_float<TO>(acc[n][a][b] * inv * w[c] * sr_gate(g[c], p.gate_act));
+        for (int b = 0; b < 4; ++b) y[b] = acc[n][a][b] * inv * wv[b] * sr_gate(gv[b], p.gate_act);
+        store4(dst + c, y);
+      } else {
+#pragma unroll
+        for (int b = 0; b < 4; ++b)
+          if (c + b < dv) dst[c + b] = from_float<TO>(acc[n][a][b] * inv * w[c + b] * sr_gate(g[c + b], p.gate_act));
       }
     }
   }

@@ -23,8 +23,14 @@
 // ---------------------------------------------------------------------------
 // y: the normalised rows, 32-bit [tokens, width], or null: then row t is residual + update + shift
 // (written back), normalised here, and every entry brings one token.
-template <typename TU, typename TO>
-__global__ void __launch_bounds__(256)
+// V: neighbouring elements a thread takes at a time.
+template <int V> __device__ __forceinline__ void ts_load(const float* p, float* v) { if constexpr (V == 4) load4(p, v); else v[0] = p[0]; }
+template <int V> __device__ __forceinline__ void ts_load(const bf16* p, float* v) { if constexpr (V == 4) load4(p, v); else v[0] = to_float(p[0]); }
+template <int V> __device__ __forceinline__ void ts_store(float* p, const float* v) { if constexpr (V == 4) store4(p, v); else p[0] = v[0]; }
+template <int V> __device__ __forceinline__ void ts_store(bf16* p, const float* v) { if constexpr (V == 4) store4(p, v); else p[0] = from_float<bf16>(v[0]); }
+
+template <typename TU, typename TO, int V>
+__global__ void __launch_bounds__(1024)
 token_shift_kernel(const float* __restrict__ y, float* __restrict__ residual, const TU* __restrict__ update,
                    const float* __restrict__ shift, long long shift_stride, const float* __restrict__ weight, float eps,
                    const float* __restrict__ mu, int mixes, float* __restrict__ state, const int* __restrict__ slots,
@@ -43,27 +49,53 @@ token_shift_kernel(const float* __restrict__ y, float* __restrict__ residual, co
   if (y == nullptr) {
     float* res = residual + (size_t)t * width;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < width; i += blockDim.x) {
-      float x = res[i];
-      if (update != nullptr) x += to_float(update[(size_t)t * width + i]);
-      if (shift != nullptr) x += shift[(size_t)t * shift_stride + i];
-      res[i] = x;
-      row[i] = x;
-      ss = fmaf(x, x, ss);
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+      float x[V], u[V];
+      ts_load<V>(res + i, x);
+      if (update != nullptr) {
+        ts_load<V>(update + (size_t)t * width + i, u);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] += u[e];
+      }
+      if (shift != nullptr) {
+        ts_load<V>(shift + (size_t)t * shift_stride + i, u);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] += u[e];
+      }
+      ts_store<V>(res + i, x);
+      ts_store<V>(row + i, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) ss = fmaf(x[e], x[e], ss);
     }
     inv = rsqrtf(block_sum(ss, scratch) / (float)width + eps);
   } else {
     mine = y + (size_t)t * width;
   }
-  for (int i = threadIdx.x; i < width; i += blockDim.x) {
-    const float h = y == nullptr ? row[i] * inv * weight[i] : mine[i];
+  for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+    float h[V], d[V], w[V];
+    ts_load<V>(mine + i, h);
     // only the block of an entry's first token touches the state: it reads it, then leaves the last row
-    const float before = t == first ? st[i] : y[(size_t)(t - 1) * width + i];
-    if (t == first) st[i] = t == last ? h : y[(size_t)last * width + i];
-    const float d = before - h;
-    for (int j = 0; j < mixes; ++j)
-      mixed[((size_t)j * n_tokens + t) * width + i] = from_float<TO>(fmaf(d, mu[(size_t)j * width + i], h));
-    if (plain != nullptr) plain[(size_t)t * width + i] = from_float<TO>(h);
+    ts_load<V>(t == first ? st + i : y + (size_t)(t - 1) * width + i, d);
+    if (y == nullptr) {
+      ts_load<V>(weight + i, w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) h[e] = h[e] * inv * w[e];
+    }
+    if (t == first) {
+      if (t != last) ts_load<V>(y + (size_t)last * width + i, w);
+      ts_store<V>(st + i, t == last ? h : w);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) d[e] -= h[e];
+#pragma unroll 5
+    for (int j = 0; j < mixes; ++j) {
+      float m[V];
+      ts_load<V>(mu + (size_t)j * width + i, m);
+#pragma unroll
+      for (int e = 0; e < V; ++e) m[e] = fmaf(d[e], m[e], h[e]);
+      ts_store<V>(mixed + ((size_t)j * n_tokens + t) * width + i, m);
+    }
+    if (plain != nullptr) ts_store<V>(plain + (size_t)t * width + i, h);
   }
 }
 
@@ -77,19 +109,30 @@ FE_EXPORT int fe_token_shift(const float* y, float* residual, const void* update
   if (smem > 200 * 1024) return FE_ERR_TOO_LARGE;
   int rc = FE_ERR_BAD_DTYPE;
   if (update == nullptr) update_dtype = FE_DTYPE_F32;
-#define SHIFT(TU, TO)                                                                                                  \
+  const bool wide = width % 4 == 0 && shift_stride % 4 == 0 &&
+                    (((uintptr_t)y | (uintptr_t)residual | (uintptr_t)update | (uintptr_t)shift | (uintptr_t)weight | (uintptr_t)mu |
+                      (uintptr_t)state | (uintptr_t)mixed | (uintptr_t)plain) & 15) == 0;
+  const int items = wide ? width / 4 : width;
+  const int threads = items >= 1024 ? 1024 : (items + 31) / 32 * 32;
+#define SHIFT_V(TU, TO, V)                                                                                             \
   do {                                                                                                                 \
     if (smem > 47 * 1024)                                                                                              \
-      cudaFuncSetAttribute(token_shift_kernel<TU, TO>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);        \
-    rc = fe_launch_dependent(token_shift_kernel<TU, TO>, dim3(n_tokens), dim3(256), smem, stream, y, residual,         \
+      cudaFuncSetAttribute(token_shift_kernel<TU, TO, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
+    rc = fe_launch_dependent(token_shift_kernel<TU, TO, V>, dim3(n_tokens), dim3(threads), smem, stream, y, residual,  \
                              (const TU*)update, shift, shift_stride, weight, eps, mu, mixes, state, slots, cu_tokens,  \
                              token_entry, (TO*)mixed, (TO*)plain, n_tokens, width);                                    \
+  } while (0)
+#define SHIFT(TU, TO)                \
+  do {                               \
+    if (wide) SHIFT_V(TU, TO, 4);    \
+    else SHIFT_V(TU, TO, 1);         \
   } while (0)
   if (update_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_F32) SHIFT(float, float);
   else if (update_dtype == FE_DTYPE_F32 && out_dtype == FE_DTYPE_BF16) SHIFT(float, bf16);
   else if (update_dtype == FE_DTYPE_BF16 && out_dtype == FE_DTYPE_F32) SHIFT(bf16, float);
   else if (update_dtype == FE_DTYPE_BF16 && out_dtype == FE_DTYPE_BF16) SHIFT(bf16, bf16);
 #undef SHIFT
+#undef SHIFT_V
   return rc ? rc : fe_last_error();
 }
 
@@ -97,35 +140,47 @@ FE_EXPORT int fe_token_shift(const float* y, float* residual, const void* update
 // wkv_decay: out[t, c] = exp(-exp(base[c] + sum_j tanh(low[t, j]) up[j, c])), all 32-bit
 // ---------------------------------------------------------------------------
 #define WD_TOKENS 8
-__global__ void __launch_bounds__(128)
+#define WD_CHANNELS 64
+// A block takes WD_TOKENS tokens and 64 channels; four groups of threads share the rank and meet
+// in shared memory in a fixed order.
+__global__ void __launch_bounds__(4 * WD_CHANNELS)
 wkv_decay_kernel(const float* __restrict__ low, const float* __restrict__ up, const float* __restrict__ base,
                  float* __restrict__ out, int n_tokens, int rank, int channels) {
   extern __shared__ __align__(16) float th[];       // [rank][WD_TOKENS]
+  __shared__ float part[4][WD_TOKENS][WD_CHANNELS];
   pdl_trigger();
   pdl_wait();
   const int t0 = blockIdx.y * WD_TOKENS, count = min(WD_TOKENS, n_tokens - t0);
   for (int i = threadIdx.x; i < rank * WD_TOKENS; i += blockDim.x) {
-    const int t = i / rank, j = i - t * rank;
-    th[j * WD_TOKENS + t] = t < count ? tanhf(low[(size_t)(t0 + t) * rank + j]) : 0.f;
+    const int j = i / WD_TOKENS, t = i - j * WD_TOKENS;
+    th[i] = t < count ? tanhf(low[(size_t)(t0 + t) * rank + j]) : 0.f;
   }
   __syncthreads();
-  const int c = blockIdx.x * blockDim.x + threadIdx.x;
-  if (c >= channels) return;
+  const int g = threadIdx.x / WD_CHANNELS, x = threadIdx.x - g * WD_CHANNELS, c = blockIdx.x * WD_CHANNELS + x;
   float acc[WD_TOKENS];
 #pragma unroll
   for (int t = 0; t < WD_TOKENS; ++t) acc[t] = 0.f;
-#pragma unroll 4
-  for (int j = 0; j < rank; ++j) {
-    const float u = up[(size_t)j * channels + c];
-    const float4 a = *reinterpret_cast<const float4*>(th + j * WD_TOKENS);
-    const float4 b = *reinterpret_cast<const float4*>(th + j * WD_TOKENS + 4);
-    acc[0] = fmaf(a.x, u, acc[0]), acc[1] = fmaf(a.y, u, acc[1]), acc[2] = fmaf(a.z, u, acc[2]), acc[3] = fmaf(a.w, u, acc[3]);
-    acc[4] = fmaf(b.x, u, acc[4]), acc[5] = fmaf(b.y, u, acc[5]), acc[6] = fmaf(b.z, u, acc[6]), acc[7] = fmaf(b.w, u, acc[7]);
+  if (c < channels) {
+#pragma unroll 8
+    for (int j = g; j < rank; j += 4) {
+      const float u = up[(size_t)j * channels + c];
+      const float4 a = *reinterpret_cast<const float4*>(th + j * WD_TOKENS);
+      const float4 b = *reinterpret_cast<const float4*>(th + j * WD_TOKENS + 4);
+      acc[0] = fmaf(a.x, u, acc[0]), acc[1] = fmaf(a.y, u, acc[1]), acc[2] = fmaf(a.z, u, acc[2]), acc[3] = fmaf(a.w, u, acc[3]);
+      acc[4] = fmaf(b.x, u, acc[4]), acc[5] = fmaf(b.y, u, acc[5]), acc[6] = fmaf(b.z, u, acc[6]), acc[7] = fmaf(b.w, u, acc[7]);
+    }
   }
+#pragma unroll
+  for (int t = 0; t < WD_TOKENS; ++t) part[g][t][x] = acc[t];
+  __syncthreads();
+  if (c >= channels) return;
   const float b0 = base[c];
 #pragma unroll
-  for (int t = 0; t < WD_TOKENS; ++t)
-    if (t < count) out[(size_t)(t0 + t) * channels + c] = expf(-expf(b0 + acc[t]));
+  for (int h = 0; h < WD_TOKENS / 4; ++h) {
+    const int t = g + 4 * h;
+    if (t < count)
+      out[(size_t)(t0 + t) * channels + c] = expf(-expf(b0 + ((part[0][t][x] + part[1][t][x]) + (part[2][t][x] + part[3][t][x]))));
+  }
 }
 
 FE_EXPORT int fe_wkv_decay(const float* low, const float* up, const float* base, float* out, int n_tokens, int rank,
@@ -135,9 +190,9 @@ FE_EXPORT int fe_wkv_decay(const float* low, const float* up, const float* base,
   const size_t smem = sizeof(float) * (size_t)rank * WD_TOKENS;
   const int blocks_y = (n_tokens + WD_TOKENS - 1) / WD_TOKENS;
   if (smem > 200 * 1024 || blocks_y > 65535) return FE_ERR_TOO_LARGE;
-  if (smem > 48 * 1024) cudaFuncSetAttribute(wkv_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const int rc = fe_launch_dependent(wkv_decay_kernel, dim3((channels + 127) / 128, blocks_y), dim3(128), smem, stream, low,
-                                     up, base, out, n_tokens, rank, channels);
+  if (smem > 38 * 1024) cudaFuncSetAttribute(wkv_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const int rc = fe_launch_dependent(wkv_decay_kernel, dim3((channels + WD_CHANNELS - 1) / WD_CHANNELS, blocks_y), dim3(4 * WD_CHANNELS),
+                                     smem, stream, low, up, base, out, n_tokens, rank, channels);
   return rc ? rc : fe_last_error();
 }
 
@@ -195,26 +250,28 @@ struct Wkv {
   }
   __device__ __forceinline__ float scale(const float*, const float*, int) const { return 1.f; }
 
-  __device__ __forceinline__ float query(const StateRun& p, int head, const ChunkAt& at, int t, int d) const {
-    return qb[((size_t)(at.first + t) * p.heads + head) * p.dk + d];
+  __device__ __forceinline__ Rows queries(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{qb + ((size_t)at.first * p.heads + head) * p.dk, (long long)p.heads * p.dk};
   }
-  __device__ __forceinline__ float start(const StateRun& p, int head, const ChunkAt& at, int d, int c) const {
-    return local[(((size_t)at.slot * p.heads + head) * p.dk + d) * p.dv + c];
+  __device__ __forceinline__ float query_mul() const { return 1.f; }
+  __device__ __forceinline__ Rows starts(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{local + ((size_t)at.slot * p.heads + head) * p.dk * p.dv, p.dv};
   }
-  __device__ __forceinline__ float local_row(const StateRun& p, int head, const ChunkAt& at, int t, int c) const {
-    return o_local[((size_t)(at.first + t) * p.heads + head) * p.dv + c];
+  __device__ __forceinline__ Rows locals(const StateRun& p, int head, const ChunkAt& at) const {
+    return Rows{o_local + ((size_t)at.first * p.heads + head) * p.dv, (long long)p.heads * p.dv};
   }
   __device__ __forceinline__ void out_begin(const StateRun&, int, const ChunkAt& at, double*, double*, float* ea, float*) const {
-    if (threadIdx.x < SR_LONG) ea[threadIdx.x] = (int)threadIdx.x < at.count ? 1.f : 0.f;
+    for (int t = threadIdx.x; t < SR_LONG; t += 32) ea[t] = t < at.count ? 1.f : 0.f;
   }
 };
 
 // One chunk from a zero state.  A thread keeps rows s * KPT .. of two columns, so that a token's
 // decays, keys and receptances are read 16 bytes at a time and serve both; rows past dk are padded
-// with zeros, and a pitch of KPT + 4 keeps a column's lanes in different banks.
+// with zeros, and a pitch of KPT + 4 keeps a column's lanes in different banks.  Tokens come in
+// stretches of SR_CHUNK, the next one on its way into the other half of the buffers meanwhile.
 #define WL_KPT 16
 #define WL_KP (WL_KPT + 4)
-__global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const StateRun p, int splits, int cols) {
+__global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const StateRun p, int splits, int cols, int wide) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
@@ -222,42 +279,65 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
   if (!sr_locate(p, &at)) return;
   const int head = blockIdx.x / splits, split = blockIdx.x - head * splits;
   const int dk = p.dk, dv = p.dv, ds = p.ds, pitch = ds * WL_KP, tid = threadIdx.x;
-  float* fs = smem;                          // [SR_CHUNK][ds][WL_KP]
-  float* rs = fs + SR_CHUNK * pitch;
-  float* ks = rs + SR_CHUNK * pitch;
-  float* vs = ks + SR_CHUNK * pitch;         // [SR_CHUNK][cols]
-  float* bonus = vs + SR_CHUNK * cols;       // [SR_CHUNK]
+  const int part = SR_CHUNK * pitch, half_size = 3 * part + SR_CHUNK * cols;
+  float* bonus = smem + 2 * half_size;       // [SR_CHUNK]
   float* bs = bonus + SR_CHUNK;              // [dk]: the product of the decays so far
   const int v = tid / ds, s = tid - v * ds, half = cols >> 1, col0 = split * cols;
+  const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
   const bool live = v < half;
   float S0[WL_KPT], S1[WL_KPT];
 #pragma unroll
   for (int i = 0; i < WL_KPT; ++i) S0[i] = S1[i] = 0.f;
-  for (int i = tid; i < 3 * SR_CHUNK * pitch; i += blockDim.x) smem[i] = 0.f;
+  for (int i = tid; i < 2 * half_size; i += blockDim.x) smem[i] = 0.f;
   for (int d = tid; d < dk; d += blockDim.x) bs[d] = 1.f;
   __syncthreads();
-  for (int c0 = 0; c0 < at.count; c0 += SR_CHUNK) {
+  const size_t head_at = (size_t)head * dk;
+  // half of the buffers: decays [SR_CHUNK][ds][WL_KP], receptances, keys, values [SR_CHUNK][cols]
+  auto fetch = [&](int c0, float* buf) {
     const int nt = min(SR_CHUNK, at.count - c0), first = at.first + c0;
-    for (int i = tid; i < nt * dk; i += blockDim.x) {
-      const int t = i / dk, d = i - t * dk;
-      const size_t src = (size_t)(first + t) * m.ld + (size_t)head * dk + d;
-      const int dst = t * pitch + (d / WL_KPT) * WL_KP + d % WL_KPT;
-      fs[dst] = m.f[src], rs[dst] = m.r[src], ks[dst] = m.k[src];
+    for (int t = warp; t < nt; t += warps) {
+      const size_t row = (size_t)(first + t) * m.ld + head_at;
+      float* dst = buf + t * pitch;
+      if (wide) {
+        for (int d = 4 * lane; d < dk; d += 128) {
+          float* to = dst + (d / WL_KPT) * WL_KP + d % WL_KPT;
+          sr_copy16(to, m.f + row + d), sr_copy16(to + part, m.r + row + d), sr_copy16(to + 2 * part, m.k + row + d);
+        }
+      } else {
+        for (int d = lane; d < dk; d += 32) {
+          float* to = dst + (d / WL_KPT) * WL_KP + d % WL_KPT;
+          sr_copy4(to, m.f + row + d), sr_copy4(to + part, m.r + row + d), sr_copy4(to + 2 * part, m.k + row + d);
+        }
+      }
+      const float* value = p.v + (size_t)(first + t) * p.v_ld + (size_t)head * dv + col0;
+      for (int c = lane; c < cols && col0 + c < dv; c += 32) sr_copy4(buf + 3 * part + t * cols + c, value + c);
     }
-    for (int i = tid; i < nt * cols; i += blockDim.x) {
-      const int t = i / cols, c = i - t * cols;
-      vs[i] = col0 + c < dv ? p.v[(size_t)(first + t) * p.v_ld + (size_t)head * dv + col0 + c] : 0.f;
-    }
-    for (int t = tid >> 5; t < nt; t += blockDim.x >> 5) {
-      const float b = m.bonus(p, head, first + t);
-      if ((tid & 31) == 0) bonus[t] = b;
-    }
+    sr_copy_commit();
+  };
+  fetch(0, smem);
+  int turn = 0;
+  for (int c0 = 0; c0 < at.count; c0 += SR_CHUNK, turn ^= 1) {
+    const int nt = min(SR_CHUNK, at.count - c0), first = at.first + c0;
+    float* buf = smem + turn * half_size;
+    const float *fs = buf, *rs = buf + part, *ks = rs + part, *vs = ks + part;
+    sr_copy_wait<0>();
     __syncthreads();
+    if (c0 + SR_CHUNK < at.count) fetch(c0 + SR_CHUNK, smem + (turn ^ 1) * half_size);
+    for (int t = warp; t < nt; t += warps) {
+      float b = 0.f;
+      for (int d = lane; d < dk; d += 32) {
+        const int i = t * pitch + (d / WL_KPT) * WL_KP + d % WL_KPT;
+        b = fmaf(rs[i] * m.u[head_at + d], ks[i], b);
+      }
+      b = warp_sum(b);
+      if (lane == 0) bonus[t] = b;
+    }
     if (split == 0) {
       for (int d = tid; d < dk; d += blockDim.x) {
         const int from = (d / WL_KPT) * WL_KP + d % WL_KPT;
         float b = bs[d];
         float* dst = m.qb + ((size_t)first * p.heads + head) * dk + d;
+#pragma unroll 4
         for (int t = 0; t < nt; ++t) {
           dst[(size_t)t * p.heads * dk] = rs[t * pitch + from] * b;
           b *= fs[t * pitch + from];
@@ -265,6 +345,7 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
         bs[d] = b;
       }
     }
+    __syncthreads();
     for (int t = 0; t < nt; ++t) {
       const float v0 = live ? vs[t * cols + v] : 0.f, v1 = live ? vs[t * cols + half + v] : 0.f;
       const float4* f4 = reinterpret_cast<const float4*>(fs + t * pitch + s * WL_KP);
@@ -290,7 +371,6 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
         if (col0 + half + v < dv) dst[half + v] = fmaf(bonus[t], v1, a1);
       }
     }
-    __syncthreads();
   }
   const size_t cell = (size_t)at.slot * p.heads + head;
 #pragma unroll
@@ -394,9 +474,10 @@ FE_EXPORT int fe_wkv(const float* r, const float* k, const float* v, const float
   m.decay = m.local + (size_t)sr_slots(tokens, entries) * heads * dk * dv;
   p.ds = ds;
   const int threads = (cols / 2 * ds + 31) / 32 * 32;
-  const size_t smem = sizeof(float) * ((size_t)SR_CHUNK * (3 * ds * WL_KP + cols + 1) + dk);
+  const size_t smem = sizeof(float) * ((size_t)SR_CHUNK * (2 * (3 * ds * WL_KP + cols) + 1) + dk);
+  const int wide = dk % 4 == 0 && ld % 4 == 0 && (((uintptr_t)r | (uintptr_t)k | (uintptr_t)decay) & 15) == 0;
   if (smem > 48 * 1024) cudaFuncSetAttribute(wkv_local_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  rc = fe_launch_dependent(wkv_local_kernel, dim3(heads * splits, entries, chunks), dim3(threads), smem, stream, m, p, splits, cols);
+  rc = fe_launch_dependent(wkv_local_kernel, dim3(heads * splits, entries, chunks), dim3(threads), smem, stream, m, p, splits, cols, wide);
   if (rc) return rc;
   rc = fe_launch_dependent(wkv_scan_kernel, dim3(heads, entries, (dk * dv + 255) / 256), dim3(256), 0, stream, m, p, status);
   if (rc) return rc;
