@@ -224,18 +224,23 @@ struct Delta {
 };
 
 // W and U of one chunk of one head: the triangular system solved for the columns of beta e^c k
-// and beta v, a thread per column with the column in registers.
-__global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const StateRun p) {
+// and beta v, sixteen rows at a time.  A block of rows first loses what the rows before it give (a
+// small product), then a thread per column solves the 16 x 16 triangle in registers and stores the
+// result, also for the blocks below.
+#define DS_THREADS 256
+__global__ void __launch_bounds__(DS_THREADS) delta_solve_kernel(const Delta m, const StateRun p) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
   ChunkAt at;
   if (!sr_locate(p, &at)) return;
   const int head = blockIdx.x, dk = p.dk, dv = p.dv, tid = threadIdx.x;
+  const int v0 = (dk + 3) & ~3, ldx = v0 + ((dv + 3) & ~3);      // columns of k, then of v
   __shared__ double c[SR_LONG];
   __shared__ float bt[SR_LONG], be[SR_LONG];
-  float* L = smem;                           // [SR_LONG rows t][SR_LONG]
-  float* kt = L + SR_LONG * SR_LONG;         // [dk][SR_TP]
+  float* lt = smem;                          // [SR_LONG columns j][SR_TP rows t]: L transposed
+  float* X = lt + SR_LONG * SR_TP;           // [SR_LONG][ldx]
+  float* kt = X + SR_LONG * ldx;             // [dk][SR_TP]
   if (tid < 32) {
     double sums[2];
     m.chunk_sums(p, head, at, sums);
@@ -252,55 +257,81 @@ __global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const S
     }
     if (tid == 0) decays[SR_LONG] = expf((float)end);
   }
-  sr_stage_transposed(kt, m.keys(p, head, at), dk, at.count);
+  const Rows keys = m.keys(p, head, at), values{p.v + (size_t)at.first * p.v_ld + (size_t)head * dv, p.v_ld};
+  sr_stage_transposed(kt, keys, dk, at.count);
   __syncthreads();
-  for (int item = tid; item < 256; item += blockDim.x) {
-    const int row = 4 * (item & 15), col = 4 * (item >> 4);
+  // the right sides: rows of beta e^c k and beta v, zero past the last token and between the two
+  const int warp = tid >> 5, lane = tid & 31;
+  for (int t = warp; t < SR_LONG; t += DS_THREADS / 32) {
+    const bool has = t < at.count;
+    const float a = be[t], b = bt[t];
+    float* x = X + t * ldx;
+    for (int d = lane; d < v0; d += 32) x[d] = d < dk ? a * kt[d * SR_TP + t] : 0.f;
+    for (int d = lane; d < ldx - v0; d += 32) x[v0 + d] = has && d < dv ? b * values.row(t)[d] : 0.f;
+  }
+  {
+    const int row = 4 * (tid & 15), col = 4 * (tid >> 4);
     float a[4][4] = {};
     if (col <= row + 3) sr_mm44(a, kt, SR_TP, kt, SR_TP, dk, row, col);
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-      const int t = row + e;
+    for (int b = 0; b < 4; ++b) {
       float l[4];
 #pragma unroll
-      for (int b = 0; b < 4; ++b) l[b] = col + b < t ? a[e][b] * bt[t] * expf((float)(c[t] - c[col + b])) : 0.f;
-      store4(L + t * SR_LONG + col, l);
+      for (int e = 0; e < 4; ++e) {
+        const int t = row + e;
+        l[e] = col + b < t ? a[e][b] * bt[t] * expf((float)(c[t] - c[col + b])) : 0.f;
+      }
+      store4(lt + (col + b) * SR_TP + row, l);
     }
   }
-  __syncthreads();
   const size_t cell = m.cell(p, at, head);
-  for (int i = tid; i < dk + dv; i += blockDim.x) {
-    float x[SR_LONG];
-    if (i < dk) {
+  for (int r0 = 0; r0 < SR_LONG; r0 += 16) {
+    __syncthreads();
+    if (r0 > 0) {
+      const int row = r0 + 4 * (tid & 3);
+      for (int col = 2 * (tid >> 2); col < ldx; col += DS_THREADS / 2) {
+        float acc[4][2] = {};
+#pragma unroll 8
+        for (int j = 0; j < r0; ++j) {
+          const float4 l = *reinterpret_cast<const float4*>(lt + j * SR_TP + row);
+          const float2 x = *reinterpret_cast<const float2*>(X + j * ldx + col);
+          acc[0][0] = fmaf(l.x, x.x, acc[0][0]), acc[0][1] = fmaf(l.x, x.y, acc[0][1]);
+          acc[1][0] = fmaf(l.y, x.x, acc[1][0]), acc[1][1] = fmaf(l.y, x.y, acc[1][1]);
+          acc[2][0] = fmaf(l.z, x.x, acc[2][0]), acc[2][1] = fmaf(l.z, x.y, acc[2][1]);
+          acc[3][0] = fmaf(l.w, x.x, acc[3][0]), acc[3][1] = fmaf(l.w, x.y, acc[3][1]);
+        }
 #pragma unroll
-      for (int t = 0; t < SR_LONG; ++t) x[t] = be[t] * kt[i * SR_TP + t];
-    } else {
-      const float* v = p.v + (size_t)at.first * p.v_ld + (size_t)head * dv + (i - dk);
-#pragma unroll
-      for (int t = 0; t < SR_LONG; ++t) x[t] = t < at.count ? bt[t] * v[(size_t)t * p.v_ld] : 0.f;
-    }
-#pragma unroll
-    for (int t = 1; t < SR_LONG; ++t) {
-      const float4* l4 = reinterpret_cast<const float4*>(L + t * SR_LONG);
-      float s0 = 0.f, s1 = 0.f, s2 = 0.f, s3 = 0.f;
-#pragma unroll
-      for (int j = 0; j < t; j += 4) {
-        const float4 l = l4[j >> 2];           // entries at and past the diagonal are zero
-        s0 = fmaf(l.x, x[j], s0);
-        s1 = fmaf(l.y, x[j + 1], s1);
-        s2 = fmaf(l.z, x[j + 2], s2);
-        s3 = fmaf(l.w, x[j + 3], s3);
+        for (int e = 0; e < 4; ++e) {
+          float2* x2 = reinterpret_cast<float2*>(X + (row + e) * ldx + col);
+          *x2 = make_float2(x2->x - acc[e][0], x2->y - acc[e][1]);
+        }
       }
-      x[t] -= (s0 + s1) + (s2 + s3);
+      __syncthreads();
     }
-    if (i < dk) {
-      float* dst = m.w + (cell * dk + i) * SR_LONG;
+    for (int i = tid; i < ldx; i += DS_THREADS) {
+      float x[16];
 #pragma unroll
-      for (int t = 0; t < SR_LONG; t += 4) store4(dst + t, x + t);
-    } else {
-      float* dst = m.u + cell * SR_LONG * dv + (i - dk);
+      for (int t = 0; t < 16; ++t) x[t] = X[(r0 + t) * ldx + i];
 #pragma unroll
-      for (int t = 0; t < SR_LONG; ++t) dst[(size_t)t * dv] = x[t];
+      for (int j = 0; j < 15; ++j) {
+        float l[16];
+#pragma unroll
+        for (int t = 0; t < 16; t += 4)
+          if (t + 3 > j) load4(lt + (r0 + j) * SR_TP + r0 + t, l + t);
+#pragma unroll
+        for (int t = j + 1; t < 16; ++t) x[t] = fmaf(-l[t], x[j], x[t]);
+      }
+#pragma unroll
+      for (int t = 0; t < 16; ++t) X[(r0 + t) * ldx + i] = x[t];
+      if (i < dk) {
+        float* dst = m.w + (cell * dk + i) * SR_LONG + r0;
+#pragma unroll
+        for (int t = 0; t < 16; t += 4) store4(dst + t, x + t);
+      } else if (i >= v0 && i - v0 < dv) {
+        float* dst = m.u + (cell * SR_LONG + r0) * dv + (i - v0);
+#pragma unroll
+        for (int t = 0; t < 16; ++t) dst[(size_t)t * dv] = x[t];
+      }
     }
   }
 }
@@ -308,7 +339,8 @@ __global__ void __launch_bounds__(128) delta_solve_kernel(const Delta m, const S
 // The chain over an entry's chunks for one head and COLS value columns: u = U - W S, then
 // S <- e^(c_end) S + sum_j k_j (e^(c_end - c_j) u_j)^T.  The state's columns stay in shared memory;
 // the next chunk's W and keys are on their way while a chunk is worked on.  Thread (rg, cg) of
-// 16 x COLS / 2 owns four rows and two columns of a product.
+// 16 x COLS / 2 owns four rows and two columns of a product; two such groups of threads take half of
+// a product's depth each, the second one's share is added by (W S) or after (the state) the first's.
 template <int COLS>
 __device__ __forceinline__ void dc_mm42(float (&acc)[4][2], const float* xt, int ldx, const float* y, int depth, int row, int col) {
 #pragma unroll 8
@@ -323,7 +355,7 @@ __device__ __forceinline__ void dc_mm42(float (&acc)[4][2], const float* xt, int
 }
 
 template <int COLS>
-__global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, const StateRun p, int* status) {
+__global__ void __launch_bounds__(16 * COLS) delta_chain_kernel(const Delta m, const StateRun p, int* status) {
   extern __shared__ __align__(16) float smem[];
   pdl_trigger();
   pdl_wait();
@@ -339,8 +371,11 @@ __global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, co
   const int cols = min(COLS, dv - col0), half = dk * SR_LONG + SR_LONG * kp;
   float* S = smem;                           // [kp][COLS]
   float* us = S + kp * COLS;                 // [SR_LONG][COLS], weighted
-  float* buffers = us + SR_LONG * COLS;      // 2 x (W transposed [dk][SR_LONG], keys [SR_LONG][kp])
-  const int row = 4 * (tid & 15), col = 2 * (tid >> 4);
+  float* share = us + SR_LONG * COLS;        // [SR_LONG][COLS]: the second group's part of W S
+  float* buffers = share + SR_LONG * COLS;   // 2 x (W transposed [dk][SR_LONG], keys [SR_LONG][kp])
+  const int group = tid / (8 * COLS), mine = tid - group * 8 * COLS;
+  const int row = 4 * (mine & 15), col = 2 * (mine >> 4);
+  const int d_from = group == 0 ? 0 : dk / 2, d_count = group == 0 ? dk / 2 : dk - dk / 2;
   float* st = p.state + ((size_t)slot * p.heads + head) * dk * dv + col0;
   for (int i = tid; i < kp * COLS; i += blockDim.x) {
     const int d = i / COLS, c = i - d * COLS;
@@ -381,22 +416,17 @@ __global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, co
     for (int e = 0; e < 4; ++e) {
       w[e] = decays[row + e];
 #pragma unroll
-      for (int b = 0; b < 2; ++b) x[e][b] = col + b < cols ? u[(size_t)e * dv + b] : 0.f;
+      for (int b = 0; b < 2; ++b) x[e][b] = group == 0 && col + b < cols ? u[(size_t)e * dv + b] : 0.f;
     }
     const float keep = decays[SR_LONG];
     sr_copy_wait<0>();
     __syncthreads();
     if (chunk + 1 < chunks) fetch(chunk + 1, buffers + ((chunk + 1) & 1) * half);
     float a[4][2] = {};
-    dc_mm42<COLS>(a, buf, SR_LONG, S, dk, row, col);
+    dc_mm42<COLS>(a, buf + d_from * SR_LONG, SR_LONG, S + d_from * COLS, d_count, row, col);
+    if (group == 1) {
 #pragma unroll
-    for (int e = 0; e < 4; ++e) {
-#pragma unroll
-      for (int b = 0; b < 2; ++b) {
-        x[e][b] -= a[e][b];
-        if (col + b < cols) u[(size_t)e * dv + b] = x[e][b];
-      }
-      *reinterpret_cast<float2*>(us + (row + e) * COLS + col) = make_float2(x[e][0] * w[e], x[e][1] * w[e]);
+      for (int e = 0; e < 4; ++e) *reinterpret_cast<float2*>(share + (row + e) * COLS + col) = make_float2(a[e][0], a[e][1]);
     }
     // the state before the chunk, for state_out
     float* dst = m.before + cell * dk * dv + col0;
@@ -405,15 +435,40 @@ __global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, co
       if (c < cols) dst[(size_t)d * dv + c] = S[i];
     }
     __syncthreads();
-    const float* ks = buf + dk * SR_LONG;
-    for (int d0 = 0; d0 < kp; d0 += 64) {
-      float b[4][2] = {};
-      dc_mm42<COLS>(b, ks + d0, kp, us, SR_LONG, row, col);
+    if (group == 0) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) {
-        float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * COLS + col);
-        const float2 old = *s2;
-        *s2 = make_float2(fmaf(keep, old.x, b[e][0]), fmaf(keep, old.y, b[e][1]));
+        const float2 more = *reinterpret_cast<const float2*>(share + (row + e) * COLS + col);
+        x[e][0] -= a[e][0] + more.x;
+        x[e][1] -= a[e][1] + more.y;
+        *reinterpret_cast<float2*>(us + (row + e) * COLS + col) = make_float2(x[e][0] * w[e], x[e][1] * w[e]);
+#pragma unroll
+        for (int b = 0; b < 2; ++b)
+          if (col + b < cols) u[(size_t)e * dv + b] = x[e][b];
+      }
+    }
+    __syncthreads();
+    const float* ks = buf + dk * SR_LONG;
+    const int t_from = group * (SR_LONG / 2);
+    for (int d0 = 0; d0 < kp; d0 += 64) {
+      float b[4][2] = {};
+      dc_mm42<COLS>(b, ks + t_from * kp + d0, kp, us + t_from * COLS, SR_LONG / 2, row, col);
+      if (group == 0) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * COLS + col);
+          const float2 old = *s2;
+          *s2 = make_float2(fmaf(keep, old.x, b[e][0]), fmaf(keep, old.y, b[e][1]));
+        }
+      }
+      __syncthreads();
+      if (group == 1) {
+#pragma unroll
+        for (int e = 0; e < 4; ++e) {
+          float2* s2 = reinterpret_cast<float2*>(S + (d0 + row + e) * COLS + col);
+          const float2 old = *s2;
+          *s2 = make_float2(old.x + b[e][0], old.y + b[e][1]);
+        }
       }
     }
   }
@@ -424,15 +479,18 @@ __global__ void __launch_bounds__(8 * COLS) delta_chain_kernel(const Delta m, co
   }
 }
 
-static size_t delta_solve_smem(int dk) { return sizeof(float) * ((size_t)SR_LONG * SR_LONG + (size_t)dk * SR_TP); }
+static size_t delta_solve_smem(int dk, int dv) {
+  const size_t ldx = (size_t)((dk + 3) / 4 * 4) + (dv + 3) / 4 * 4;
+  return sizeof(float) * ((size_t)SR_LONG * SR_TP + SR_LONG * ldx + (size_t)dk * SR_TP);
+}
 // Value columns of a block of delta_chain: few where the heads are small, so that there are more blocks.
 static int delta_chain_cols(int dv) { return dv <= 64 ? 16 : 32; }
 static size_t delta_chain_smem(int dk, int cols) {
   const size_t kp = (size_t)(dk + 63) / 64 * 64;
-  return sizeof(float) * (kp * cols + (size_t)SR_LONG * cols + 2 * ((size_t)dk * SR_LONG + SR_LONG * kp));
+  return sizeof(float) * (kp * cols + (size_t)2 * SR_LONG * cols + 2 * ((size_t)dk * SR_LONG + SR_LONG * kp));
 }
 static bool delta_chunk_takes(int dk, int dv) {
-  return chunk_takes(dk, dv, true) && delta_solve_smem(dk) <= 200 * 1024 && delta_chain_smem(dk, delta_chain_cols(dv)) <= 200 * 1024;
+  return chunk_takes(dk, dv, true) && delta_solve_smem(dk, dv) <= 200 * 1024 && delta_chain_smem(dk, delta_chain_cols(dv)) <= 200 * 1024;
 }
 
 FE_EXPORT long long fe_delta_rule_scratch(int tokens, int entries, int heads, int dk, int dv, int max_new) {
@@ -464,19 +522,19 @@ FE_EXPORT int fe_delta_rule(const float* qkv, long long ld, const float* gates, 
   m.u = m.w + cells * dk * SR_LONG;
   m.decays = m.u + cells * SR_LONG * dv;
   m.before = m.decays + cells * (SR_LONG + 4);
-  size_t smem = delta_solve_smem(dk);
+  size_t smem = delta_solve_smem(dk, dv);
   cudaFuncSetAttribute(delta_solve_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  rc = fe_launch_dependent(delta_solve_kernel, dim3(heads, entries, chunks), dim3(128), smem, stream, m, p);
+  rc = fe_launch_dependent(delta_solve_kernel, dim3(heads, entries, chunks), dim3(DS_THREADS), smem, stream, m, p);
   if (rc) return rc;
   const int cols = delta_chain_cols(dv);
   smem = delta_chain_smem(dk, cols);
   const dim3 chain(heads, entries, (dv + cols - 1) / cols);
   if (cols == 16) {
     cudaFuncSetAttribute(delta_chain_kernel<16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    rc = fe_launch_dependent(delta_chain_kernel<16>, chain, dim3(128), smem, stream, m, p, status);
+    rc = fe_launch_dependent(delta_chain_kernel<16>, chain, dim3(256), smem, stream, m, p, status);
   } else {
     cudaFuncSetAttribute(delta_chain_kernel<32>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-    rc = fe_launch_dependent(delta_chain_kernel<32>, chain, dim3(256), smem, stream, m, p, status);
+    rc = fe_launch_dependent(delta_chain_kernel<32>, chain, dim3(512), smem, stream, m, p, status);
   }
   if (rc) return rc;
   rc = launch_out(m, p, out_dtype, entries, chunks, stream);

@@ -139,60 +139,77 @@ FE_EXPORT int fe_token_shift(const float* y, float* residual, const void* update
 // ---------------------------------------------------------------------------
 // wkv_decay: out[t, c] = exp(-exp(base[c] + sum_j tanh(low[t, j]) up[j, c])), all 32-bit
 // ---------------------------------------------------------------------------
-#define WD_TOKENS 8
-#define WD_CHANNELS 64
-// A block takes WD_TOKENS tokens and 64 channels; four groups of threads share the rank and meet
-// in shared memory in a fixed order.
-__global__ void __launch_bounds__(4 * WD_CHANNELS)
+// A block takes TOKENS tokens and 256 / SPLIT channels; SPLIT groups of threads share the rank and
+// meet in shared memory in a fixed order.
+template <int TOKENS, int SPLIT>
+__global__ void __launch_bounds__(256)
 wkv_decay_kernel(const float* __restrict__ low, const float* __restrict__ up, const float* __restrict__ base,
                  float* __restrict__ out, int n_tokens, int rank, int channels) {
-  extern __shared__ __align__(16) float th[];       // [rank][WD_TOKENS]
-  __shared__ float part[4][WD_TOKENS][WD_CHANNELS];
+  constexpr int CHANNELS = 256 / SPLIT;
+  extern __shared__ __align__(16) float th[];       // [rank][TOKENS], then the groups' sums
   pdl_trigger();
   pdl_wait();
-  const int t0 = blockIdx.y * WD_TOKENS, count = min(WD_TOKENS, n_tokens - t0);
-  for (int i = threadIdx.x; i < rank * WD_TOKENS; i += blockDim.x) {
-    const int j = i / WD_TOKENS, t = i - j * WD_TOKENS;
+  const int t0 = blockIdx.y * TOKENS, count = min(TOKENS, n_tokens - t0);
+  for (int i = threadIdx.x; i < rank * TOKENS; i += blockDim.x) {
+    const int j = i / TOKENS, t = i - j * TOKENS;
     th[i] = t < count ? tanhf(low[(size_t)(t0 + t) * rank + j]) : 0.f;
   }
   __syncthreads();
-  const int g = threadIdx.x / WD_CHANNELS, x = threadIdx.x - g * WD_CHANNELS, c = blockIdx.x * WD_CHANNELS + x;
-  float acc[WD_TOKENS];
+  const int g = threadIdx.x / CHANNELS, x = threadIdx.x - g * CHANNELS, c = blockIdx.x * CHANNELS + x;
+  float acc[TOKENS];
 #pragma unroll
-  for (int t = 0; t < WD_TOKENS; ++t) acc[t] = 0.f;
+  for (int t = 0; t < TOKENS; ++t) acc[t] = 0.f;
   if (c < channels) {
 #pragma unroll 8
-    for (int j = g; j < rank; j += 4) {
+    for (int j = g; j < rank; j += SPLIT) {
       const float u = up[(size_t)j * channels + c];
-      const float4 a = *reinterpret_cast<const float4*>(th + j * WD_TOKENS);
-      const float4 b = *reinterpret_cast<const float4*>(th + j * WD_TOKENS + 4);
-      acc[0] = fmaf(a.x, u, acc[0]), acc[1] = fmaf(a.y, u, acc[1]), acc[2] = fmaf(a.z, u, acc[2]), acc[3] = fmaf(a.w, u, acc[3]);
-      acc[4] = fmaf(b.x, u, acc[4]), acc[5] = fmaf(b.y, u, acc[5]), acc[6] = fmaf(b.z, u, acc[6]), acc[7] = fmaf(b.w, u, acc[7]);
+#pragma unroll
+      for (int t = 0; t < TOKENS; t += 4) {
+        const float4 a = *reinterpret_cast<const float4*>(th + j * TOKENS + t);
+        acc[t] = fmaf(a.x, u, acc[t]), acc[t + 1] = fmaf(a.y, u, acc[t + 1]);
+        acc[t + 2] = fmaf(a.z, u, acc[t + 2]), acc[t + 3] = fmaf(a.w, u, acc[t + 3]);
+      }
     }
   }
+  const float b0 = c < channels ? base[c] : 0.f;
+  if constexpr (SPLIT == 1) {
+    if (c < channels)
 #pragma unroll
-  for (int t = 0; t < WD_TOKENS; ++t) part[g][t][x] = acc[t];
-  __syncthreads();
-  if (c >= channels) return;
-  const float b0 = base[c];
+      for (int t = 0; t < TOKENS; ++t)
+        if (t < count) out[(size_t)(t0 + t) * channels + c] = expf(-expf(b0 + acc[t]));
+  } else {
+    float* part = th + rank * TOKENS;               // [SPLIT][TOKENS][CHANNELS]
 #pragma unroll
-  for (int h = 0; h < WD_TOKENS / 4; ++h) {
-    const int t = g + 4 * h;
-    if (t < count)
-      out[(size_t)(t0 + t) * channels + c] = expf(-expf(b0 + ((part[0][t][x] + part[1][t][x]) + (part[2][t][x] + part[3][t][x]))));
+    for (int t = 0; t < TOKENS; ++t) part[(g * TOKENS + t) * CHANNELS + x] = acc[t];
+    __syncthreads();
+    if (c >= channels) return;
+    for (int t = g; t < count; t += SPLIT) {
+      float sum = 0.f;
+#pragma unroll
+      for (int k = 0; k < SPLIT; ++k) sum += part[(k * TOKENS + t) * CHANNELS + x];
+      out[(size_t)(t0 + t) * channels + c] = expf(-expf(b0 + sum));
+    }
   }
+}
+
+template <int TOKENS, int SPLIT>
+static int launch_decay(const float* low, const float* up, const float* base, float* out, int n_tokens, int rank, int channels,
+                        cudaStream_t stream) {
+  const size_t smem = sizeof(float) * TOKENS * ((size_t)rank + (SPLIT > 1 ? 256 : 0));
+  const int channels_a_block = 256 / SPLIT, blocks_y = (n_tokens + TOKENS - 1) / TOKENS;
+  if (smem > 200 * 1024 || blocks_y > 65535) return FE_ERR_TOO_LARGE;
+  if (smem > 48 * 1024)
+    cudaFuncSetAttribute(wkv_decay_kernel<TOKENS, SPLIT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  return fe_launch_dependent(wkv_decay_kernel<TOKENS, SPLIT>, dim3((channels + channels_a_block - 1) / channels_a_block, blocks_y),
+                             dim3(256), smem, stream, low, up, base, out, n_tokens, rank, channels);
 }
 
 FE_EXPORT int fe_wkv_decay(const float* low, const float* up, const float* base, float* out, int n_tokens, int rank,
                            int channels, cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (rank < 1 || channels < 1) return FE_ERR_BAD_SHAPE;
-  const size_t smem = sizeof(float) * (size_t)rank * WD_TOKENS;
-  const int blocks_y = (n_tokens + WD_TOKENS - 1) / WD_TOKENS;
-  if (smem > 200 * 1024 || blocks_y > 65535) return FE_ERR_TOO_LARGE;
-  if (smem > 38 * 1024) cudaFuncSetAttribute(wkv_decay_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const int rc = fe_launch_dependent(wkv_decay_kernel, dim3((channels + WD_CHANNELS - 1) / WD_CHANNELS, blocks_y), dim3(4 * WD_CHANNELS),
-                                     smem, stream, low, up, base, out, n_tokens, rank, channels);
+  const int rc = n_tokens > 256 && rank <= 1024 ? launch_decay<32, 1>(low, up, base, out, n_tokens, rank, channels, stream)
+                                                : launch_decay<8, 8>(low, up, base, out, n_tokens, rank, channels, stream);
   return rc ? rc : fe_last_error();
 }
 
@@ -285,9 +302,9 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
   const int v = tid / ds, s = tid - v * ds, half = cols >> 1, col0 = split * cols;
   const int lane = tid & 31, warp = tid >> 5, warps = blockDim.x >> 5;
   const bool live = v < half;
-  float S0[WL_KPT], S1[WL_KPT];
+  uint64_t S0[WL_KPT / 2], S1[WL_KPT / 2];      // neighbouring rows in pairs
 #pragma unroll
-  for (int i = 0; i < WL_KPT; ++i) S0[i] = S1[i] = 0.f;
+  for (int i = 0; i < WL_KPT / 2; ++i) S0[i] = S1[i] = 0;
   for (int i = tid; i < 2 * half_size; i += blockDim.x) smem[i] = 0.f;
   for (int d = tid; d < dk; d += blockDim.x) bs[d] = 1.f;
   __syncthreads();
@@ -348,23 +365,25 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
     __syncthreads();
     for (int t = 0; t < nt; ++t) {
       const float v0 = live ? vs[t * cols + v] : 0.f, v1 = live ? vs[t * cols + half + v] : 0.f;
-      const float4* f4 = reinterpret_cast<const float4*>(fs + t * pitch + s * WL_KP);
-      const float4* r4 = reinterpret_cast<const float4*>(rs + t * pitch + s * WL_KP);
-      const float4* k4 = reinterpret_cast<const float4*>(ks + t * pitch + s * WL_KP);
-      float a0 = 0.f, a1 = 0.f;
+      const ulonglong2* f2 = reinterpret_cast<const ulonglong2*>(fs + t * pitch + s * WL_KP);
+      const ulonglong2* r2 = reinterpret_cast<const ulonglong2*>(rs + t * pitch + s * WL_KP);
+      const ulonglong2* k2 = reinterpret_cast<const ulonglong2*>(ks + t * pitch + s * WL_KP);
+      const uint64_t vv0 = sr_pair(v0, v0), vv1 = sr_pair(v1, v1);
+      uint64_t acc0 = 0, acc1 = 0;
 #pragma unroll
       for (int i = 0; i < WL_KPT / 4; ++i) {
-        const float4 f = f4[i], r = r4[i], k = k4[i];
-        const float ff[4] = {f.x, f.y, f.z, f.w}, rr[4] = {r.x, r.y, r.z, r.w}, kk[4] = {k.x, k.y, k.z, k.w};
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          a0 = fmaf(S0[4 * i + e], rr[e], a0);
-          a1 = fmaf(S1[4 * i + e], rr[e], a1);
-          S0[4 * i + e] = fmaf(ff[e], S0[4 * i + e], kk[e] * v0);
-          S1[4 * i + e] = fmaf(ff[e], S1[4 * i + e], kk[e] * v1);
-        }
+        const ulonglong2 f = f2[i], r = r2[i], k = k2[i];
+        acc0 = sr_fma2(S0[2 * i], r.x, acc0);
+        acc1 = sr_fma2(S1[2 * i], r.x, acc1);
+        S0[2 * i] = sr_fma2(f.x, S0[2 * i], sr_mul2(k.x, vv0));
+        S1[2 * i] = sr_fma2(f.x, S1[2 * i], sr_mul2(k.x, vv1));
+        acc0 = sr_fma2(S0[2 * i + 1], r.y, acc0);
+        acc1 = sr_fma2(S1[2 * i + 1], r.y, acc1);
+        S0[2 * i + 1] = sr_fma2(f.y, S0[2 * i + 1], sr_mul2(k.y, vv0));
+        S1[2 * i + 1] = sr_fma2(f.y, S1[2 * i + 1], sr_mul2(k.y, vv1));
       }
-      a0 = sr_column_sum(a0, ds), a1 = sr_column_sum(a1, ds);
+      const float2 sum0 = sr_unpair(acc0), sum1 = sr_unpair(acc1);
+      const float a0 = sr_column_sum(sum0.x + sum0.y, ds), a1 = sr_column_sum(sum1.x + sum1.y, ds);
       if (live && s == 0) {
         float* dst = m.o_local + ((size_t)(first + t) * p.heads + head) * dv + col0;
         if (col0 + v < dv) dst[v] = fmaf(bonus[t], v0, a0);
@@ -378,8 +397,9 @@ __global__ void __launch_bounds__(512) wkv_local_kernel(const Wkv m, const State
     const int d = s * WL_KPT + i;
     if (!live || d >= dk) continue;
     float* dst = m.local + (cell * dk + d) * dv + col0;
-    if (col0 + v < dv) dst[v] = S0[i];
-    if (col0 + half + v < dv) dst[half + v] = S1[i];
+    const float2 x0 = sr_unpair(S0[i / 2]), x1 = sr_unpair(S1[i / 2]);
+    if (col0 + v < dv) dst[v] = i & 1 ? x0.y : x0.x;
+    if (col0 + half + v < dv) dst[half + v] = i & 1 ? x1.y : x1.x;
   }
   if (split == 0)
     for (int d = tid; d < dk; d += blockDim.x) m.decay[cell * dk + d] = bs[d];
