@@ -42,26 +42,43 @@ struct DeltaPrepare {
 
 // One token's channels of one row - a q, k or v head - by a warp: convolution from `input(j)` (the
 // inputs j tokens back), silu, and for q and k the unit vector.  `buf` is the warp's own; a lane reads
-// back only what it wrote.
-template <typename F>
+// back only what it wrote.  V: neighbouring channels a lane takes at a time.
+template <int V> __device__ __forceinline__ void dp_load(const float* p, float* v) { if constexpr (V == 4) load4(p, v); else v[0] = p[0]; }
+template <int V> __device__ __forceinline__ void dp_store(float* p, const float* v) { if constexpr (V == 4) store4(p, v); else p[0] = v[0]; }
+
+template <int V, typename F>
 __device__ __forceinline__ void delta_prepare_row(const DeltaPrepare& p, int t, int r, float* buf, F input) {
   const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv, lane = threadIdx.x & 31;
   const bool unit = r < 2 * p.kv_heads;
   const int base = unit ? r * p.dk : 2 * qk + (r - 2 * p.kv_heads) * p.dv, size = unit ? p.dk : p.dv;
   float* out = p.out + (size_t)t * channels + base;
   float ss = 0.f;
-  for (int d = lane; d < size; d += 32) {
-    float sum = 0.f;
+  for (int d = lane * V; d < size; d += 32 * V) {
+    float y[V], w[V], x[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] = 0.f;
 #pragma unroll 4
-    for (int j = p.taps - 1; j >= 0; --j) sum = fmaf(p.conv[(size_t)(p.taps - 1 - j) * channels + base + d], input(j)[base + d], sum);
-    const float y = sum / (1.f + expf(-sum));
-    if (unit) buf[d] = y;
-    else out[d] = y;
-    ss = fmaf(y, y, ss);
+    for (int j = p.taps - 1; j >= 0; --j) {
+      dp_load<V>(p.conv + (size_t)(p.taps - 1 - j) * channels + base + d, w), dp_load<V>(input(j) + base + d, x);
+#pragma unroll
+      for (int e = 0; e < V; ++e) y[e] = fmaf(w[e], x[e], y[e]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) {
+      y[e] = y[e] / (1.f + expf(-y[e]));
+      ss = fmaf(y[e], y[e], ss);
+    }
+    dp_store<V>(unit ? buf + d : out + d, y);
   }
   if (!unit) return;
   const float inv = (r < p.kv_heads ? 1.f / sqrtf((float)p.dk) : 1.f) / sqrtf(warp_sum(ss) + 1e-6f);
-  for (int d = lane; d < size; d += 32) out[d] = buf[d] * inv;
+  for (int d = lane * V; d < size; d += 32 * V) {
+    float y[V];
+    dp_load<V>(buf + d, y);
+#pragma unroll
+    for (int e = 0; e < V; ++e) y[e] *= inv;
+    dp_store<V>(out + d, y);
+  }
 }
 
 __device__ __forceinline__ void delta_prepare_gates(const DeltaPrepare& p, int t) {
@@ -73,6 +90,7 @@ __device__ __forceinline__ void delta_prepare_gates(const DeltaPrepare& p, int t
   }
 }
 
+template <int V>
 __global__ void __launch_bounds__(32 * DP_WARPS) delta_prepare_kernel(DeltaPrepare p) {
   extern __shared__ __align__(16) float smem[];      // [DP_WARPS][dk]
   pdl_trigger();
@@ -84,7 +102,7 @@ __global__ void __launch_bounds__(32 * DP_WARPS) delta_prepare_kernel(DeltaPrepa
     // a token with all its taps inside the step
     const int t = blockIdx.x;
     if (t - p.cu_tokens[p.token_entry[t]] < back) return;
-    if (r < rows) delta_prepare_row(p, t, r, buf, [&](int j) { return p.proj + (size_t)(t - j) * p.ld; });
+    if (r < rows) delta_prepare_row<V>(p, t, r, buf, [&](int j) { return p.proj + (size_t)(t - j) * p.ld; });
     if (blockIdx.y == 0) delta_prepare_gates(p, t);
     return;
   }
@@ -98,11 +116,12 @@ __global__ void __launch_bounds__(32 * DP_WARPS) delta_prepare_kernel(DeltaPrepa
   const int qk = p.kv_heads * p.dk, channels = 2 * qk + p.heads * p.dv;
   float* st = p.state + (size_t)p.slots[entry] * back * channels;
   for (int i = 0; i < edge; ++i)
-    delta_prepare_row(p, first + i, r, buf, [&](int j) {
+    delta_prepare_row<V>(p, first + i, r, buf, [&](int j) {
       return j <= i ? p.proj + (size_t)(first + i - j) * p.ld : (const float*)st + (size_t)(back + i - j) * channels;
     });
-  // the last taps - 1 rows of (state rows, the step's rows); a channel is one lane's, which reads a
-  // state row only before it overwrites it
+  // the last taps - 1 rows of (state rows, the step's rows), once the warp has read the old ones; a
+  // channel is one lane's here, which reads a state row only before it overwrites it
+  __syncwarp();
   const int base = r < 2 * p.kv_heads ? r * p.dk : 2 * qk + (r - 2 * p.kv_heads) * p.dv;
   for (int d = lane; d < (r < 2 * p.kv_heads ? p.dk : p.dv); d += 32)
     for (int k = 0; k < back; ++k) {
@@ -122,8 +141,11 @@ FE_EXPORT int fe_delta_prepare(const float* proj, long long ld, int b_off, int a
   const size_t smem = sizeof(float) * (size_t)DP_WARPS * dk;
   const int pieces = (2 * kv_heads + heads + DP_WARPS - 1) / DP_WARPS;
   if (smem > 48 * 1024 || pieces > 65535) return FE_ERR_TOO_LARGE;
-  const int rc = fe_launch_dependent(delta_prepare_kernel, dim3(n_tokens + (taps > 1 ? n_entries : 0), pieces), dim3(32 * DP_WARPS), smem,
-                                     stream, p);
+  const bool wide = dk % 4 == 0 && dv % 4 == 0 && ld % 4 == 0 &&
+                    (((uintptr_t)proj | (uintptr_t)conv | (uintptr_t)state | (uintptr_t)out) & 15) == 0;
+  const dim3 grid(n_tokens + (taps > 1 ? n_entries : 0), pieces);
+  const int rc = wide ? fe_launch_dependent(delta_prepare_kernel<4>, grid, dim3(32 * DP_WARPS), smem, stream, p)
+                      : fe_launch_dependent(delta_prepare_kernel<1>, grid, dim3(32 * DP_WARPS), smem, stream, p);
   return rc ? rc : fe_last_error();
 }
 
