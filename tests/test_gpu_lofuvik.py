@@ -375,18 +375,22 @@ OTHER = {
 }
 
 
+@pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("name", sorted(OTHER))
-def test_other_sizes_and_values_that_are_one_or_equal(tmp_path, name):
+def test_other_sizes_and_values_that_are_one_or_equal(tmp_path, name, dtype):
     options = dict(OTHER[name])
-    cfg = pl.config(options.pop("layers"), **options)
+    layers = options.pop("layers")
+    if dtype == "bfloat16":      # no router that chooses
+        layers = [dict(layer, mlp=layer["mlp"] and pl.routed(experts=2, top=2, ff=layer["mlp"]["expert"]["ff"])) for layer in layers]
+    cfg = pl.config(layers, **options)
     weights = write_model(tmp_path / "m", cfg, 21)
     tokens = tokens_of(cfg, 140, 10)
-    runner = make_runner(tmp_path / "m", "float32", page_size=8, num_pages=48)
+    runner = make_runner(tmp_path / "m", dtype, page_size=8, num_pages=48)
     ref = oracle(cfg, weights, tokens)
     whole = run_schedule(runner, {"a": tokens}, [[("a", 140)]])["a"]
     cut = run_schedule(runner, {"b": tokens}, [[("b", 19)], [("b", 2)], [("b", 101)], [("b", 2)]] + [[("b", 1)] for _ in range(16)])["b"]
-    assert_close(whole, ref, "float32", name)
-    assert_close(cut, ref, "float32", name + ", cut")
+    assert_close(whole, ref, dtype, name)
+    assert_close(cut, ref, dtype, name + ", cut")
 
 
 @pytest.mark.parametrize("rank", (1, 3, 48))
