@@ -27,17 +27,31 @@ class PagedKVSpec:
     ``v_head_dim``: size of a value head where it differs (None: ``head_dim``; 0: the run
     keeps one vector per token and head, no second one - a latent that is key and value).
     ``keep_first``: with a window, positions below it stay visible for ever, so the pages
-    that hold them are never given back."""
+    that hold them are never given back.  ``chunk`` (not together with a window): a token sees
+    its own chunk of that many positions only, counted from position 0."""
 
     num_kv_heads: int
     head_dim: int
     window: int | None = None
     v_head_dim: int | None = None
     keep_first: int = 0
+    chunk: int | None = None
 
     def kept_pages(self, page_size: int) -> int:
         """Leading pages a window never releases."""
         return 0 if self.window is None or self.keep_first <= 0 else _ceil_div(self.keep_first, page_size)
+
+    @property
+    def reach(self) -> int | None:
+        """Most keys a token sees, or None where it sees every earlier one."""
+        return self.window if self.chunk is None else self.chunk
+
+    def first_needed(self, position: int) -> int:
+        """The first position that the token at ``position`` and those after it see (kept first
+        tokens aside)."""
+        if self.chunk is not None:
+            return position - position % self.chunk
+        return 0 if self.window is None else max(0, position - self.window + 1)
 
     @property
     def value_dim(self) -> int:
@@ -309,18 +323,16 @@ class CacheManager:
             del table.pages[keep:]
 
     def advance(self, key, new_length: int) -> None:
-        """Record that positions < new_length are written; release pages a window has passed."""
+        """Record that positions < new_length are written; release pages a window or chunk has passed."""
         entry = self.request(key)
         if new_length < entry.length:
             raise ValueError("a request's length cannot shrink")
         entry.length = new_length
         for group, table in zip(self.groups, entry.tables):
-            window = group.spec.window
-            if window is None:
+            if group.spec.reach is None:
                 continue
-            # the next query sits at position new_length and sees keys >= new_length - window + 1
-            first_needed = new_length - window + 1
-            dead_pages = max(0, first_needed) // self.page_size
+            # the next query sits at position new_length
+            dead_pages = group.spec.first_needed(new_length) // self.page_size
             dead_pages = min(dead_pages, len(table.pages))
             released = []
             # pages that hold kept first tokens stay; ``first_live`` counts from behind them
@@ -351,11 +363,11 @@ class CacheManager:
         out = []
         full = _ceil_div(total_length, self.page_size)
         for group in self.groups:
-            window = group.spec.window
-            if window is None:
+            reach = group.spec.reach
+            if reach is None:
                 out.append(full)
             else:
-                span = window - 1 + max_portion  # live keys just before a step's release
+                span = reach - 1 + max_portion  # live keys just before a step's release
                 out.append(min(full, _ceil_div(span, self.page_size) + 1 + group.spec.kept_pages(self.page_size)))
         return out
 

@@ -2,6 +2,7 @@
 
 from .engine import EngineConfig, SchedulerConfig
 from .lofuvik import LofuvikConfig
+from .lozezen import LozezenConfig
 from .nuvivik import NuvivikConfig
 from .qwen3 import Qwen3Config
 from .registry import (
@@ -27,10 +28,13 @@ from .specs import (
     NoPositionSpec,
     NormSpec,
     OutputNormSpec,
+    RetentionSpec,
+    RGLRUSpec,
     RotarySpec,
     RoutedMLPSpec,
     RunSpec,
     SandwichConvSpec,
+    SandwichSpec,
     SideBySideSpec,
     StreamMixSpec,
     WKVSpec,
@@ -67,6 +71,11 @@ register_architecture(
     replace=True,
 )
 
+register_architecture(
+    Architecture("Lozezen", LozezenConfig.from_dict, LozezenConfig.to_model_spec),
+    replace=True,
+)
+
 __all__ = [
     "Architecture",
     "AttentionSpec",
@@ -81,6 +90,7 @@ __all__ = [
     "LayerSpec",
     "LinearRecurrenceSpec",
     "LofuvikConfig",
+    "LozezenConfig",
     "MatrixMemorySpec",
     "ModelSpec",
     "NoPositionSpec",
@@ -88,10 +98,13 @@ __all__ = [
     "NuvivikConfig",
     "OutputNormSpec",
     "Qwen3Config",
+    "RGLRUSpec",
+    "RetentionSpec",
     "RotarySpec",
     "RoutedMLPSpec",
     "RunSpec",
     "SandwichConvSpec",
+    "SandwichSpec",
     "SchedulerConfig",
     "SideBySideSpec",
     "StreamMixSpec",

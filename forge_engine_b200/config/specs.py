@@ -76,6 +76,8 @@ class RotarySpec:
     # ln(original / (2 pi t)) / (2 ln theta), lo = max(floor(dim(fast)), 0), hi = min(ceil(dim(slow)),
     # rotary_dim - 1); cosine and sine are multiplied by 0.1 ln(factor) + 1 ("YaRN").
     yarn: tuple | None = None
+    # Every frequency is divided by this number ("linear scaling").
+    frequency_divisor: float = 1.0
 
 
 @dataclass(frozen=True)
@@ -149,6 +151,9 @@ class AttentionSpec:
     # True: the heads' outputs are multiplied element by element by sigmoid(W x), x the mixer's input;
     # the checkpoint holds ``gate_proj.weight`` [heads * v_head_dim, hidden].  (Not with ``head_gate``.)
     output_gate: bool = False
+    # None, or c: the sequence is cut into chunks of c positions, counted from position 0, and a query
+    # sees the keys of its own chunk up to its own position.  (Not with ``window``.)
+    chunk: int | None = None
 
 
 @dataclass(frozen=True)
@@ -207,6 +212,44 @@ class LinearRecurrenceSpec:
     norm_eps: float
     activation: str = "silu"
     kind: str = "linear_recurrence"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
+class RetentionSpec:
+    """Retention: linear attention with a fixed decay per head and no activation, S_t = decay_h S_(t-1)
+    + c k_t v_t^T, o_t = S_t^T q_t with q and k rotated by ``position`` (a RotarySpec or NoPositionSpec)
+    and c = ``key_scale``.  Each head's o is divided by its root mean square over its values, multiplied
+    by silu(W_g x) and projected; ``norm_weight``: and by one weight vector [v_head_dim] before the gate
+    (tensor ``norm``)."""
+
+    hidden_size: int
+    num_heads: int
+    head_dim: int
+    v_head_dim: int
+    decay: tuple
+    norm_eps: float
+    position: object
+    key_scale: float = 1.0
+    norm_weight: bool = False
+    kind: str = "retention"
+    rename: tuple = ()
+
+
+@dataclass(frozen=True)
+class RGLRUSpec:
+    """Griffin's recurrent block around a real-gated linear recurrent unit: y = gelu_tanh(W_y x + b) and
+    u = conv(W_x x + b), a causal convolution over time with ``taps`` taps and a bias per channel, both of
+    ``width``; u falls into ``blocks`` equal parts, each with gates r = sigmoid(R_b u_b + b) and
+    i = sigmoid(I_b u_b + b); log a = -``strength`` r softplus(lam); S_t = a S_(t-1) + sqrt(1 - a^2) i u
+    per channel from zero, and W_o (S y)."""
+
+    hidden_size: int
+    width: int
+    blocks: int
+    taps: int
+    strength: float = 8.0
+    kind: str = "rglru"
     rename: tuple = ()
 
 
@@ -288,7 +331,8 @@ class MatrixMemorySpec:
 class SideBySideSpec:
     """Two mixers that read the same input; the result is half the sum of their outputs, each
     divided by its root mean square over the width and weighted (tensors ``left.<name>`` and
-    ``right.<name>`` of the mixers, ``left.out`` and ``right.out`` [hidden] of the norms)."""
+    ``right.<name>`` of the mixers, ``left.out`` and ``right.out`` [hidden] of the norms), or with
+    ``scales`` (a, b) a * left + b * right as they are (no norms, no tensors of its own)."""
 
     hidden_size: int
     left: object
@@ -296,6 +340,7 @@ class SideBySideSpec:
     norm_eps: float
     kind: str = "side_by_side"
     rename: tuple = ()
+    scales: tuple | None = None
 
 
 @dataclass(frozen=True)
@@ -401,6 +446,17 @@ class StreamMixSpec:
     streams: int = 1
     learned: bool = False
     update_scale: float = 1.0
+
+
+@dataclass(frozen=True)
+class SandwichSpec:
+    """Options of the "sandwich" arrangement: a norm on both sides of every sublayer,
+    x += norm_b(sublayer(norm(x))), for the mixer and then for the feed-forward.
+    ``mixer_out_norm`` / ``ffn_out_norm``: the specs of the norms norm_b (roles of the same
+    names; the second is None for a layer without feed-forward)."""
+
+    mixer_out_norm: object = None
+    ffn_out_norm: object = None
 
 
 @dataclass(frozen=True)

@@ -19,6 +19,14 @@ struct PagedKV {
   int head_dim;
 };
 
+// First key position a query at `pos` sees: a window keeps the `window` most recent keys (its own
+// included); chunks of `chunk` tokens, counted from the sequence's start, keep those of the query's own
+// chunk; with neither (both zero) every earlier key is seen.
+__device__ __forceinline__ int first_visible_key(int pos, int window, int chunk) {
+  if (chunk > 0) return pos > 0 ? pos - pos % chunk : 0;
+  return window > 0 ? max(0, pos - window + 1) : 0;
+}
+
 // Element offset of (page, head, slot, 0).
 __device__ __forceinline__ size_t kv_offset(const PagedKV& c, int page, int head, int slot) {
   return (((size_t)page * c.num_kv_heads + head) * c.page_size + slot) * c.head_dim;

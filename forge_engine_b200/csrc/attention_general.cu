@@ -219,6 +219,7 @@ struct GeneralAttn {
   const float* dist_bias;   // or null: [heads, dist_len], s += dist_bias[head, min(pos - key, dist_len - 1)]
   int dist_len;
   int window;
+  int chunk;                // above zero (and no window): keys of the query's own chunk only, see first_visible_key
   float scale;
   // What the plain layer does not have (all off when zero / null):
   int keep_first;           // with a window: keys below this position stay visible to every query
@@ -258,7 +259,7 @@ attention_general_kernel(GeneralAttn a, int* status) {
   float* part_m = part_acc + GA_WARPS * RMAX * a.v_dim; // [GA_WARPS][RMAX]
   float* part_l = part_m + GA_WARPS * RMAX;
   const int pos = a.positions[token], entry = a.token_entry[token];
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int lo = first_visible_key(pos, a.window, a.chunk);
   const int* table = a.block_table + (size_t)entry * a.max_pages;
   const int head0 = kvh * groups + first;
 
@@ -463,7 +464,7 @@ FE_EXPORT int fe_attention_general(const void* q, long long q_token_stride, long
                                    long long o_token_stride, long long o_head_stride, int dtype, const int* block_table,
                                    int max_pages, int page_size, int num_pages, int num_kv_heads, int num_q_heads,
                                    const int* positions, const int* token_entry, const float* slopes,
-                                   const float* dist_bias, int dist_len, int window,
+                                   const float* dist_bias, int dist_len, int window, int chunk,
                                    float scale, int keep_first, float softcap, float temp_coef, int temp_every,
                                    int parts, long long q_part_stride, int k_part_stride, long long o_part_stride,
                                    const float* gate, long long gate_stride, int gate_dim, int out_f32, const float* sinks,
@@ -472,10 +473,11 @@ FE_EXPORT int fe_attention_general(const void* q, long long q_token_stride, long
   if (parts < 1) parts = 1;
   if (num_kv_heads < 1 || num_q_heads % num_kv_heads || (long long)num_kv_heads * parts > 65535) return FE_ERR_BAD_SHAPE;
   if (k_dim < 1 || v_dim < 1 || k_part_stride * (parts - 1) + k_dim > k_row || v_dim > v_row) return FE_ERR_BAD_SHAPE;
+  if (window < 0 || chunk < 0 || (window > 0 && chunk > 0)) return FE_ERR_BAD_SHAPE;
   if (keep_first < 0 || temp_every < 0 || softcap < 0.f || (dist_bias != nullptr && dist_len < 1)) return FE_ERR_BAD_SHAPE;
   GeneralAttn a{q, q_token_stride, q_head_stride, k_cache, k_row, k_dim, v_cache, v_row, v_dim, out, o_token_stride,
                 o_head_stride, block_table, max_pages, page_size, num_pages, num_kv_heads, num_q_heads, positions,
-                token_entry, slopes, dist_bias, dist_len, window, scale, keep_first, softcap, temp_coef, temp_every, parts, q_part_stride,
+                token_entry, slopes, dist_bias, dist_len, window, chunk, scale, keep_first, softcap, temp_coef, temp_every, parts, q_part_stride,
                 k_part_stride, o_part_stride, gate, gate_stride, gate_dim, out_f32, sinks};
   if (dtype == FE_DTYPE_F32) return dispatch_general<float>(a, n_tokens, status, stream);
   if (dtype == FE_DTYPE_BF16) return dispatch_general<bf16>(a, n_tokens, status, stream);

@@ -12,6 +12,7 @@
 // Few rows and many keys (decoding): `splits` blocks share a row tile's key tiles and leave
 // (sum, maximum, normaliser) in a workspace that a second kernel combines.
 #include "attention_common.cuh"
+#include "mma_sync.cuh"
 
 #ifndef FE_DK
 #error "compile with -DFE_DK=... -DFE_DV=... -DFE_V_IN_K=..."
@@ -49,7 +50,7 @@ struct Params {
   void* out; long long o_ts, o_hs;
   const int* table; int max_pages, page_size, num_pages, nkv, groups;
   const int* cu_tokens; const int* starts;
-  const float* slopes; const float* dist_bias; int dist_len; int window; float scale;
+  const float* slopes; const float* dist_bias; int dist_len; int window, chunk; float scale;
   int splits; int tiles; float* part;
   // what the plain layer does not have (off when zero / null); see GeneralAttn in attention_general.cu
   int keep_first; float softcap, temp_coef; int temp_every;
@@ -66,40 +67,6 @@ __device__ __forceinline__ float sigmoidf(float x) { return 1.f / (1.f + expf(-x
 // tanh as 1 - 2 / (1 + e^(2x)) on the fast exponential: the absolute error stays below 3e-7,
 // which is what a capped score (cap * tanh, the cap a few tens) needs; it saturates to +-1
 __device__ __forceinline__ float tanh_capped(float x) { return 1.f - __fdividef(2.f, 1.f + __expf(2.f * x)); }
-
-__device__ __forceinline__ unsigned smem_addr(const void* p) { return (unsigned)__cvta_generic_to_shared(p); }
-
-__device__ __forceinline__ void cp_async16(void* dst, const void* src, bool valid) {
-  const int bytes = valid ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(bytes) : "memory");
-}
-__device__ __forceinline__ void cp_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
-
-__device__ __forceinline__ void ldsm4(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(smem_addr(p)));
-}
-__device__ __forceinline__ void ldsm4_trans(unsigned& r0, unsigned& r1, unsigned& r2, unsigned& r3, const void* p) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];"
-               : "=r"(r0), "=r"(r1), "=r"(r2), "=r"(r3) : "r"(smem_addr(p)));
-}
-__device__ __forceinline__ void mma16816(float* c, const unsigned* a, unsigned b0, unsigned b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-               : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ unsigned pack2(float x, float y) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  return *reinterpret_cast<const unsigned*>(&h);
-}
-// the rounded pair and the rounded remainders
-__device__ __forceinline__ void split2(float x, float y, unsigned& hi, unsigned& lo) {
-  const __nv_bfloat162 h = __floats2bfloat162_rn(x, y);
-  const float2 back = __bfloat1622float2(h);
-  hi = *reinterpret_cast<const unsigned*>(&h);
-  lo = pack2(x - back.x, y - back.y);
-}
 
 __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, int* status) {
   extern __shared__ __align__(16) unsigned char raw[];
@@ -134,7 +101,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
 
   const int tok_lo = row0 / p.groups, tok_hi = min(count - 1, (row0 + BM - 1) / p.groups);
   const int key_hi = start + tok_hi;                                        // last key any row sees
-  const int key_lo = p.window > 0 ? max(0, start + tok_lo - p.window + 1) : 0;
+  const int key_lo = first_visible_key(start + tok_lo, p.window, p.chunk);
   const int kt_lo = key_lo / BN, kt_hi = key_hi / BN + 1;
   // keys below keep_first stay visible after the window has passed them: their tiles (those that
   // lie before the window's first tile) are walked first; step i of the walk is key tile tile_of(i)
@@ -172,7 +139,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
 
   // this thread's two rows: r_a = lane / 4 and r_a + 8 of the warp's sixteen
   const int quad = lane >> 2, pair = lane & 3;
-  int row_pos[2];
+  int row_pos[2], row_lo[2];   // position, first key seen
   float row_slope[2], row_scale[2];
   const float* row_bias[2];    // the row's head in the table of biases by distance, or null
   bool row_live[2];
@@ -185,6 +152,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
     const int rho = row0 + rw * 16 + quad + 8 * h;
     row_live[h] = rho < rows_total;
     row_pos[h] = row_live[h] ? start + rho / p.groups : -1;
+    row_lo[h] = first_visible_key(max(row_pos[h], 0), p.window, p.chunk);
     row_slope[h] = (row_live[h] && p.slopes) ? p.slopes[kvh * p.groups + rho % p.groups] * LOG2E : 0.f;
     row_bias[h] = (row_live[h] && p.dist_bias) ? p.dist_bias + (size_t)(kvh * p.groups + rho % p.groups) * p.dist_len : nullptr;
     const float natural = p.scale * query_temperature(max(row_pos[h], 0), p.temp_coef, p.temp_every);
@@ -193,6 +161,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
   // rows of this warp, first and last position (all sixteen live), for tiles that need no mask
   const bool warp_full = row0 + rw * 16 + 15 < rows_total;
   const int warp_pos_lo = start + (row0 + rw * 16) / p.groups, warp_pos_hi = start + (row0 + rw * 16 + 15) / p.groups;
+  const int warp_lo = first_visible_key(warp_pos_hi, p.window, p.chunk);       // the first key all of them see
   const bool warp_live = row0 + rw * 16 < rows_total;
   float o[DVW / 8][4];
 #pragma unroll
@@ -245,7 +214,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
     // scale, bias, mask; running maximum and normaliser
     float mx[2] = {-INFINITY, -INFINITY};
     // every key of the tile is visible to every row of the warp: no comparisons
-    const bool inside = warp_full && kt * BN + BN - 1 <= warp_pos_lo && (p.window <= 0 || kt * BN > warp_pos_hi - p.window);
+    const bool inside = warp_full && kt * BN + BN - 1 <= warp_pos_lo && kt * BN >= warp_lo;
     if (inside) {
 #pragma unroll
       for (int j = 0; j < BN / 8; ++j) {
@@ -268,8 +237,7 @@ __global__ void __launch_bounds__(WARPS * 32, 1) attention_mma_kernel(Params p, 
         for (int c = 0; c < 4; ++c) {
           const int h = c >> 1;
           const int key = kt * BN + j * 8 + pair * 2 + (c & 1);
-          const bool visible = row_live[h] && key <= row_pos[h] &&
-                               (p.window <= 0 || key > row_pos[h] - p.window || key < sink_keys);
+          const bool visible = row_live[h] && key <= row_pos[h] && (key >= row_lo[h] || key < sink_keys);
           float sc = s[j][c] * row_scale[h];
           if (capped) sc = cap2 * tanh_capped(sc);
           sc = visible ? sc - row_slope[h] * (float)(row_pos[h] - key) : -INFINITY;
@@ -453,7 +421,7 @@ FE_EXPORT int GM_NAME(fe_attention_gmma_)(const void* q, long long q_ts, long lo
                                           const int* block_table, int max_pages, int page_size, int num_pages, int nkv,
                                           int num_q_heads, const int* cu_tokens, const int* starts, int entries,
                                           int max_new, const float* slopes, const float* dist_bias, int dist_len,
-                                          int window, float scale, int splits,
+                                          int window, int chunk, float scale, int splits,
                                           float* workspace, int keep_first, float softcap, float temp_coef,
                                           int temp_every, int parts, long long q_ps, int k_ps, long long o_ps,
                                           const float* gate, long long gate_stride, int gate_dim, int out_f32, int row_hi,
@@ -461,6 +429,7 @@ FE_EXPORT int GM_NAME(fe_attention_gmma_)(const void* q, long long q_ts, long lo
   if (entries <= 0 || max_new <= 0) return 0;
   if (parts < 1) parts = 1;
   if (nkv < 1 || num_q_heads % nkv || (long long)nkv * parts > 65535 || entries > 65535) return FE_ERR_BAD_SHAPE;
+  if (window < 0 || chunk < 0 || (window > 0 && chunk > 0)) return FE_ERR_BAD_SHAPE;
   if (dist_bias != nullptr && dist_len < 1) return FE_ERR_BAD_SHAPE;
   if (keep_first < 0 || temp_every < 0 || softcap < 0.f || k_ps * (parts - 1) + DK > k_row) return FE_ERR_BAD_SHAPE;
   if (k_row % 8 || v_row % 8 || q_ts % 8 || q_hs % 8 || o_ts % 2 || o_hs % 2 || q_ps % 8 || k_ps % 8 || o_ps % 2) return FE_ERR_BAD_ALIGN;
@@ -471,7 +440,7 @@ FE_EXPORT int GM_NAME(fe_attention_gmma_)(const void* q, long long q_ts, long lo
   const int groups = num_q_heads / nkv;
   const int tiles = (int)(((long long)max_new * groups + BM - 1) / BM);
   Params p{(const bf16*)q, q_ts, q_hs, (const bf16*)k_cache, k_row, (const bf16*)v_cache, v_row, out, o_ts, o_hs,
-           block_table, max_pages, page_size, num_pages, nkv, groups, cu_tokens, starts, slopes, dist_bias, dist_len, window, scale,
+           block_table, max_pages, page_size, num_pages, nkv, groups, cu_tokens, starts, slopes, dist_bias, dist_len, window, chunk, scale,
            splits, tiles, workspace, keep_first, softcap, temp_coef, temp_every, parts, q_ps, k_ps, o_ps, gate,
            gate_stride, gate_dim, out_f32, row_hi, sinks};
   static bool configured = false;

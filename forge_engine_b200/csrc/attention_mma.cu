@@ -73,6 +73,7 @@ struct AttnParams {
   // sigmoid(gate[token * gate_stride + head * gate_dim + d]); exp(sinks[head]) joins the softmax's
   // denominator once, with no key and no value.
   int keep_first = 0;
+  int chunk = 0;         // above zero (and no window): keys of the query's own chunk only, see first_visible_key
   const float* gate = nullptr;
   long long gate_stride = 0;
   int gate_dim = 0;
@@ -1181,7 +1182,8 @@ static __device__ __align__(256) float fe_noalloc_scratch[FE_NOALLOC_SCRATCH_FLO
 
 // The tcgen05 prefill kernel alone, for layers whose other entries another kernel serves:
 // entries with more than `row_lo` rows (new tokens x heads per kv head).  Beyond what
-// fe_attention_mma_d gives it: with a window, keys below `keep_first` stay visible; row
+// fe_attention_mma_d gives it: `chunk` above zero shows a query the keys of its own chunk only; with a
+// window, keys below `keep_first` stay visible; row
 // (token, head) of `out` is multiplied by sigmoid(gate[token * gate_stride + head]) (gate
 // null: no gate); `softcap` above zero caps the scaled scores by softcap tanh(. / softcap) (not
 // together with dist_bias).  q rows are `q_stride` apart, out is [tokens, heads * D].  Returns
@@ -1190,13 +1192,14 @@ static __device__ __align__(256) float fe_noalloc_scratch[FE_NOALLOC_SCRATCH_FLO
 FE_EXPORT int SYM(fe_attention_prefill_tc5_d)(const void* q, int q_stride, void* out, const void* k_cache,
                                               const void* v_cache, const int* block_table, int max_pages, int page_size,
                                               int num_pages, int num_kv_heads, int groups, const int* cu_tokens,
-                                              const int* starts, int entries, int max_new, int total_tokens, int window,
+                                              const int* starts, int entries, int max_new, int total_tokens, int window, int chunk,
                                               int keep_first, float scale, const float* gate, long long gate_stride,
                                               int gate_dim, int row_lo, const float* dist_bias, int dist_len, float softcap,
                                               const float* sinks,
                                               int* status, cudaStream_t stream) {
   if (entries <= 0 || max_new * groups <= row_lo) return 0;
   if (dist_bias != nullptr && dist_len < 1) return FE_ERR_BAD_SHAPE;
+  if (window < 0 || chunk < 0 || (window > 0 && chunk > 0)) return FE_ERR_BAD_SHAPE;
   if (softcap < 0.f || (softcap > 0.f && dist_bias != nullptr)) return FE_ERR_BAD_SHAPE;
   if (gate_dim > 0 && (gate_dim != D || ((uintptr_t)gate & 15) || gate_stride % 4)) return FE_ERR_BAD_ALIGN;
   if (entries > 65535 || num_kv_heads > 65535) return FE_ERR_TOO_LARGE;
@@ -1213,7 +1216,7 @@ FE_EXPORT int SYM(fe_attention_prefill_tc5_d)(const void* q, int q_stride, void*
   p.window = window; p.scale_log2 = scale * 1.4426950408889634f; p.status = status;
   p.row_lo = row_lo; p.row_hi = 0x7fffffff;
   p.num_splits = 1; p.ws_acc = nullptr; p.ws_ml = nullptr; p.ws_count = nullptr; p.cluster_merge = 0;
-  p.keep_first = keep_first; p.gate = gate; p.gate_stride = gate_stride; p.gate_dim = gate_dim; p.sinks = sinks;
+  p.keep_first = keep_first; p.chunk = chunk; p.gate = gate; p.gate_stride = gate_stride; p.gate_dim = gate_dim; p.sinks = sinks;
   p.dist_bias = dist_bias; p.dist_len = dist_len;
   if (softcap > 0.f) { p.cap_over_scale = softcap / scale; p.scale_over_cap = scale / softcap; }
   CUtensorMap mk, mv, mq;

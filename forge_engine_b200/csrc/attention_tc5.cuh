@@ -190,14 +190,14 @@ struct Tc5Tile {
   bool valid;
   int row0, pos_first, pos_last, key_end, tile_begin, tile_end;
 };
-__device__ __forceinline__ Tc5Tile tc5_tile(int row0, int rows_total, int start, int groups, int window) {
+__device__ __forceinline__ Tc5Tile tc5_tile(int row0, int rows_total, int start, int groups, int window, int chunk) {
   Tc5Tile t;
   t.row0 = row0;
   t.valid = row0 < rows_total;
   const int last_row = min(rows_total, row0 + TC5_ROWS) - 1;
   t.pos_first = start + row0 / groups;
   t.pos_last = start + last_row / groups;
-  const int key_lo = window > 0 ? max(0, t.pos_first - window + 1) : 0;
+  const int key_lo = first_visible_key(t.pos_first, window, chunk);
   t.key_end = t.pos_last + 1;
   t.tile_begin = key_lo / TC5_KEYS;
   t.tile_end = (t.key_end + TC5_KEYS - 1) / TC5_KEYS;
@@ -253,8 +253,8 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int* table = p.block_table + (size_t)entry * p.max_pages;
 
   // tile 1 holds later tokens: its keys start no earlier and end no earlier than tile 0's
-  const Tc5Tile t0 = tc5_tile(row0, rows_total, start, p.groups, p.window);
-  const Tc5Tile t1 = tc5_tile(row0 + TC5_ROWS, rows_total, start, p.groups, p.window);
+  const Tc5Tile t0 = tc5_tile(row0, rows_total, start, p.groups, p.window, p.chunk);
+  const Tc5Tile t1 = tc5_tile(row0 + TC5_ROWS, rows_total, start, p.groups, p.window, p.chunk);
   const int tile_begin = t0.tile_begin;
   const int tile_end = t1.valid ? t1.tile_end : t0.tile_end;
   // Keys below keep_first stay visible behind a window: the key tiles that hold them and lie
@@ -266,7 +266,7 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
   const int n_tiles = sink_tiles + tile_end - tile_begin;
   auto tile_of = [&](int i) -> int { return i < sink_tiles ? i : tile_begin + i - sink_tiles; };
   const int key_end = t1.valid ? t1.key_end : t0.key_end;
-  const int key_lo = p.window > 0 ? max(0, t0.pos_first - p.window + 1) : 0;
+  const int key_lo = first_visible_key(t0.pos_first, p.window, p.chunk);
   // does query tile x take part in step i?  (Tile 1's window starts later than tile 0's; a key
   // tile before it still counts for tile 1 when it holds kept keys.)
   auto active = [&](int x, int i) -> bool {
@@ -423,6 +423,9 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
     const unsigned lane_addr = tmem_base + ((unsigned)(quarter * 32) << 16);
     const unsigned s_addr = lane_addr + TC5_COL_S + x * TC5_KEYS;
     const unsigned o_addr = lane_addr + TC5_COL_O + x * 128;
+    const bool limited = p.window > 0 || p.chunk > 0;
+    const int row_lo = first_visible_key(pos, p.window, p.chunk);                      // first key this row sees
+    const int tile_lo = first_visible_key(mine.pos_last, p.window, p.chunk);           // first key all rows see
     float m_used = -INFINITY, l = 0.f;
     bool ok = mine.valid;
     unsigned count = 0;                                // key tiles this query tile has taken
@@ -454,12 +457,12 @@ attn_prefill_tc5_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_
       }
       // every key of the tile visible to every row of the tile?
       const bool clear = key0 + TC5_KEYS - 1 <= mine.pos_first && key0 + TC5_KEYS <= mine.key_end &&
-                         mine.row0 + TC5_ROWS <= rows_total && (p.window <= 0 || mine.pos_last - key0 < p.window);
+                         mine.row0 + TC5_ROWS <= rows_total && key0 >= tile_lo;
       if (!clear) {
         // this row sees the keys j_lo..j_hi of the tile (none when the row is past the end)
         const int j_hi = min(pos, mine.key_end - 1) - key0;
-        if (p.window > 0) {
-          const int j_lo = pos - p.window + 1 - key0, j_kept = sink_keys - key0;      // kept keys: j < j_kept
+        if (limited) {
+          const int j_lo = row_lo - key0, j_kept = sink_keys - key0;      // kept keys: j < j_kept
 #pragma unroll
           for (int j = 0; j < TC5_KEYS; ++j) raw[j] = (j <= j_hi && (j >= j_lo || j < j_kept)) ? raw[j] : 0xff800000u;   // -inf
         } else {

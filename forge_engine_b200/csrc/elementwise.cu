@@ -458,3 +458,34 @@ FE_EXPORT int fe_norm_pair(const float* a, const float* b, const float* w_a, con
   const int rc = fe_launch_dependent(norm_pair_kernel, dim3(rows), dim3(256), 0, stream, a, b, w_a, w_b, out, size, eps, scale);
   return rc ? rc : fe_last_error();
 }
+
+// ---------------------------------------------------------------------------
+// weighted_sum: out = sa * a + sb * b, all 32-bit (two mixers side by side, added as they are)
+// ---------------------------------------------------------------------------
+template <int V>
+__global__ void __launch_bounds__(256)
+weighted_sum_kernel(const float* __restrict__ a, const float* __restrict__ b, float sa, float sb, float* __restrict__ out, long long count) {
+  pdl_trigger();
+  pdl_wait();
+  const long long i = ((long long)blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (i >= count) return;
+  if constexpr (V == 4) {
+    float x[4], y[4];
+    load4(a + i, x), load4(b + i, y);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[e] = sa * x[e] + sb * y[e];
+    store4(out + i, x);
+  } else {
+    out[i] = sa * a[i] + sb * b[i];
+  }
+}
+
+FE_EXPORT int fe_weighted_sum(const float* a, const float* b, float sa, float sb, float* out, long long count, cudaStream_t stream) {
+  if (count <= 0) return 0;
+  const bool wide = count % 4 == 0 && (((uintptr_t)a | (uintptr_t)b | (uintptr_t)out) & 15) == 0;
+  const long long blocks = (count / (wide ? 4 : 1) + 255) / 256;
+  if (blocks > 0x7fffffffLL) return FE_ERR_TOO_LARGE;
+  const int rc = wide ? fe_launch_dependent(weighted_sum_kernel<4>, dim3((unsigned)blocks), dim3(256), 0, stream, a, b, sa, sb, out, count)
+                      : fe_launch_dependent(weighted_sum_kernel<1>, dim3((unsigned)blocks), dim3(256), 0, stream, a, b, sa, sb, out, count);
+  return rc ? rc : fe_last_error();
+}

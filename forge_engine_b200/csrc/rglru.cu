@@ -1,0 +1,604 @@
+// The real-gated linear recurrent unit of Griffin's recurrent block, with the short convolution in front
+// of it and the gate behind it.  Per channel c of `width`, in part b of `part` channels:
+//
+//     u_t = conv(x)_t + conv_b          causal, over time
+//     r = sigmoid(R_b u_b + br),  i = sigmoid(I_b u_b + bi)
+//     log a = rate r  (rate = -strength softplus(lam), at most 0),  a = exp(log a)
+//     S_t = a S_(t-1) + sqrt(1 - a^2) i u_t
+//     out_t = S_t gelu_tanh(y_t)
+//
+// x and y are 32-bit sums of the projection.  Everything here is 32-bit; with bfloat16 gate matrices u
+// enters their product as the sum of two bfloat16 numbers (the rounded one and the rounded remainder).
+//
+//   rglru_gates   tiles of RM tokens of the step (whatever entries they belong to) x NC channels of one
+//                 part: convolution, both products, gates, and the recurrence from zero inside the tile.
+//                 Leaves, per token, h (the state if the tile had started from zero, or the entry began
+//                 inside it) and the product of the a since then, so that S = h + prod * S_in.
+//   rglru_chain   walks an entry's tiles with one multiply-add each, leaves every tile's incoming state,
+//                 the request's new state, and the convolution's last inputs.
+//   rglru_out     S and the output of every token.
+//   rglru_step    steps in which every entry brings one token (bfloat16): all of it in one launch.  The
+//                 blocks of a part form a cluster; each convolves its own channels, moves their history
+//                 on and hands them to the others through shared memory.
+#include <cooperative_groups.h>
+
+#include "mma_sync.cuh"
+
+namespace cg = cooperative_groups;
+
+struct Rglru {
+  const float* proj;        // [tokens, ld]: y from column y_off, x from x_off
+  long long ld;
+  int y_off, x_off;
+  const float* conv_w;      // [taps, width], the last tap weighs the token itself
+  const float* conv_b;      // [width]
+  int taps;
+  const void *wr, *wi;      // [blocks, part, part], a gate's row is the output channel
+  const float *br, *bi, *rate;      // [width]
+  float* state;             // [rows, width]
+  float* conv_state;        // [rows, taps - 1, width], oldest first
+  int state_rows;
+  const int *slots, *cu_tokens, *token_entry;
+  int width, part, n_tokens, n_entries;
+  float *h, *prod;          // [tokens, width]
+  float *carry, *init;      // [tiles, width]: state before a tile's first token; [entries, width]: before an entry's
+  void* out;                // [tokens, width]
+};
+
+#define RG_KC 64            // channels of a part taken at a time
+#define RG_WP (RG_KC + 8)   // pitch of a bfloat16 tile
+#define RG_FP (RG_KC + 4)   // pitch of a 32-bit tile
+
+__device__ __forceinline__ float rg_sigmoid(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
+__device__ __forceinline__ float rg_gelu(float z) {
+  // 0.5 (1 + tanh(t)) = sigmoid(2 t)
+  return z * rg_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+// a and the input's factor sqrt(1 - a^2) i from the gates' sums
+__device__ __forceinline__ void rg_gates(float zr, float zi, float rate, float* a, float* scale) {
+  const float log_a = rate * rg_sigmoid(zr);
+  *a = expf(log_a);
+  *scale = sqrtf(-expm1f(2.f * log_a)) * rg_sigmoid(zi);
+}
+__device__ __forceinline__ void rg_copy4(void* dst, const void* src, bool valid) {
+  const int bytes = valid ? 4 : 0;
+  asm volatile("cp.async.ca.shared.global [%0], [%1], 4, %2;" ::"r"(smem_addr(dst)), "l"(src), "r"(bytes) : "memory");
+}
+
+// Rows n0 .. n0 + rows - 1 of one part's gate matrix, columns k0 .. k0 + cols - 1, into dst[row * pitch + col];
+// zero outside the matrix.  `cols` is a multiple of 8.
+__device__ __forceinline__ void rg_load_weight(bf16* dst, int pitch, const bf16* w, int part, int n0, int rows, int k0, int cols) {
+  if (part % 8 == 0) {
+    const int pieces = cols >> 3;
+    for (int i = threadIdx.x; i < rows * pieces; i += blockDim.x) {
+      const int n = i / pieces, k = (i - n * pieces) * 8;
+      const bool has = n0 + n < part && k0 + k < part;
+      cp_async16(dst + n * pitch + k, has ? w + (size_t)(n0 + n) * part + k0 + k : w, has);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < rows * cols; i += blockDim.x) {
+    const int n = i / cols, k = i - n * cols;
+    dst[n * pitch + k] = n0 + n < part && k0 + k < part ? w[(size_t)(n0 + n) * part + k0 + k] : __float2bfloat16_rn(0.f);
+  }
+}
+__device__ __forceinline__ void rg_load_weight(float* dst, int pitch, const float* w, int part, int n0, int rows, int k0, int cols) {
+  if (part % 4 == 0) {
+    const int pieces = cols >> 2;
+    for (int i = threadIdx.x; i < rows * pieces; i += blockDim.x) {
+      const int n = i / pieces, k = (i - n * pieces) * 4;
+      const bool has = n0 + n < part && k0 + k < part;
+      cp_async16(dst + n * pitch + k, has ? w + (size_t)(n0 + n) * part + k0 + k : w, has);
+    }
+    return;
+  }
+  for (int i = threadIdx.x; i < rows * cols; i += blockDim.x) {
+    const int n = i / cols, k = i - n * cols;
+    const bool has = n0 + n < part && k0 + k < part;
+    rg_copy4(dst + n * pitch + k, has ? w + (size_t)(n0 + n) * part + k0 + k : w, has);
+  }
+}
+
+// ---------------------------------------------------------------------------
+// rglru_gates
+// ---------------------------------------------------------------------------
+#define RG_RM 64            // tokens of a tile
+
+template <typename TW, int NC>
+struct RgShape {
+  static constexpr bool MMA = sizeof(TW) == 2;
+  static constexpr int THREADS = 4 * NC;
+  static constexpr int WPITCH = MMA ? RG_WP : RG_FP;
+  static constexpr size_t W_BYTES = sizeof(TW) * 2 * NC * WPITCH;                      // both gates, one stage
+  static constexpr size_t A_BYTES = MMA ? sizeof(bf16) * 2 * RG_RM * RG_WP : sizeof(float) * RG_RM * RG_FP;
+  static constexpr size_t U_BYTES = sizeof(float) * RG_RM * NC;
+  static constexpr size_t GATE_BYTES = sizeof(float) * 2 * RG_RM * (NC + 1);           // over the stages, afterwards
+  static size_t stages(int taps) {
+    const size_t s = 2 * (W_BYTES + sizeof(float) * (RG_RM + taps - 1) * RG_KC);
+    return s > GATE_BYTES ? s : GATE_BYTES;
+  }
+  static size_t bytes(int taps) { return stages(taps) + A_BYTES + U_BYTES; }
+};
+
+// TAPS: 4, or 0 for any number.
+template <typename TW, int NC, int TAPS>
+__global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int stage_bytes, int* status) {
+  using Shape = RgShape<TW, NC>;
+  extern __shared__ __align__(16) unsigned char raw[];
+  __shared__ int since[RG_RM], slot_of[RG_RM];       // tokens since the entry's first; the request's row (-1: past the end)
+  __shared__ float seg_h[4][NC], seg_p[4][NC];
+  pdl_trigger();
+  pdl_wait();
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n0 = blockIdx.x * NC, block = blockIdx.y, t0 = blockIdx.z * RG_RM;
+  const int part = p.part, taps = TAPS > 0 ? TAPS : p.taps, back = taps - 1;
+  const int rows = min(RG_RM, p.n_tokens - t0);
+  TW* ws = reinterpret_cast<TW*>(raw);                                         // [2 stages][2 gates][NC][pitch]
+  float* xs = reinterpret_cast<float*>(raw + 2 * Shape::W_BYTES);              // [2 stages][RM + back][KC]
+  unsigned char* as = raw + stage_bytes;                                       // u: hi and lo [RM][RG_WP], or 32-bit [RM][RG_FP]
+  float* us = reinterpret_cast<float*>(as + Shape::A_BYTES);                   // [RM][NC]: u of the block's own channels
+  if (tid < RG_RM) {
+    int s = -1, n = 0;
+    if (tid < rows) {
+      const int entry = p.token_entry[t0 + tid];
+      n = t0 + tid - p.cu_tokens[entry];
+      s = p.slots[entry];
+      if (s < 0 || s >= p.state_rows) {
+        atomicOr(status, FE_STATUS_BAD_PAGE);
+        s = -1;
+      }
+    }
+    since[tid] = n, slot_of[tid] = s;
+  }
+  const TW* wr = (const TW*)p.wr + (size_t)block * part * part;
+  const TW* wi = (const TW*)p.wi + (size_t)block * part * part;
+  const int x0 = block * part;                       // the part's first channel
+  const bool wide = part % 4 == 0 && p.ld % 4 == 0 && p.x_off % 4 == 0 && ((uintptr_t)p.proj & 15) == 0;
+  auto load = [&](int k0, int stage) {
+    TW* w = ws + stage * 2 * NC * Shape::WPITCH;
+    rg_load_weight(w, Shape::WPITCH, wr, part, n0, NC, k0, RG_KC);
+    rg_load_weight(w + NC * Shape::WPITCH, Shape::WPITCH, wi, part, n0, NC, k0, RG_KC);
+    float* x = xs + stage * (RG_RM + back) * RG_KC;
+    const float* src = p.proj + p.x_off + x0 + k0;
+    if (wide) {
+      for (int i = tid; i < (RG_RM + back) * (RG_KC / 4); i += Shape::THREADS) {
+        const int r = i / (RG_KC / 4), c = (i - r * (RG_KC / 4)) * 4, t = t0 + r - back;
+        const bool has = t >= 0 && t < p.n_tokens && k0 + c < part;
+        cp_async16(x + r * RG_KC + c, has ? src + (size_t)t * p.ld + c : p.proj, has);
+      }
+    } else {
+      for (int i = tid; i < (RG_RM + back) * RG_KC; i += Shape::THREADS) {
+        const int r = i / RG_KC, c = i - r * RG_KC, t = t0 + r - back;
+        const bool has = t >= 0 && t < p.n_tokens && k0 + c < part;
+        rg_copy4(x + r * RG_KC + c, has ? src + (size_t)t * p.ld + c : p.proj, has);
+      }
+    }
+    cp_commit();
+  };
+
+  // products: a warp takes 16 tokens x 32 channels of both gates; 32-bit: a thread 4 x 4
+  float acc[2][4][4];
+#pragma unroll
+  for (int g = 0; g < 2; ++g)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) acc[g][j][e] = 0.f;
+  const int rw = warp & 3, cw = warp >> 2;
+  const int fr = (tid & 15) * 4, fc = tid >> 4;      // 32-bit: rows fr .. fr + 3, channels fc + NC / 4 * e
+
+  load(0, 0);
+  for (int k0 = 0, stage = 0; k0 < part; k0 += RG_KC, stage ^= 1) {
+    if (k0 + RG_KC < part) {
+      load(k0 + RG_KC, stage ^ 1);
+      cp_wait<1>();
+    } else {
+      cp_wait<0>();
+    }
+    __syncthreads();
+    {
+      // the convolution: a thread takes one channel of RM / (NC / 16) neighbouring tokens
+      constexpr int GROUPS = Shape::THREADS / RG_KC, PER = RG_RM / GROUPS;
+      const int c = tid & (RG_KC - 1), r0 = (tid / RG_KC) * PER, ch = x0 + k0 + c;
+      const bool live = k0 + c < part;
+      const float* x = xs + stage * (RG_RM + back) * RG_KC + c;
+      const float bias = live ? p.conv_b[ch] : 0.f;
+      float w[TAPS > 0 ? TAPS : 1], hist[TAPS > 0 ? TAPS : 1];
+      if constexpr (TAPS > 0) {
+#pragma unroll
+        for (int j = 0; j < TAPS; ++j) {
+          w[j] = live ? p.conv_w[(size_t)j * p.width + ch] : 0.f;
+          hist[j] = j < TAPS - 1 ? x[(r0 + j) * RG_KC] : 0.f;
+        }
+      }
+#pragma unroll 4
+      for (int r = r0; r < r0 + PER; ++r) {
+        float u = bias;
+        if constexpr (TAPS > 0) hist[TAPS - 1] = x[(r + back) * RG_KC];
+        if (since[r] >= back) {
+          if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j < TAPS; ++j) u = fmaf(w[j], hist[j], u);
+          } else if (live) {
+            for (int j = 0; j < taps; ++j) u = fmaf(p.conv_w[(size_t)j * p.width + ch], x[(r + j) * RG_KC], u);
+          }
+        } else if (live) {
+          // an entry's first tokens: the inputs before them come from the request's state
+          for (int j = 0; j < taps; ++j) {
+            const int at = since[r] + j;             // index into (state rows, the entry's rows)
+            float v = 0.f;
+            if (at >= back) v = x[(r + j) * RG_KC];
+            else if (slot_of[r] >= 0) v = p.conv_state[((size_t)slot_of[r] * back + at) * p.width + ch];
+            u = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u);
+          }
+        }
+        if constexpr (TAPS > 0) {
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
+        }
+        if (!live || r >= rows) u = 0.f;
+        if constexpr (Shape::MMA) {
+          bf16* hi = reinterpret_cast<bf16*>(as) + r * RG_WP + c;
+          const bf16 rounded = __float2bfloat16_rn(u);
+          hi[0] = rounded;
+          hi[RG_RM * RG_WP] = __float2bfloat16_rn(u - __bfloat162float(rounded));
+        } else {
+          reinterpret_cast<float*>(as)[r * RG_FP + c] = u;
+        }
+        const int own = k0 + c - n0;
+        if (own >= 0 && own < NC) us[r * NC + own] = u;
+      }
+    }
+    __syncthreads();
+    const TW* w = ws + stage * 2 * NC * Shape::WPITCH;
+    if constexpr (Shape::MMA) {
+      const bf16* hi = reinterpret_cast<const bf16*>(as);
+#pragma unroll
+      for (int kk = 0; kk < RG_KC / 16; ++kk) {
+        unsigned ah[4], al[4];
+        const int a_at = (rw * 16 + (lane & 15)) * RG_WP + kk * 16 + (lane >> 4) * 8;
+        ldsm4(ah[0], ah[1], ah[2], ah[3], hi + a_at);
+        ldsm4(al[0], al[1], al[2], al[3], hi + RG_RM * RG_WP + a_at);
+#pragma unroll
+        for (int g = 0; g < 2; ++g) {
+#pragma unroll
+          for (int j = 0; j < 4; j += 2) {
+            unsigned b0, b1, b2, b3;
+            ldsm4(b0, b1, b2, b3, reinterpret_cast<const bf16*>(w) + (g * NC + cw * 32 + (j + (lane >> 4)) * 8 + (lane & 7)) * RG_WP +
+                                      kk * 16 + ((lane >> 3) & 1) * 8);
+            mma16816(acc[g][j], ah, b0, b1);
+            mma16816(acc[g][j + 1], ah, b2, b3);
+            mma16816(acc[g][j], al, b0, b1);
+            mma16816(acc[g][j + 1], al, b2, b3);
+          }
+        }
+      }
+    } else {
+      const float* u = reinterpret_cast<const float*>(as);
+      for (int k = 0; k < RG_KC; ++k) {
+        float a[4];
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[e] = u[(fr + e) * RG_FP + k];
+#pragma unroll
+        for (int g = 0; g < 2; ++g)
+#pragma unroll
+          for (int j = 0; j < 4; ++j) {
+            const float b = reinterpret_cast<const float*>(w)[(g * NC + fc + NC / 4 * j) * RG_FP + k];
+#pragma unroll
+            for (int e = 0; e < 4; ++e) acc[g][j][e] = fmaf(a[e], b, acc[g][j][e]);
+          }
+      }
+    }
+    __syncthreads();
+  }
+
+  // the sums of both gates, [gate][RM][NC + 1], over the stages
+  float* gates = reinterpret_cast<float*>(raw);
+  constexpr int GP = NC + 1;
+#pragma unroll
+  for (int g = 0; g < 2; ++g)
+#pragma unroll
+    for (int j = 0; j < 4; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        int r, c;
+        if constexpr (Shape::MMA) r = rw * 16 + (lane >> 2) + 8 * (e >> 1), c = cw * 32 + j * 8 + (lane & 3) * 2 + (e & 1);
+        else r = fr + e, c = fc + NC / 4 * j;
+        gates[(g * RG_RM + r) * GP + c] = acc[g][j][e];
+      }
+  __syncthreads();
+
+  // the recurrence from zero: a thread takes one channel of 16 tokens, then learns what the tile's
+  // earlier tokens leave (unless an entry begins in between)
+  const int c = tid % NC, seg = tid / NC, r_from = seg * 16;
+  const bool live = n0 + c < part;
+  const int ch = x0 + n0 + c;
+  float h = 0.f, prod = 1.f;
+  int fresh = RG_RM;                     // the segment's first row that begins an entry
+  if (live) {
+    const float br = p.br[ch], bi = p.bi[ch], rate = p.rate[ch];
+#pragma unroll 4
+    for (int r = r_from; r < r_from + 16; ++r) {
+      float a, scale;
+      rg_gates(gates[r * GP + c] + br, gates[(RG_RM + r) * GP + c] + bi, rate, &a, &scale);
+      if (since[r] == 0) {
+        h = 0.f, prod = 1.f;
+        if (fresh == RG_RM) fresh = r;
+      }
+      h = fmaf(a, h, scale * us[r * NC + c]);
+      prod *= a;
+      gates[r * GP + c] = h;
+      gates[(RG_RM + r) * GP + c] = prod;
+    }
+  }
+  seg_h[seg][c] = h, seg_p[seg][c] = prod;
+  __syncthreads();
+  if (!live) return;
+  float ch_in = 0.f, cp_in = 1.f;
+  for (int s = 0; s < seg; ++s) {
+    bool begins = false;
+    for (int r = s * 16; r < s * 16 + 16; ++r) begins = begins || since[r] == 0;
+    ch_in = begins ? seg_h[s][c] : fmaf(seg_p[s][c], ch_in, seg_h[s][c]);
+    cp_in = begins ? seg_p[s][c] : seg_p[s][c] * cp_in;
+  }
+#pragma unroll 4
+  for (int r = r_from; r < r_from + 16; ++r) {
+    if (r >= rows) break;
+    float hr = gates[r * GP + c], pr = gates[(RG_RM + r) * GP + c];
+    if (r < fresh) hr = fmaf(pr, ch_in, hr), pr *= cp_in;
+    const size_t at = (size_t)(t0 + r) * p.width + ch;
+    p.h[at] = hr;
+    p.prod[at] = pr;
+  }
+}
+
+// ---------------------------------------------------------------------------
+// rglru_chain: a thread per entry and channel
+// ---------------------------------------------------------------------------
+__global__ void __launch_bounds__(64) rglru_chain_kernel(const Rglru p) {
+  pdl_trigger();
+  pdl_wait();
+  const int entry = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
+  const int first = p.cu_tokens[entry], end = p.cu_tokens[entry + 1], slot = p.slots[entry];
+  if (c >= p.width || end <= first || slot < 0 || slot >= p.state_rows) return;
+  float* cell = p.state + (size_t)slot * p.width + c;
+  float s = *cell;
+  p.init[(size_t)entry * p.width + c] = s;
+  const int k_from = first / RG_RM, k_to = (end - 1) / RG_RM;
+  for (int k0 = k_from; k0 <= k_to; k0 += 16) {
+    float h[16], a[16];
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const bool has = k0 + j <= k_to;
+      const size_t at = (size_t)(has ? min((k0 + j + 1) * RG_RM, end) - 1 : first) * p.width + c;
+      h[j] = has ? p.h[at] : 0.f;
+      a[j] = has ? p.prod[at] : 1.f;
+    }
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      s = fmaf(a[j], s, h[j]);
+      if (k0 + j < k_to) p.carry[(size_t)(k0 + j + 1) * p.width + c] = s;
+    }
+  }
+  *cell = s;
+  // the last taps - 1 of (the state's inputs, the step's): a row is read before it is overwritten
+  const int back = p.taps - 1, count = end - first;
+  float* st = p.conv_state + (size_t)slot * back * p.width + c;
+  for (int k = 0; k < back; ++k) {
+    const int at = count + k;
+    st[(size_t)k * p.width] = at < back ? st[(size_t)at * p.width] : p.proj[(size_t)(first + at - back) * p.ld + p.x_off + c];
+  }
+}
+
+// ---------------------------------------------------------------------------
+// rglru_out: S and the output, V neighbouring channels a thread
+// ---------------------------------------------------------------------------
+template <typename TO, int V>
+__global__ void __launch_bounds__(256) rglru_out_kernel(const Rglru p) {
+  pdl_trigger();
+  pdl_wait();
+  const int t = blockIdx.x, c = (blockIdx.y * blockDim.x + threadIdx.x) * V;
+  if (c >= p.width) return;
+  const int entry = p.token_entry[t], tile = t / RG_RM;
+  const float* in = p.cu_tokens[entry] >= tile * RG_RM ? p.init + (size_t)entry * p.width : p.carry + (size_t)tile * p.width;
+  const size_t at = (size_t)t * p.width + c;
+  const float* yp = p.proj + (size_t)t * p.ld + p.y_off + c;
+  float h[V], a[V], s[V], y[V];
+  if constexpr (V == 4) load4(p.h + at, h), load4(p.prod + at, a), load4(in + c, s), load4(yp, y);
+  else h[0] = p.h[at], a[0] = p.prod[at], s[0] = in[c], y[0] = yp[0];
+#pragma unroll
+  for (int e = 0; e < V; ++e) h[e] = fmaf(a[e], s[e], h[e]) * rg_gelu(y[e]);
+  if constexpr (V == 4) store4((TO*)p.out + at, h);
+  else ((TO*)p.out)[at] = from_float<TO>(h[0]);
+}
+
+// ---------------------------------------------------------------------------
+// rglru_step
+// ---------------------------------------------------------------------------
+#define RG_SM 16            // entries of a tile
+
+template <int NC>
+static size_t rg_step_smem(int part) {
+  const size_t pitch = (size_t)(part + 15) / 16 * 16 + 8;
+  return sizeof(bf16) * (2 * NC + 2 * RG_SM) * pitch + sizeof(float) * 3 * RG_SM * (NC + 1);
+}
+
+template <typename TO, int NC>
+__global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* status) {
+  extern __shared__ __align__(16) unsigned char raw[];
+  cg::cluster_group cluster = cg::this_cluster();
+  constexpr int THREADS = 4 * NC, GP = NC + 1;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int n0 = blockIdx.x * NC, block = blockIdx.y, t0 = blockIdx.z * RG_SM;
+  const int part = p.part, k_all = (part + 15) / 16 * 16, pitch = k_all + 8, back = p.taps - 1;
+  const int rows = min(RG_SM, p.n_tokens - t0);
+  bf16* ws = reinterpret_cast<bf16*>(raw);            // [2 gates][NC][pitch]
+  bf16* hi = ws + 2 * NC * pitch;                     // [SM][pitch]: u of the whole part, rounded; then the remainders
+  float* us = reinterpret_cast<float*>(hi + 2 * RG_SM * pitch);      // [SM][GP]: u of the block's own channels
+  float* gates = us + RG_SM * GP;                     // [2][SM][GP]
+  pdl_trigger();
+  // the gate matrices are nobody's output: on their way before the kernels ahead have finished
+  rg_load_weight(ws, pitch, (const bf16*)p.wr + (size_t)block * part * part, part, n0, NC, 0, k_all);
+  rg_load_weight(ws + NC * pitch, pitch, (const bf16*)p.wi + (size_t)block * part * part, part, n0, NC, 0, k_all);
+  cp_commit();
+  for (int i = tid; i < 2 * RG_SM * pitch; i += THREADS) hi[i] = __float2bfloat16_rn(0.f);
+  pdl_wait();
+  cluster.sync();                                     // every block of the cluster is there, its tiles are zero
+  const int x0 = block * part, cols = min(NC, part - n0);
+  const int peers = (int)cluster.num_blocks();
+  for (int i = tid; i < RG_SM * NC; i += THREADS) {
+    const int r = i / NC, c = i - r * NC;
+    float u = 0.f;
+    if (r < rows && c < cols) {
+      const int ch = x0 + n0 + c, slot = p.slots[t0 + r];
+      const float x = p.proj[(size_t)(t0 + r) * p.ld + p.x_off + ch];
+      u = p.conv_b[ch];
+      if (slot >= 0 && slot < p.state_rows) {
+        // the oldest input leaves the history, the others move up
+        float* st = p.conv_state + (size_t)slot * back * p.width + ch;
+        for (int j = 0; j < back; ++j) {
+          const float v = st[(size_t)j * p.width];
+          u = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u);
+          if (j > 0) st[(size_t)(j - 1) * p.width] = v;
+        }
+        if (back > 0) st[(size_t)(back - 1) * p.width] = x;
+      } else {
+        atomicOr(status, FE_STATUS_BAD_PAGE);
+      }
+      u = fmaf(p.conv_w[(size_t)back * p.width + ch], x, u);
+    }
+    us[r * GP + c] = u;
+  }
+  __syncthreads();
+  // channels of a part in pairs: n0 is even
+  for (int i = tid; i < rows * (NC / 2); i += THREADS) {
+    const int r = i / (NC / 2), c = (i - r * (NC / 2)) * 2;
+    if (c >= cols) continue;
+    unsigned h, l;
+    split2(us[r * GP + c], us[r * GP + c + 1], h, l);       // past the last channel: zero
+    const int at = r * pitch + n0 + c;
+    for (int peer = 0; peer < peers; ++peer) {
+      bf16* dst = cluster.map_shared_rank(hi, peer);
+      *reinterpret_cast<unsigned*>(dst + at) = h;
+      *reinterpret_cast<unsigned*>(dst + RG_SM * pitch + at) = l;
+    }
+  }
+  cp_wait<0>();
+  __syncthreads();
+  cluster.sync();                                     // the whole part's u is in place
+  {
+    // a warp takes 16 channels of one gate
+    const int g = warp / (NC / 16), c0 = (warp - g * (NC / 16)) * 16;
+    float acc[2][4] = {};
+    for (int kk = 0; kk < k_all / 16; ++kk) {
+      unsigned ah[4], al[4], b0, b1, b2, b3;
+      const int a_at = (lane & 15) * pitch + kk * 16 + (lane >> 4) * 8;
+      ldsm4(ah[0], ah[1], ah[2], ah[3], hi + a_at);
+      ldsm4(al[0], al[1], al[2], al[3], hi + RG_SM * pitch + a_at);
+      ldsm4(b0, b1, b2, b3, ws + (g * NC + c0 + (lane >> 4) * 8 + (lane & 7)) * pitch + kk * 16 + ((lane >> 3) & 1) * 8);
+      mma16816(acc[0], ah, b0, b1);
+      mma16816(acc[1], ah, b2, b3);
+      mma16816(acc[0], al, b0, b1);
+      mma16816(acc[1], al, b2, b3);
+    }
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+#pragma unroll
+      for (int e = 0; e < 4; ++e)
+        gates[(g * RG_SM + (lane >> 2) + 8 * (e >> 1)) * GP + c0 + j * 8 + (lane & 3) * 2 + (e & 1)] = acc[j][e];
+  }
+  __syncthreads();
+  for (int i = tid; i < rows * NC; i += THREADS) {
+    const int r = i / NC, c = i - r * NC;
+    if (c >= cols) continue;
+    const int ch = x0 + n0 + c, slot = p.slots[t0 + r];
+    if (slot < 0 || slot >= p.state_rows) continue;
+    float a, scale;
+    rg_gates(gates[r * GP + c] + p.br[ch], gates[(RG_SM + r) * GP + c] + p.bi[ch], p.rate[ch], &a, &scale);
+    float* cell = p.state + (size_t)slot * p.width + ch;
+    const float s = fmaf(a, *cell, scale * us[r * GP + c]);
+    *cell = s;
+    ((TO*)p.out)[(size_t)(t0 + r) * p.width + ch] = from_float<TO>(s * rg_gelu(p.proj[(size_t)(t0 + r) * p.ld + p.y_off + ch]));
+  }
+}
+
+// ---------------------------------------------------------------------------
+// launchers
+// ---------------------------------------------------------------------------
+template <typename TO, int NC>
+static int rg_launch_step(const Rglru& p, int* status, cudaStream_t stream) {
+  const size_t smem = rg_step_smem<NC>(p.part);
+  if (smem > 48 * 1024) cudaFuncSetAttribute(rglru_step_kernel<TO, NC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const unsigned tiles = (unsigned)((p.part + NC - 1) / NC);
+  return fe_launch_dependent_shaped(rglru_step_kernel<TO, NC>, dim3(tiles, p.width / p.part, (p.n_tokens + RG_SM - 1) / RG_SM), dim3(4 * NC),
+                                    smem, stream, dim3(tiles, 1, 1), p, status);
+}
+
+// Channels of a block of rglru_step for parts of this size: at most 8 blocks share a part; 0: not taken.
+static int rg_step_cols(int part) {
+  if (part <= 8 * 32 && rg_step_smem<32>(part) <= 200 * 1024) return 32;
+  if (part <= 8 * 64 && rg_step_smem<64>(part) <= 200 * 1024) return 64;
+  return 0;
+}
+
+template <typename TW, int NC, int TAPS>
+static int rg_launch_gates(const Rglru& p, int* status, cudaStream_t stream) {
+  using Shape = RgShape<TW, NC>;
+  const size_t smem = Shape::bytes(p.taps);
+  if (smem > 220 * 1024) return FE_ERR_TOO_LARGE;
+  cudaFuncSetAttribute(rglru_gates_kernel<TW, NC, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const dim3 grid((p.part + NC - 1) / NC, p.width / p.part, (p.n_tokens + RG_RM - 1) / RG_RM);
+  return fe_launch_dependent(rglru_gates_kernel<TW, NC, TAPS>, grid, dim3(Shape::THREADS), smem, stream, p, (int)Shape::stages(p.taps), status);
+}
+
+// Whether a step in which every entry brings one token is one launch.
+FE_EXPORT int fe_rglru_one_launch(int part, int weight_dtype) { return weight_dtype == FE_DTYPE_BF16 && rg_step_cols(part) > 0; }
+
+// Floats of scratch a step of these sizes needs otherwise.
+FE_EXPORT long long fe_rglru_scratch(int tokens, int entries, int width) {
+  return (2LL * tokens + (tokens + RG_RM - 1) / RG_RM + 1 + entries) * ((width + 3) / 4 * 4);
+}
+
+FE_EXPORT int fe_rglru(const float* proj, long long ld, int y_off, int x_off, const float* conv_w, const float* conv_b, int taps,
+                       const void* wr, const void* wi, int weight_dtype, const float* br, const float* bi, const float* rate,
+                       float* state, float* conv_state, int state_rows, const int* slots, const int* cu_tokens,
+                       const int* token_entry, void* out, int out_dtype, int width, int part, int tokens, int entries, int max_new,
+                       float* scratch, int* status, cudaStream_t stream) {
+  if (tokens <= 0 || entries <= 0) return 0;
+  if (taps < 1 || width < 1 || part < 1 || width % part || width / part > 65535 || entries > 65535 || (taps > 1 && conv_state == nullptr))
+    return FE_ERR_BAD_SHAPE;
+  if ((tokens + RG_SM - 1) / RG_SM > 65535) return FE_ERR_TOO_LARGE;
+  if (((uintptr_t)wr | (uintptr_t)wi) & 15) return FE_ERR_BAD_ALIGN;
+  Rglru p{proj, ld, y_off, x_off, conv_w, conv_b, taps, wr, wi, br, bi, rate, state, conv_state, state_rows, slots, cu_tokens,
+          token_entry, width, part, tokens, entries, nullptr, nullptr, nullptr, nullptr, out};
+  int rc = FE_ERR_BAD_DTYPE;
+  if (max_new == 1 && tokens == entries && fe_rglru_one_launch(part, weight_dtype)) {
+    const int cols = rg_step_cols(part);
+    if (out_dtype == FE_DTYPE_BF16) rc = cols == 32 ? rg_launch_step<bf16, 32>(p, status, stream) : rg_launch_step<bf16, 64>(p, status, stream);
+    else if (out_dtype == FE_DTYPE_F32) rc = cols == 32 ? rg_launch_step<float, 32>(p, status, stream) : rg_launch_step<float, 64>(p, status, stream);
+    return rc ? rc : fe_last_error();
+  }
+  if (scratch == nullptr) return FE_ERR_BAD_SHAPE;
+  const size_t tiles = (size_t)(tokens + RG_RM - 1) / RG_RM, pitch = (size_t)width;
+  p.h = scratch;
+  p.prod = p.h + (size_t)tokens * pitch;
+  p.carry = p.prod + (size_t)tokens * pitch;
+  p.init = p.carry + (tiles + 1) * pitch;
+  if (weight_dtype == FE_DTYPE_BF16) rc = taps == 4 ? rg_launch_gates<bf16, 64, 4>(p, status, stream) : rg_launch_gates<bf16, 64, 0>(p, status, stream);
+  else if (weight_dtype == FE_DTYPE_F32) rc = taps == 4 ? rg_launch_gates<float, 64, 4>(p, status, stream) : rg_launch_gates<float, 64, 0>(p, status, stream);
+  if (rc) return rc;
+  rc = fe_launch_dependent(rglru_chain_kernel, dim3((width + 63) / 64, entries), dim3(64), 0, stream, p);
+  if (rc) return rc;
+  const bool wide = width % 4 == 0 && ld % 4 == 0 && y_off % 4 == 0 && (((uintptr_t)proj | (uintptr_t)scratch | (uintptr_t)out) & 15) == 0;
+  const int per = wide ? 4 : 1;
+  int threads = 32;
+  while (threads < 256 && threads * per < width) threads <<= 1;
+  const dim3 grid(tokens, (width + threads * per - 1) / (threads * per));
+  if (out_dtype == FE_DTYPE_BF16)
+    rc = wide ? fe_launch_dependent(rglru_out_kernel<bf16, 4>, grid, dim3(threads), 0, stream, p) : fe_launch_dependent(rglru_out_kernel<bf16, 1>, grid, dim3(threads), 0, stream, p);
+  else if (out_dtype == FE_DTYPE_F32)
+    rc = wide ? fe_launch_dependent(rglru_out_kernel<float, 4>, grid, dim3(threads), 0, stream, p) : fe_launch_dependent(rglru_out_kernel<float, 1>, grid, dim3(threads), 0, stream, p);
+  else
+    rc = FE_ERR_BAD_DTYPE;
+  return rc ? rc : fe_last_error();
+}

@@ -1,4 +1,4 @@
-// What the matrix-state recurrences share (wkv.cu, delta_rule.cu, matrix_memory.cu).
+// What the matrix-state recurrences share (wkv.cu, delta_rule.cu, matrix_memory.cu, retention.cu).
 //
 // Each of them keeps, per request and head, a 32-bit state S [dk, dv] that every token first
 // changes and reads; they differ in the change (the mechanism M below).  Two ways through an
@@ -36,7 +36,7 @@ struct StateRun {
   int heads, dk, dv, ds;
   const float* v;          // value of token t, head h, column c: v[t * v_ld + h * dv + c]
   long long v_ld;
-  const float* norm_w;     // weight of head h, column c: norm_w[h * norm_stride + c]
+  const float* norm_w;     // weight of head h, column c: norm_w[h * norm_stride + c]; null: none
   int norm_stride;
   const float* gate;       // act(gate[t * gate_ld + h * dv + c]) multiplies the normalised output
   long long gate_ld;
@@ -69,10 +69,10 @@ __device__ __forceinline__ void sr_store_row(const StateRun& p, const float* o, 
     ss = fmaf(x, x, ss);
   }
   const float inv = scale / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
-  const float* w = p.norm_w + (size_t)head * p.norm_stride;
+  const float* w = p.norm_w == nullptr ? nullptr : p.norm_w + (size_t)head * p.norm_stride;
   const float* g = p.gate + (size_t)token * p.gate_ld + (size_t)head * p.dv;
   TO* dst = (TO*)p.out + ((size_t)token * p.heads + head) * p.dv;
-  for (int c = lane; c < p.dv; c += 32) dst[c] = from_float<TO>(o[c] * inv * w[c] * sr_gate(g[c], p.gate_act));
+  for (int c = lane; c < p.dv; c += 32) dst[c] = from_float<TO>(o[c] * inv * (w == nullptr ? 1.f : w[c]) * sr_gate(g[c], p.gate_act));
 }
 
 // A mechanism M of the walk has
@@ -508,7 +508,7 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
 #pragma unroll
   for (int a = 0; a < 4; ++a) part[cg][row + a] = ss[a];
   __syncthreads();
-  const float* w = p.norm_w + (size_t)head * p.norm_stride;
+  const float* w = p.norm_w == nullptr ? nullptr : p.norm_w + (size_t)head * p.norm_stride;
   const bool wide = (dv & 3) == 0 && (p.norm_stride & 3) == 0 && (p.gate_ld & 3) == 0 &&
                     (((uintptr_t)p.norm_w | (uintptr_t)p.gate | (uintptr_t)p.out) & 15) == 0;
 #pragma unroll
@@ -526,15 +526,16 @@ __global__ void __launch_bounds__(256) state_out_kernel(const M m, const StateRu
       const int c = 64 * n + 4 * cg;
       if (wide) {
         if (c >= dv) continue;
-        float wv[4], gv[4], y[4];
-        load4(w + c, wv), load4(g + c, gv);
+        float wv[4] = {1.f, 1.f, 1.f, 1.f}, gv[4], y[4];
+        if (w != nullptr) load4(w + c, wv);
+        load4(g + c, gv);
 #pragma unroll
         for (int b = 0; b < 4; ++b) y[b] = acc[n][a][b] * inv * wv[b] * sr_gate(gv[b], p.gate_act);
         store4(dst + c, y);
       } else {
 #pragma unroll
         for (int b = 0; b < 4; ++b)
-          if (c + b < dv) dst[c + b] = from_float<TO>(acc[n][a][b] * inv * w[c + b] * sr_gate(g[c + b], p.gate_act));
+          if (c + b < dv) dst[c + b] = from_float<TO>(acc[n][a][b] * inv * (w == nullptr ? 1.f : w[c + b]) * sr_gate(g[c + b], p.gate_act));
       }
     }
   }

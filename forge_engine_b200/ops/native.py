@@ -62,7 +62,7 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_gated_rmsnorm": [p, p, i, i, p, p, i, i, i, f, p],
         "fe_qkv_prepare": [p, i, i, i, i, i, i, p, i, p, i, i, i, i, i, p, i, p, i, i, i, f, p, i, i, p, ll, ll, i,
                            p, p, i, p, i, i, i, p, p, i, p, p],
-        "fe_attention_general": [p, ll, ll, p, i, i, p, i, i, p, ll, ll, i, p, i, i, i, i, i, p, p, p, p, i, i, f,
+        "fe_attention_general": [p, ll, ll, p, i, i, p, i, i, p, ll, ll, i, p, i, i, i, i, i, p, p, p, p, i, i, i, f,
                                  i, f, f, i, i, ll, i, ll, p, ll, i, i, p, i, p, p],
         "fe_differential_combine": [p, p, i, ll, i, f, f, f, p],
         "fe_bias_xielu": [p, i, p, p, i, ll, i, f, f, p],
@@ -82,6 +82,7 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_linear_recurrence_chunks": [i, i],
         "fe_gemm_simt_batched": [p, i, p, i, p, i, i, i, i, i, ll, ll, ll, ll, ll, p],
         "fe_add_rmsnorm": [p, p, i, p, p, i, p, p, ll, i, i, f, i, p],
+        "fe_weighted_sum": [p, p, f, f, p, ll, p],
         "fe_norm_pair": [p, p, p, p, p, i, i, f, f, p],
         "fe_silu_mul": [p, p, i, i, i, i, p],
         "fe_qk_rope_cache": [p, i, p, p, f, p, p, i, p, p, p, p, p, i, i, i, i, i, i, i, i, p, p],
@@ -104,13 +105,19 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_delta_rule_scratch": [i, i, i, i, i, i],
         "fe_matrix_memory": [p, ll, i, i, i, i, i, i, p, p, f, f, p, f, p, p, p, i, p, p, p, i, i, i, i, i, i, i, p, p, p],
         "fe_matrix_memory_scratch": [i, i, i, i, i, i],
+        "fe_retention": [p, ll, i, i, i, i, f, p, p, i, i, p, f, p, i, p, p, p, i, i, i, i, i, i, i, p, p, p],
+        "fe_retention_scratch": [i, i, i, i, i, i],
+        "fe_rglru": [p, ll, i, i, p, p, i, p, p, i, p, p, p, p, p, i, p, p, p, p, i, i, i, i, i, i, p, p, p],
+        "fe_rglru_scratch": [i, i, i],
+        "fe_rglru_one_launch": [i, i],
         "fe_gemm_tc5_qkv_rope": [p, p, p, p, i, i, i, p, p, f, p, p, p, p, p, p, i, i, i, i, i, i, p, p],
     }
     for name, argtypes in signatures.items():
         fn = getattr(handle, name)
         fn.argtypes = argtypes
         fn.restype = c_int
-    for name in ("fe_gated_recurrence_scratch", "fe_wkv_scratch", "fe_delta_rule_scratch", "fe_matrix_memory_scratch"):
+    for name in ("fe_gated_recurrence_scratch", "fe_wkv_scratch", "fe_delta_rule_scratch", "fe_matrix_memory_scratch",
+                 "fe_retention_scratch", "fe_rglru_scratch"):
         getattr(handle, name).restype = ctypes.c_longlong
     handle.fe_uniform_host.argtypes = [c_ulonglong, c_ulonglong]
     handle.fe_uniform_host.restype = c_float
@@ -156,7 +163,8 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
                           max_new: int, num_q_heads: int, window: int | None, keep_first: int, scale: float,
                           gate: torch.Tensor | None, row_lo: int, status: torch.Tensor,
                           distance_bias: torch.Tensor | None = None, softcap: float | None = None,
-                          sinks: torch.Tensor | None = None, gate_per_element: bool = False) -> None:
+                          sinks: torch.Tensor | None = None, gate_per_element: bool = False,
+                          chunk: int | None = None) -> None:
     """The tcgen05 prefill attention for the entries of a step with more than ``row_lo`` rows
     (new tokens x heads per kv head): ``q`` [N, heads * D] and ``out`` [N, heads * D] bfloat16,
     caches [pages, kv_heads, page_size, D].  ``window`` with ``keep_first``: keys below it
@@ -165,7 +173,8 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     head's row is added to the score before the scale, so it holds the bias over the scale;
     ``softcap`` c (not together with the bias): scaled scores become c tanh(score / c);
     ``sinks`` (32-bit, per query head): exp(sink) joins the denominator once; ``gate_per_element``:
-    ``gate`` is [N, heads * D], one sigmoid gate per element of the output."""
+    ``gate`` is [N, heads * D], one sigmoid gate per element of the output; ``chunk`` (not together with
+    ``window``): a query sees the keys of its own chunk of that many positions only."""
     _dense(q, "q"), _dense(out, "out"), _dense(k_cache, "k_cache"), _dense(v_cache, "v_cache"), _dense(block_table, "block_table")
     num_pages, nkv, page_size, d = k_cache.shape
     n = q.shape[0]
@@ -178,7 +187,7 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     fn = getattr(handle, f"fe_attention_prefill_tc5_d{d}")
     if not getattr(fn, "_declared", False):
         p, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
-        fn.argtypes = [p, i, p, p, p, p, i, i, i, i, i, p, p, i, i, i, i, i, f, p, ll, i, i, p, i, f, p, p, p]
+        fn.argtypes = [p, i, p, p, p, p, i, i, i, i, i, p, p, i, i, i, i, i, i, f, p, ll, i, i, p, i, f, p, p, p]
         fn.restype = c_int
         fn._declared = True
     assert not (softcap and distance_bias is not None)
@@ -187,7 +196,7 @@ def attention_prefill_tc5(q: torch.Tensor, k_cache: torch.Tensor, v_cache: torch
     gate_stride = 0 if gate is None else (int(gate.stride(0)) if n > 1 else int(gate.shape[1]))
     check(fn(ptr(q), int(q.shape[1]), ptr(out), ptr(k_cache), ptr(v_cache), ptr(block_table), block_table.shape[1],
              page_size, num_pages, nkv, num_q_heads // nkv, ptr(cu_tokens), ptr(starts), int(n_entries), int(max_new), n,
-             int(window or 0), int(keep_first or 0), float(scale), ptr(gate), gate_stride, d if gate_per_element else 0, int(row_lo),
+             int(window or 0), int(chunk or 0), int(keep_first or 0), float(scale), ptr(gate), gate_stride, d if gate_per_element else 0, int(row_lo),
              ptr(distance_bias), 0 if distance_bias is None else int(distance_bias.shape[1]), float(softcap or 0.0),
              ptr(sinks), ptr(status), stream()), "attention_prefill_tc5")
 
@@ -802,7 +811,7 @@ def general_attention_lib(key_dim: int, value_dim: int, value_in_key: bool):
         suffix = f"{key_dim}_{value_dim}_{1 if value_in_key else 0}"
         run = getattr(handle, f"fe_attention_gmma_{suffix}")
         p, i, f, ll = c_void_p, c_int, c_float, ctypes.c_longlong
-        run.argtypes = [p, ll, ll, p, i, p, i, p, ll, ll, p, i, i, i, i, i, p, p, i, i, p, p, i, i, f, i, p,
+        run.argtypes = [p, ll, ll, p, i, p, i, p, ll, ll, p, i, i, i, i, i, p, p, i, i, p, p, i, i, i, f, i, p,
                         i, f, f, i, i, ll, i, ll, p, ll, i, i, i, p, p, p]
         run.restype = c_int
         space = getattr(handle, f"fe_attention_gmma_workspace_{suffix}")
@@ -821,7 +830,7 @@ def general_mma_takes(dtype, key_dim: int, value_dim: int) -> bool:
 
 
 def general_splits(entries: list, groups: int, kv_heads: int, window: int | None, slots: int = 296,
-                   keep_first: int = 0) -> int:
+                   keep_first: int = 0, chunk: int | None = None) -> int:
     """How many blocks share the keys of one row tile, for a step of ``entries`` ((slot,
     cached, new) each).  Only steps whose entries all fit one row tile (decoding, short
     portions) are split: enough blocks to fill the GPU once, each with at least two key
@@ -831,6 +840,8 @@ def general_splits(entries: list, groups: int, kv_heads: int, window: int | None
     longest = max(start + count for _, start, count in entries)
     if window:
         longest = min(longest, window + max(count for _, _, count in entries) + int(keep_first or 0))
+    if chunk:
+        longest = min(longest, chunk + max(count for _, _, count in entries))
     tiles = -(-longest // 64)
     wish = min(slots // max(1, len(entries) * kv_heads), tiles // 2, 32)
     return 1 if wish < 2 else 1 << (wish.bit_length() - 1)
@@ -865,6 +876,7 @@ def attention_general(
     distance_bias: torch.Tensor | None = None,
     sinks: torch.Tensor | None = None,
     gate_per_element: bool = False,
+    chunk: int | None = None,
 ) -> None:
     """Paged causal attention for any key and value size: scores, softmax and sums in 32-bit.
 
@@ -881,7 +893,8 @@ def attention_general(
     row (``v_cache`` may be ``k_cache`` itself: one cached vector that is key and value).
     ``slopes`` (per query head, 32-bit) takes slope * (query position - key position) off
     every score; ``distance_bias`` (32-bit [heads, L]) adds entry [head, min(distance, L - 1)] to
-    every (scaled, capped) score; ``window`` keeps the query's own and the window - 1 keys before it, and with
+    every (scaled, capped) score; ``window`` keeps the query's own and the window - 1 keys before it, ``chunk`` (not together with it)
+    the keys of the query's own chunk of that many positions, counted from position 0, and with
     ``keep_first`` the keys at positions below it as well.  ``softcap`` c: scores become
     c tanh(score / c); ``query_temperature`` (coef, every): a query at position p has its
     scores multiplied by 1 + coef ln(floor((p + 1) / every) + 1).  ``parts`` > 1: every head has
@@ -924,7 +937,7 @@ def attention_general(
             run(ptr(q), int(q_strides[0]), int(q_strides[1]), ptr(k_cache), k_row, ptr(v_cache), v_row, ptr(out),
                 int(o_strides[0]), int(o_strides[1]), ptr(block_table), block_table.shape[1], page_size, num_pages, nkv,
                 int(num_q_heads), ptr(cu_tokens), ptr(starts), int(n_entries), int(max_new), ptr(slopes),
-                ptr(distance_bias), dist_len, int(window or 0), float(scale), int(splits), ptr(workspace), *extras, int(row_hi), ptr(sinks), ptr(status), stream()),
+                ptr(distance_bias), dist_len, int(window or 0), int(chunk or 0), float(scale), int(splits), ptr(workspace), *extras, int(row_hi), ptr(sinks), ptr(status), stream()),
             "attention_general (tensor cores)",
         )
         if splits > 1:
@@ -937,7 +950,7 @@ def attention_general(
             ptr(q), int(q_strides[0]), int(q_strides[1]), ptr(k_cache), k_row, int(k_dim), ptr(v_cache), v_row,
             int(v_dim), ptr(out), int(o_strides[0]), int(o_strides[1]), code(q), ptr(block_table),
             block_table.shape[1], page_size, num_pages, nkv, int(num_q_heads), ptr(positions), ptr(token_entry),
-            ptr(slopes), ptr(distance_bias), dist_len, int(window or 0), float(scale), *extras, ptr(sinks), n, ptr(status), stream(),
+            ptr(slopes), ptr(distance_bias), dist_len, int(window or 0), int(chunk or 0), float(scale), *extras, ptr(sinks), n, ptr(status), stream(),
         ),
         "attention_general",
     )
@@ -1068,9 +1081,9 @@ def state_long_from() -> int:
     return int(lib().fe_state_long_from())
 
 
-def _state_checks(state: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor, norm: torch.Tensor, out: torch.Tensor) -> tuple:
+def _state_checks(state: torch.Tensor, slots: torch.Tensor, cu_tokens: torch.Tensor, norm: torch.Tensor | None, out: torch.Tensor) -> tuple:
     _dense(state, "state"), _dense(out, "out")
-    assert state.dtype == torch.float32 and norm.dtype == torch.float32 and norm.is_contiguous()
+    assert state.dtype == torch.float32 and (norm is None or (norm.dtype == torch.float32 and norm.is_contiguous()))
     assert slots.dtype == torch.int32 and cu_tokens.dtype == torch.int32
     rows, heads, dk, dv = state.shape
     assert out.shape[1] == heads * dv
@@ -1210,6 +1223,67 @@ def matrix_memory(proj: torch.Tensor, offsets: tuple, i_bias: torch.Tensor, f_bi
                                  ptr(cu_tokens), ptr(out), code(out), int(n_entries), heads, dk, dv, n, int(max_new), ptr(scratch),
                                  ptr(status), stream()), "matrix_memory")
     _count_chunked(max_new)
+
+
+def retention(proj: torch.Tensor, offsets: tuple, q_scale: float, decay: torch.Tensor, table: torch.Tensor | None, rot: int,
+              interleaved: bool, norm: torch.Tensor | None, eps: float, state: torch.Tensor, slots: torch.Tensor,
+              cu_tokens: torch.Tensor, out: torch.Tensor, n_entries: int, max_new: int, status: torch.Tensor) -> None:
+    """S = decay_h S + k v^T, o = S^T (q_scale q) over the tokens of every entry, from and to the 32-bit
+    state [rows, heads, dk, dv].  ``proj`` 32-bit [N, C] with q, k, v and the output gate from columns
+    ``offsets`` on; ``table`` (or None) [N, rot / 2, 2]: cosine and sine by which the leading ``rot``
+    elements of q and k are rotated first (only for steps without entries of ``state_long_from`` tokens or
+    more: there they come rotated).  ``out`` [N, heads * dv] gets o divided by its root mean square per
+    head, times ``norm`` [dv] (or None) and silu(gate)."""
+    rows, heads, dk, dv = _state_checks(state, slots, cu_tokens, norm, out)
+    q_off, k_off, v_off, g_off = (int(o) for o in offsets)
+    n = int(out.shape[0])
+    ld = _columns(proj, max(q_off + heads * dk, k_off + heads * dk, v_off + heads * dv, g_off + heads * dv))
+    assert decay.dtype == torch.float32 and decay.is_contiguous() and decay.numel() == heads and (norm is None or norm.numel() == dv)
+    assert table is None or (table.dtype == torch.float32 and table.is_contiguous() and table.shape == (n, rot // 2, 2))
+    scratch = _state_scratch(out.device, int(lib().fe_retention_scratch(n, int(n_entries), heads, dk, dv, int(max_new))))
+    check(lib().fe_retention(ptr(proj), ld, q_off, k_off, v_off, g_off, float(q_scale), ptr(decay), ptr(table), int(rot),
+                             1 if interleaved else 0, ptr(norm), float(eps), ptr(state), rows, ptr(slots), ptr(cu_tokens), ptr(out),
+                             code(out), int(n_entries), heads, dk, dv, n, int(max_new), ptr(scratch), ptr(status), stream()), "retention")
+    _count_chunked(max_new)
+
+
+def rglru(proj: torch.Tensor, y_off: int, x_off: int, conv: torch.Tensor, conv_bias: torch.Tensor, w_r: torch.Tensor,
+          w_i: torch.Tensor, b_r: torch.Tensor, b_i: torch.Tensor, rate: torch.Tensor, state: torch.Tensor,
+          conv_state: torch.Tensor | None, slots: torch.Tensor, cu_tokens: torch.Tensor, token_entry: torch.Tensor,
+          out: torch.Tensor, n_entries: int, max_new: int, status: torch.Tensor) -> None:
+    """out_t = S_t gelu_tanh(y_t) over the tokens of every entry, S_t = a S_(t-1) + sqrt(1 - a^2) i u_t per
+    channel from and to the 32-bit ``state`` [rows, width]; u = conv(x) + conv_bias, a causal convolution over
+    time (``conv`` [taps, width], the last tap weighing the token itself; ``conv_state`` [rows, taps - 1,
+    width]: its last inputs); r, i = sigmoid(W u + b) per part of the channels (``w_r``, ``w_i`` [blocks, part,
+    part]), log a = ``rate`` r.  y and x: 32-bit columns of ``proj`` [N, C] from ``y_off``, ``x_off`` on."""
+    rows, width = state.shape
+    taps, n = int(conv.shape[0]), int(out.shape[0])
+    blocks, part = int(w_r.shape[0]), int(w_r.shape[1])
+    for name, t in (("conv", conv), ("conv_bias", conv_bias), ("b_r", b_r), ("b_i", b_i), ("rate", rate), ("state", state)):
+        _dense(t, name)
+        assert t.dtype == torch.float32, name
+    _dense(w_r, "w_r"), _dense(w_i, "w_i"), _dense(out, "out")
+    assert w_r.shape == w_i.shape == (blocks, part, part) and w_r.dtype == w_i.dtype and blocks * part == width
+    assert conv.shape == (taps, width) and conv_bias.numel() == b_r.numel() == b_i.numel() == rate.numel() == width
+    assert out.shape == (n, width) and slots.dtype == cu_tokens.dtype == token_entry.dtype == torch.int32
+    assert taps == 1 or (conv_state.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.shape == (rows, taps - 1, width))
+    once = max_new == 1 and n == n_entries and bool(lib().fe_rglru_one_launch(part, code(w_r)))
+    scratch = None if once else _state_scratch(out.device, int(lib().fe_rglru_scratch(n, int(n_entries), width)))
+    check(lib().fe_rglru(ptr(proj), _columns(proj, max(y_off, x_off) + width), int(y_off), int(x_off), ptr(conv), ptr(conv_bias), taps,
+                         ptr(w_r), ptr(w_i), code(w_r), ptr(b_r), ptr(b_i), ptr(rate), ptr(state), ptr(conv_state), rows, ptr(slots),
+                         ptr(cu_tokens), ptr(token_entry), ptr(out), code(out), width, part, n, int(n_entries), int(max_new),
+                         ptr(scratch), ptr(status), stream()), "rglru")
+    if not once:
+        global LAUNCHES
+        LAUNCHES += 2
+
+
+def weighted_sum(a: torch.Tensor, b: torch.Tensor, scale_a: float, scale_b: float, out: torch.Tensor) -> None:
+    """out = scale_a * a + scale_b * b, 32-bit."""
+    for name, t in (("a", a), ("b", b), ("out", out)):
+        _dense(t, name)
+        assert t.dtype == torch.float32 and t.shape == out.shape, name
+    check(lib().fe_weighted_sum(ptr(a), ptr(b), float(scale_a), float(scale_b), ptr(out), int(out.numel()), stream()), "weighted_sum")
 
 
 def silu_mul(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0) -> None:

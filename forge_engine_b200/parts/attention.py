@@ -134,13 +134,15 @@ class GQAttention(Mixer):
         """Whether the layer needs what only the general kernels do: values of another size
         than keys, q and k normalised over the whole projection, a bias on the distance, kept
         first tokens, capped scores, a query temperature, a gate per head or per element, sinks, two
-        maps per head, q and k normalised without a weight or after the rotation."""
+        maps per head, q and k normalised without a weight or after the rotation, keys of the query's own
+        chunk only, neighbours rotated."""
         return (getattr(spec, "v_head_dim", None) not in (None, spec.head_dim)
                 or (spec.qk_norm and getattr(spec, "qk_norm_scope", "head") == "whole")
                 or getattr(spec, "distance_bias_base", None) is not None
                 or getattr(spec, "distance_bias_table", None) is not None or not getattr(spec, "kv_projection", True)
                 or bool(getattr(spec, "keep_first", 0)) or getattr(spec, "softcap", None) is not None
                 or getattr(spec, "query_temperature", None) is not None or bool(getattr(spec, "head_gate", False))
+                or getattr(spec, "chunk", None) is not None or bool(getattr(spec.position, "interleaved", False))
                 or bool(getattr(spec, "sink", False)) or bool(getattr(spec, "output_gate", False))
                 or getattr(spec, "differential", None) is not None
                 or (spec.qk_norm and (not getattr(spec, "qk_norm_weight", True) or getattr(spec, "qk_norm_after_rotation", False))))
@@ -153,6 +155,9 @@ class GQAttention(Mixer):
             )
         if spec.num_heads % spec.num_kv_heads:
             raise UnsupportedShapeError("num_heads must be a multiple of num_kv_heads")
+        self.chunk = getattr(spec, "chunk", None) or None
+        if self.chunk is not None and spec.window is not None:
+            raise ConfigError("a layer sees a window or its own chunk, not both")
         if getattr(spec, "qk_norm_scope", "head") not in ("head", "whole"):
             raise ConfigError(f"qk_norm_scope={spec.qk_norm_scope!r}; known: head, whole")
         self.spec = spec
@@ -194,9 +199,9 @@ class GQAttention(Mixer):
             rows.append(self.nq * self.dv)
             names.append(name("gate_proj.weight"))
         if spec.bias:
+            bias = fused_rows(weights, [name("q_proj.bias"), name("k_proj.bias"), name("v_proj.bias")], rows[:3])
             if self.head_gate:
-                raise ConfigError("a gate per head together with biases is not implemented")
-            bias = fused_rows(weights, [name("q_proj.bias"), name("k_proj.bias"), name("v_proj.bias")], rows)
+                bias = torch.cat([bias, bias.new_zeros(self.nq)])      # the gates' logits have none
         # q, k and v are looked up one at a time and copied into the fused tensor
         self.qkv_proj = Linear(fused_rows(weights, names, rows), bias, status=ctx.status)
         self.diff_lambda = None
@@ -229,7 +234,7 @@ class GQAttention(Mixer):
             self.distance_bias_unscaled = (self.distance_bias.double() / float(spec.scale)).float().contiguous()
         self._slots = None
         self.plan_key = ("gqa_attention", self.nq, self.nkv, self.d, spec.window) + (
-            ("general", self.dv, self.parts, self.keep_first) if self.general else ())
+            ("general", self.dv, self.parts, self.keep_first, self.chunk) if self.general else ())
         self.last_splits = None   # what the last step's decode entries ran with (0: balanced kernel)
 
     @staticmethod
@@ -299,7 +304,7 @@ class GQAttention(Mixer):
     def cache_needs(self) -> CacheNeeds:
         key = self.parts * self.d          # a differential layer caches both keys of a head in one row
         return CacheNeeds(kv=PagedKVSpec(self.nkv, key, self.spec.window, None if self.dv == key else self.dv,
-                                         self.keep_first))
+                                         self.keep_first, getattr(self.spec, "chunk", None)))
 
     def decode_slots(self) -> int:
         """Blocks of the decode kernels this device holds at once: what the balanced kernel
@@ -393,7 +398,7 @@ class GQAttention(Mixer):
                 native.attention_prefill_tc5(q, k_cache, v_cache, out, table, batch.cu_tokens, batch.starts, batch.n_entries,
                                              batch.max_new, nq, self.spec.window, self.keep_first, self.spec.scale, gate,
                                              SHORT_ENTRY_ROWS, self.ctx.status, distance_bias=self.distance_bias_unscaled,
-                                             softcap=self.softcap, sinks=self.sinks, gate_per_element=self.output_gate)
+                                             softcap=self.softcap, sinks=self.sinks, gate_per_element=self.output_gate, chunk=self.chunk)
             if short_entries:
                 native.attention_general(q, (nq * d, d), k_cache, self.d, v_cache, dv, out, (nq * parts * dv, parts * dv), table,
                                          batch.positions, batch.token_entry, nq, self.slopes, self.spec.window,
@@ -404,7 +409,7 @@ class GQAttention(Mixer):
                                          part_strides=(self.d, self.d, dv) if parts > 1 else (0, 0, 0),
                                          gate=gate, row_hi=SHORT_ENTRY_ROWS if long_entries else 0,
                                          distance_bias=self.distance_bias, sinks=self.sinks,
-                                         gate_per_element=self.output_gate)
+                                         gate_per_element=self.output_gate, chunk=self.chunk)
             if parts > 1:
                 maps = out
                 out = torch.empty((n, nq * dv), dtype=k_cache.dtype, device=x.device)
@@ -463,7 +468,7 @@ class GQAttention(Mixer):
 
     def _prefill_tc5(self, page_size: int) -> bool:
         """Whether prompt portions of this (general) layer run on the tcgen05 prefill kernel:
-        a plain softmax over one map per head (a window, kept first tokens, gates, sinks and either a
+        a plain softmax over one map per head (a window or chunks, kept first tokens, gates, sinks and either a
         bias by distance or capped scores it has), keys and values of 64 or 128."""
         return (self.parts == 1 and self.slopes is None and (self.softcap is None or self.distance_bias is None)
                 and self.query_temperature is None
@@ -508,7 +513,7 @@ class GQAttention(Mixer):
                 splits = 1
                 if short and native.general_mma_takes(self.ctx.dtype, self.d, self.dv):
                     splits = native.general_splits(short, groups, self.nkv * self.parts, self.spec.window,
-                                                   keep_first=self.keep_first)
+                                                   keep_first=self.keep_first, chunk=self.chunk)
                 plans[self.plan_key] = (splits, len(short) < len(entries), bool(short))
             return
         if self.ctx.dtype != torch.bfloat16 or self.plan_key in plans:

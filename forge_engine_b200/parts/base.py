@@ -18,6 +18,8 @@ from __future__ import annotations
 
 from dataclasses import dataclass, field
 
+import torch
+
 from ..cache.manager import CacheNeeds
 from ..errors import ConfigError
 
@@ -138,12 +140,24 @@ class Mixer(Part):
 
 class FeedForward(Part):
     """Token-wise ``forward(x) -> update`` [N, hidden].  A feed-forward with ``takes_add`` also takes
-    ``forward(x, add=...)``: a 32-bit [N, hidden] that is added to its update."""
+    ``forward(x, add=...)``: a 32-bit [N, hidden] that is added to its update; one with ``gives_sums``
+    ``forward(x, out_dtype=...)``: the dtype of the update."""
 
     takes_add = False
+    gives_sums = False
 
     def forward(self, x):
         raise NotImplementedError
+
+
+def summed_update(ctx: BuildContext, mixer, u, batch, cache: CacheView):
+    """A mixer's update, as the 32-bit sums of its output projection where it has one."""
+    attend, o_proj = getattr(mixer, "attend", None), getattr(mixer, "o_proj", None)
+    if attend is None or o_proj is None:
+        return mixer.forward(u, batch, cache)
+    heads = attend(u, batch, cache)
+    with ctx.section("mixer.o_proj"):
+        return o_proj(heads, out_dtype=torch.float32)
 
 
 _PARTS: dict[str, type] = {}

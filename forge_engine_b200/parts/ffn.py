@@ -21,6 +21,7 @@ ACTIVATIONS = {"silu": native.ACT_SILU, "gelu_tanh": native.ACT_GELU_TANH, "clam
 
 class GatedMLP(FeedForward):
     graph_safe = True
+    gives_sums = True
 
     def __init__(self, spec, weights: dict, ctx: BuildContext) -> None:
         if spec.activation not in ACTIVATIONS:
@@ -61,7 +62,8 @@ class GatedMLP(FeedForward):
             return False
         return self.down.add_into(self.gate_up.silu_mul(x, self.block, self.activation, self.limit, self.slope), residual)
 
-    def forward(self, x):
+    def forward(self, x, out_dtype=None):
+        """``out_dtype``: of the update (the 32-bit sums of the down projection, say); None: as ``x``."""
         act = self.gate_up.silu_mul(x, self.block, self.activation, self.limit, self.slope) if self.block else None
         if act is None:
             act = torch.empty((x.shape[0], self.inter), dtype=x.dtype, device=x.device)
@@ -71,7 +73,7 @@ class GatedMLP(FeedForward):
                 # the activation is taken of the 32-bit sums of the projection, not of their rounding
                 native.act_mul(self.gate_up(x, out_dtype=torch.float32), act, self.activation, self.block,
                                self.limit, self.slope)
-        return self.down(act)
+        return self.down(act, out_dtype=out_dtype)
 
 
 UNARY = {"gelu_tanh": native.UNARY_GELU_TANH, "relu2": native.UNARY_RELU2}

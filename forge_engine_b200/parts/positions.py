@@ -36,10 +36,13 @@ class RotaryEncoding(PositionEncoding):
         self.scaling = getattr(spec, "scaling", None)
         self.exact = bool(getattr(spec, "exact_frequencies", False))
         self.yarn = getattr(spec, "yarn", None)
+        self.divisor = float(getattr(spec, "frequency_divisor", 1.0))
         self.amplitude = 1.0         # what cosine and sine are multiplied by
-        if self.scaling is not None or self.exact or self.yarn is not None:
+        if self.divisor <= 0:
+            raise ValueError("frequencies are divided by a positive number")
+        if self.scaling is not None or self.exact or self.yarn is not None or self.divisor != 1.0:
             exponent = torch.arange(0, spec.rotary_dim, 2, dtype=torch.float64) / spec.rotary_dim
-            freq = self.theta ** -exponent
+            freq = self.theta ** -exponent / self.divisor
             if self.scaling is not None:
                 freq = self.stretch(freq, self.scaling)
             if self.yarn is not None:
@@ -79,7 +82,7 @@ class RotaryEncoding(PositionEncoding):
     def table(self, batch) -> torch.Tensor:
         """[tokens, rotary_dim / 2, 2] (cos, sin) of this step's angles; worked out by the
         first layer that asks and shared through the batch."""
-        key = ("rotary", self.theta, self.rotary_dim, self.interleaved, self.scaling, self.exact, self.yarn)
+        key = ("rotary", self.theta, self.rotary_dim, self.interleaved, self.scaling, self.exact, self.yarn, self.divisor)
         table = batch.shared.get(key)
         if table is None:
             table = torch.empty((batch.n_tokens, self.rotary_dim // 2, 2), dtype=torch.float32, device=self.inv_freq.device)

@@ -1,7 +1,7 @@
 """Two mixers that read the same input, joined as half the sum of their normalised outputs:
 y = 1/2 (left / rms(left) * w_left + right / rms(right) * w_right), the root mean squares over the
-model's width.  The mixers' last projections leave 32-bit sums; both norms and the sum are one
-kernel.  What the two keep between steps is kept side by side: one of them may keep keys and values,
+model's width, or (``scales``) as a weighted sum a left + b right.  The mixers' last projections
+leave 32-bit sums; joining them is one kernel.  What the two keep between steps is kept side by side: one of them may keep keys and values,
 one may keep states."""
 
 from __future__ import annotations
@@ -14,7 +14,7 @@ from ..cache.manager import CacheNeeds
 from ..config.specs import local_name
 from ..errors import ConfigError
 from ..ops import native
-from .base import BuildContext, CacheView, Mixer, WeightInfo, build_part, part_class, register_part
+from .base import BuildContext, CacheView, Mixer, WeightInfo, build_part, part_class, register_part, summed_update
 
 SIDES = ("left", "right")
 
@@ -39,7 +39,8 @@ class SideBySide(Mixer):
     def __init__(self, spec, weights: dict, ctx: BuildContext) -> None:
         self.spec, self.ctx = spec, ctx
         self.sides = [build_part(getattr(spec, side), _Side(weights, side), ctx) for side in SIDES]
-        self.norms = [weights[local_name(spec, f"{side}.out")].to(device=ctx.device, dtype=torch.float32).contiguous() for side in SIDES]
+        self.scales = None if getattr(spec, "scales", None) is None else tuple(float(s) for s in spec.scales)
+        self.norms = [] if self.scales is not None else [weights[local_name(spec, f"{side}.out")].to(device=ctx.device, dtype=torch.float32).contiguous() for side in SIDES]
         self.cache_needs()      # refuses two mixers that want the same place
 
     @classmethod
@@ -48,7 +49,8 @@ class SideBySide(Mixer):
         for side in SIDES:
             inner = getattr(spec, side)
             shapes.update({f"{side}.{name}": info for name, info in part_class(inner).weight_shapes(inner).items()})
-            shapes[local_name(spec, f"{side}.out")] = WeightInfo((spec.hidden_size,), "norm")
+            if getattr(spec, "scales", None) is None:
+                shapes[local_name(spec, f"{side}.out")] = WeightInfo((spec.hidden_size,), "norm")
         return shapes
 
     @property
@@ -76,17 +78,15 @@ class SideBySide(Mixer):
 
     def _update(self, side, x, batch, cache: CacheView):
         """A side's update, as the 32-bit sums of its output projection where it has one."""
-        attend, o_proj = getattr(side, "attend", None), getattr(side, "o_proj", None)
-        if attend is None or o_proj is None:
-            return side.forward(x, batch, cache).float()
-        heads = attend(x, batch, cache)
-        with self.ctx.section("mixer.o_proj"):
-            return o_proj(heads, out_dtype=torch.float32)
+        return summed_update(self.ctx, side, x, batch, cache).float()
 
     def forward(self, x, batch, cache: CacheView):
         left, right = (self._update(side, x, batch, cache) for side in self.sides)
         out = torch.empty_like(left)
         with self.ctx.section("mixer.join"):
+            if self.scales is not None:
+                native.weighted_sum(left, right, self.scales[0], self.scales[1], out)
+                return out
             native.norm_pair(left, right, self.norms[0], self.norms[1], out, self.spec.norm_eps, 0.5)
         return out
 
