@@ -538,8 +538,8 @@ def design_compare(args) -> int:
     of `--layers` (4) layers of one kind: the Qwen3 layer, the Zofadra attention, latent
     attention and linear-recurrence layers, the Tekilorn differential, gated window and
     routed layers, the Zabutar gated-recurrence, biased-attention and routed layers and the Nuvivik
-    attention, latent and routed layers and the Lofuvik time-mixing, delta-rule and side-by-side
-    layers at the same sizes, plus a model of each design that mixes its layers.
+    attention, latent and routed layers, the Lofuvik time-mixing, delta-rule and side-by-side
+    layers and the Lozezen recurrent-unit, window and side-by-side layers at the same sizes, plus a model of each design that mixes its layers.
     One JSON line per model: tokens/s, ms per step, the median device time of every part of a
     step (CUDA events round each part, in a second runner) and, for the token-mixing kernel,
     its share of the measured peaks (prefill: its flops over the library GEMM's burst rate;
@@ -688,6 +688,29 @@ def design_compare(args) -> int:
             "lofuvik-routed": lofuvik([l_delta] * layers),
             "lofuvik-mixed": lofuvik([l_wkv, l_delta, l_parallel, l_wkv], loop={"start": 1, "stop": 3, "times": 2}),
         })
+        # Lozezen at the same sizes: the gated linear recurrent unit as wide as the stream in parts of 256
+        # (4 taps), biased window attention with half the head rotated at Qwen3's head sizes, and chunked
+        # attention (chunks as long as the windows) beside retention with the other recurrences' states;
+        # the dense feed-forward of ff.
+        z_unit = {"type": "rglru", "mlp": mlp, "mixer": {"width": W, "blocks": W // 256, "conv": 4}}
+        z_window = {"type": "attention", "mlp": mlp, "mixer": {
+            "heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window},
+            "rot": {"base": 1e6, "dims": D // 2, "scaling": {"factor": 2.0}}}}
+        z_parallel = {"type": "parallel", "mlp": mlp, "mixer": {
+            "left_scale": 0.5, "right_scale": 0.5,
+            "left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window}},
+            "right": dict(rec, heads=H, rot={"base": 1e6, "dims": rec["dim"]}, decay=[1.0 - 2.0 ** (-5 - 3 * h / H) for h in range(H)])}}
+
+        def lozezen(kinds):
+            return {"architecture": "Lozezen", "vocab": vocab, "width": W, "norm": {"eps": 1e-5}, "embedding": {"scale": W ** 0.5},
+                    "layers": kinds}
+
+        models.update({
+            "lozezen-rglru": lozezen([z_unit] * layers),
+            "lozezen-attention": lozezen([z_window] * layers),
+            "lozezen-parallel": lozezen([z_parallel] * layers),
+            "lozezen-mixed": lozezen([z_unit, bare(z_unit), z_window, z_parallel]),
+        })
         if args.design_models:
             wanted = [w for w in args.design_models.split(",") if w]
             models = {name: raw for name, raw in models.items() if any(name.startswith(w) for w in wanted)}
@@ -714,7 +737,14 @@ def design_compare(args) -> int:
         mixer_cost["lofuvik-delta"] = mixer_cost["lofuvik-routed"] = (
             8 * H * rec["dim"] * rec["vdim"] * CONTEXT, mixer_cost["zofadra-recurrence"][1])
         mixer_cost["lofuvik-parallel"] = mixer_cost["qwen3"]
-        second_cost = {"lofuvik-parallel": ("mixer.recurrence", *mixer_cost["zofadra-recurrence"])}
+        mixer_cost["lozezen-attention"] = mixer_cost["qwen3-window"]
+        # every query sees its own chunk up to itself; the token decoded here is one of a chunk's first
+        mixer_cost["lozezen-parallel"] = (4 * H * D * sum(i % window + 1 for i in range(CONTEXT)), batch * (CONTEXT % window + 24) * G * 2 * D * 2)
+        # both gates' products; in decoding their matrices, the states and the convolution's inputs
+        mixer_cost["lozezen-rglru"] = (4 * W * 256 * CONTEXT, 2 * W * 256 * 2 + batch * W * 4 * (2 + 2 * 3 + 2) + batch * W * 2)
+        # what a prompt must move: x and y (32-bit) in, the heads (bfloat16) out
+        prefill_bytes = {"lozezen-rglru": CONTEXT * W * (4 + 4 + 2)}
+        second_cost = {"lozezen-parallel": ("mixer.recurrence", *mixer_cost["zofadra-recurrence"]), "lofuvik-parallel": ("mixer.recurrence", *mixer_cost["zofadra-recurrence"])}
         mixer_part = {"qwen3": "mixer.attention", "qwen3-window": "mixer.attention", "zofadra-attention": "mixer.attention",
                       "zofadra-latent": "mixer.attention", "zofadra-recurrence": "mixer.recurrence",
                       "tekilorn-differential": "mixer.attention", "tekilorn-window": "mixer.attention",
@@ -723,7 +753,8 @@ def design_compare(args) -> int:
                       "nuvivik-attention": "mixer.attention", "nuvivik-routed": "mixer.attention",
                       "nuvivik-latent": "mixer.attention", "lofuvik-wkv": "mixer.recurrence",
                       "lofuvik-delta": "mixer.recurrence", "lofuvik-routed": "mixer.recurrence",
-                      "lofuvik-parallel": "mixer.attention"}
+                      "lofuvik-parallel": "mixer.attention", "lozezen-rglru": "mixer.recurrence",
+                      "lozezen-attention": "mixer.attention", "lozezen-parallel": "mixer.attention"}
         for name, raw in models.items():
             n_layers = len(raw["layers"]) if "layers" in raw else raw["num_hidden_layers"]
             pages = batch * (-(-(CONTEXT + 64) // PAGE) + 1) + -(-CONTEXT // PAGE) + 8
@@ -801,6 +832,9 @@ def design_compare(args) -> int:
                     "decode_ms": result["decode_parts_ms"].get(part),
                     "decode_frac_of_copy_peak": round(moved / (result["decode_parts_ms"][part] * 1e-3) / (hbm_gbs * 1e9), 4),
                 }
+                if key == "mixer_kernel" and name in prefill_bytes:
+                    result[key]["prefill_frac_of_copy_peak"] = round(
+                        prefill_bytes[name] / (result["prefill_parts_ms"][part] * 1e-3) / (hbm_gbs * 1e9), 4)
             plain.model.ctx.timer = None
             print(json.dumps(result), flush=True)
             del plain, timed
