@@ -3,11 +3,12 @@
 // a bias on the distance between query and key, queries and outputs laid out with any
 // strides.  Two kernels:
 //
-// qkv_prepare - one block per token and side (queries; keys and values): reads the token's projected q, k (and v), normalises
-//   (per head over the head's leading elements, or over the whole projection at once, or not
-//   at all), rotates a stretch of every head by the step's cosine/sine table, stores the
-//   queries where the attention kernel wants them and k, v into their cache pages.
-//   Everything between load and store is 32-bit.
+// qkv_prepare - reads a token's projected q, k (and v), adds the projection's bias if there is one,
+//   normalises (per head over the head's leading elements, or over the whole projection at once, or
+//   not at all), rotates a stretch of every head by the step's cosine/sine table, stores the
+//   queries where the attention kernel wants them and k, v into their cache pages.  A warp takes a
+//   head of a token; with a norm over the whole projection one block takes a token and side (queries;
+//   keys and values).  Everything between load and store is 32-bit.
 //
 // attention_general - one block per (token, kv head, group of up to 8 query heads that
 //   share the kv head).  Keys [lo, pos] are cut into chunks of 32 from lo; warp w takes
@@ -39,6 +40,7 @@ struct PrepSide {
   int norm_dims;       // PREP_NORM_HEAD: leading elements of a head that are normalised
   const float* norm_w;
   int rot_off;         // first rotated element of a head; negative: this side is not rotated
+  const float* bias;   // or null: [heads * dim], added to what is read
 };
 
 __device__ __forceinline__ void prep_norm_rotate(float* row, const PrepSide& s, float eps, const float2* angles,
@@ -95,7 +97,7 @@ __device__ __forceinline__ void prep_norm_rotate(float* row, const PrepSide& s, 
 
 template <typename TI, typename TC>
 __global__ void __launch_bounds__(256)
-qkv_prepare_kernel(PrepSide q, PrepSide k, const TI* __restrict__ v_in, int v_in_stride, int v_dim, float eps,
+qkv_prepare_kernel(PrepSide q, PrepSide k, const TI* __restrict__ v_in, int v_in_stride, int v_dim, const float* __restrict__ v_bias, float eps,
                    const float2* __restrict__ table, int rot_dims, int interleaved, TC* __restrict__ q_out,
                    long long q_out_token_stride, long long q_out_head_stride, int q_out_dim_offset,
                    TC* __restrict__ k_cache, TC* __restrict__ v_cache, const int* __restrict__ block_table,
@@ -117,14 +119,14 @@ qkv_prepare_kernel(PrepSide q, PrepSide k, const TI* __restrict__ v_in, int v_in
     const TI* src = (const TI*)q.in + (size_t)token * q.in_stride;
     for (int i = threadIdx.x; i < q_total; i += blockDim.x) {
       const int h = i / q.dim;
-      q_row[i] = to_float(src[(size_t)h * q.head_stride + (i - h * q.dim)]);
+      q_row[i] = to_float(src[(size_t)h * q.head_stride + (i - h * q.dim)]) + (q.bias ? q.bias[i] : 0.f);
     }
   }
   if (do_k) {
     const TI* src = (const TI*)k.in + (size_t)token * k.in_stride;
     for (int i = threadIdx.x; i < k_total; i += blockDim.x) {
       const int h = i / k.dim;
-      k_row[i] = to_float(src[(size_t)h * k.head_stride + (i - h * k.dim)]);
+      k_row[i] = to_float(src[(size_t)h * k.head_stride + (i - h * k.dim)]) + (k.bias ? k.bias[i] : 0.f);
     }
   }
   __syncthreads();
@@ -158,15 +160,231 @@ qkv_prepare_kernel(PrepSide q, PrepSide k, const TI* __restrict__ v_in, int v_in
     const TI* src = v_in + (size_t)token * v_in_stride;
     for (int i = threadIdx.x; i < k.heads * v_dim; i += blockDim.x) {
       const int h = i / v_dim, d = i - h * v_dim;
-      v_cache[(((size_t)page * k.heads + h) * page_size + slot) * v_dim + d] = from_float<TC>(to_float(src[i]));
+      v_cache[(((size_t)page * k.heads + h) * page_size + slot) * v_dim + d] = from_float<TC>(to_float(src[i]) + (v_bias ? v_bias[i] : 0.f));
     }
   }
+}
+
+// The same without a norm over the whole projection: a warp per head of a token, `V` neighbouring
+// elements a lane at a time.
+#define PREP_WARPS 8
+
+template <int V> __device__ __forceinline__ void prep_load(const float* p, float* v) { if constexpr (V == 4) load4(p, v); else v[0] = p[0]; }
+template <int V> __device__ __forceinline__ void prep_load(const bf16* p, float* v) { if constexpr (V == 4) load4(p, v); else v[0] = to_float(p[0]); }
+template <int V> __device__ __forceinline__ void prep_store(float* p, const float* v) { if constexpr (V == 4) store4(p, v); else p[0] = v[0]; }
+template <int V> __device__ __forceinline__ void prep_store(bf16* p, const float* v) { if constexpr (V == 4) store4(p, v); else p[0] = from_float<bf16>(v[0]); }
+
+template <typename TI, typename TC, int V>
+__global__ void __launch_bounds__(32 * PREP_WARPS)
+qkv_prepare_heads_kernel(PrepSide q, PrepSide k, const TI* v_in, int v_in_stride, int v_dim, const float* v_bias, float eps,
+                         const float2* table, int rot_dims, int interleaved, TC* q_out, long long q_out_token_stride,
+                         long long q_out_head_stride, int q_out_dim_offset, TC* k_cache, TC* v_cache, const int* block_table,
+                         int max_pages, int page_size, int num_pages, const int* positions, const int* token_entry, int row_floats,
+                         int* status) {
+  extern __shared__ __align__(16) float rows[];      // [PREP_WARPS][row_floats]
+  pdl_trigger();
+  pdl_wait();
+  const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int q_heads = q.in ? q.heads : 0, k_heads = k.in ? k.heads : 0, v_heads = v_in != nullptr && v_cache != nullptr ? k.heads : 0;
+  const int row = blockIdx.y * PREP_WARPS + warp;
+  if (row >= q_heads + k_heads + v_heads) return;
+  float* buf = rows + warp * row_floats;
+  const bool is_q = row < q_heads, is_v = row >= q_heads + k_heads;
+  const int head = is_q ? row : is_v ? row - q_heads - k_heads : row - q_heads;
+  TC* dst;
+  if (is_q) {
+    dst = q_out + (size_t)token * q_out_token_stride + (size_t)head * q_out_head_stride + q_out_dim_offset;
+  } else {
+    const int pos = positions[token], logical = pos / page_size;
+    if (pos < 0 || logical >= max_pages) {
+      if (lane == 0) atomicOr(status, FE_STATUS_BAD_POSITION);
+      return;
+    }
+    const int page = block_table[(size_t)token_entry[token] * max_pages + logical];
+    if (page < 0 || page >= num_pages) {
+      if (lane == 0) atomicOr(status, FE_STATUS_BAD_PAGE);
+      return;
+    }
+    const size_t at = ((size_t)page * k.heads + head) * page_size + (pos - logical * page_size);
+    dst = is_v ? v_cache + at * v_dim : k_cache + at * k.dim;
+  }
+  if (is_v) {
+    const TI* src = v_in + (size_t)token * v_in_stride + (size_t)head * v_dim;
+    for (int i = lane * V; i < v_dim; i += 32 * V) {
+      float x[V], b[V];
+      prep_load<V>(src + i, x);
+      if (v_bias) {
+        prep_load<V>(v_bias + (size_t)head * v_dim + i, b);
+#pragma unroll
+        for (int e = 0; e < V; ++e) x[e] += b[e];
+      }
+      prep_store<V>(dst + i, x);
+    }
+    return;
+  }
+  // the side's fields one by one: a reference to either parameter would move both to memory
+  struct {
+    const void* in;
+    const float *norm_w, *bias;
+    int in_stride, head_stride, dim, norm_mode, norm_dims, rot_off;
+  } s;
+  s.in = is_q ? q.in : k.in;
+  s.norm_w = is_q ? q.norm_w : k.norm_w;
+  s.bias = is_q ? q.bias : k.bias;
+  s.in_stride = is_q ? q.in_stride : k.in_stride;
+  s.head_stride = is_q ? q.head_stride : k.head_stride;
+  s.dim = is_q ? q.dim : k.dim;
+  s.norm_mode = is_q ? q.norm_mode : k.norm_mode;
+  s.norm_dims = is_q ? q.norm_dims : k.norm_dims;
+  s.rot_off = is_q ? q.rot_off : k.rot_off;
+  const TI* src = (const TI*)s.in + (size_t)token * s.in_stride + (size_t)head * s.head_stride;
+  const bool rotates = table != nullptr && rot_dims > 0 && s.rot_off >= 0;
+  const float2* angles = rotates ? table + (size_t)token * (rot_dims >> 1) : nullptr;
+  const int half = rot_dims >> 1;
+  float ss = 0.f;
+  for (int i = lane * V; i < s.dim; i += 32 * V) {
+    float x[V], b[V];
+    prep_load<V>(src + i, x);
+    if (s.bias) {
+      prep_load<V>(s.bias + (size_t)head * s.dim + i, b);
+#pragma unroll
+      for (int e = 0; e < V; ++e) x[e] += b[e];
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e)
+      if (i + e < s.norm_dims) ss = fmaf(x[e], x[e], ss);
+    prep_store<V>(buf + i, x);
+  }
+  __syncwarp();
+  // a factor per element before the rotation (norm first) or after it (norm of the rotated head)
+  const bool first = s.norm_mode == PREP_NORM_HEAD, after = s.norm_mode == PREP_NORM_HEAD_AFTER;
+  float inv = 1.f;
+  if (first) inv = 1.f / sqrtf(warp_sum(ss) / (float)s.norm_dims + eps);
+  auto factor = [&](int i) { return i < s.norm_dims ? (s.norm_w != nullptr ? inv * s.norm_w[i] : inv) : 1.f; };
+  auto value = [&](int i) {
+    float x = first ? buf[i] * factor(i) : buf[i];
+    const int r = i - s.rot_off;
+    if (rotates && r >= 0 && r < rot_dims) {
+      // of a pair (u, v): u cos - v sin, v cos + u sin
+      const bool second = interleaved ? (r & 1) != 0 : r >= half;
+      const int pair = interleaved ? r >> 1 : second ? r - half : r;
+      const int other = interleaved ? (second ? i - 1 : i + 1) : second ? i - half : i + half;
+      const float2 cs = angles[pair];
+      const float y = first ? buf[other] * factor(other) : buf[other];
+      x = x * cs.x + y * (second ? cs.y : -cs.y);
+    }
+    return x;
+  };
+  if (after) {
+    float sum = 0.f;
+    for (int i = lane; i < s.norm_dims; i += 32) {
+      const float x = value(i);
+      sum = fmaf(x, x, sum);
+    }
+    inv = 1.f / sqrtf(warp_sum(sum) / (float)s.norm_dims + eps);
+  }
+  for (int i = lane * V; i < s.dim; i += 32 * V) {
+    float x[V];
+#pragma unroll
+    for (int e = 0; e < V; ++e) x[e] = value(i + e) * (after ? factor(i + e) : 1.f);
+    prep_store<V>(dst + i, x);
+  }
+}
+
+// The same for heads of up to 128 elements in fours whose rotation keeps to fours as well: a head in the
+// registers of `group` neighbouring lanes (a power of two, four elements a lane), so that a warp takes
+// 32 / group heads; a pair's other half comes from a lane half / 4 away.
+template <typename TI, typename TC>
+__global__ void __launch_bounds__(32 * PREP_WARPS)
+qkv_prepare_lanes_kernel(PrepSide q, PrepSide k, const TI* v_in, int v_in_stride, int v_dim, const float* v_bias, float eps,
+                         const float2* table, int rot_dims, int interleaved, TC* q_out, long long q_out_token_stride,
+                         long long q_out_head_stride, int q_out_dim_offset, TC* k_cache, TC* v_cache, const int* block_table,
+                         int max_pages, int page_size, int num_pages, const int* positions, const int* token_entry, int group,
+                         int* status) {
+  pdl_trigger();
+  pdl_wait();
+  const int token = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int q_heads = q.in ? q.heads : 0, k_heads = k.in ? k.heads : 0, v_heads = v_in != nullptr && v_cache != nullptr ? k.heads : 0;
+  const int row = (blockIdx.y * PREP_WARPS + warp) * (32 / group) + lane / group, i = (lane & (group - 1)) * 4;
+  bool live = row < q_heads + k_heads + v_heads;
+  const bool is_q = row < q_heads, is_v = row >= q_heads + k_heads;
+  const int head = is_q ? row : is_v ? row - q_heads - k_heads : row - q_heads;
+  const int dim = is_q ? q.dim : is_v ? v_dim : k.dim;
+  live = live && i < dim;
+  TC* dst = nullptr;
+  if (live && is_q) {
+    dst = q_out + (size_t)token * q_out_token_stride + (size_t)head * q_out_head_stride + q_out_dim_offset + i;
+  } else if (live) {
+    const int pos = positions[token], logical = pos / page_size;
+    int page = -1;
+    if (pos < 0 || logical >= max_pages) atomicOr(status, FE_STATUS_BAD_POSITION);
+    else if ((page = block_table[(size_t)token_entry[token] * max_pages + logical]) < 0 || page >= num_pages) atomicOr(status, FE_STATUS_BAD_PAGE), page = -1;
+    const size_t at = ((size_t)page * k.heads + head) * page_size + (pos - logical * page_size);
+    if (page >= 0) dst = (is_v ? v_cache + at * v_dim : k_cache + at * k.dim) + i;
+  }
+  float x[4] = {0.f, 0.f, 0.f, 0.f};
+  if (live) {
+    const TI* src = is_q ? (const TI*)q.in + (size_t)token * q.in_stride + (size_t)head * q.head_stride
+                         : is_v ? v_in + (size_t)token * v_in_stride + (size_t)head * v_dim
+                                : (const TI*)k.in + (size_t)token * k.in_stride + (size_t)head * k.head_stride;
+    load4(src + i, x);
+    const float* bias = is_q ? q.bias : is_v ? v_bias : k.bias;
+    if (bias != nullptr) {
+      float b[4];
+      load4(bias + (size_t)head * dim + i, b);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] += b[e];
+    }
+  }
+  const int mode = is_v ? PREP_NORM_NONE : is_q ? q.norm_mode : k.norm_mode, dims = is_q ? q.norm_dims : k.norm_dims;
+  const float* norm_w = is_q ? q.norm_w : k.norm_w;
+  auto norm = [&](bool wanted) {
+    float ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (i + e < dims) ss = fmaf(x[e], x[e], ss);
+    for (int o = group >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    const float inv = 1.f / sqrtf(ss / (float)dims + eps);
+#pragma unroll
+    for (int e = 0; e < 4; ++e)
+      if (wanted && live && i + e < dims) x[e] *= norm_w != nullptr ? inv * norm_w[i + e] : inv;
+  };
+  const bool some_first = q.norm_mode == PREP_NORM_HEAD || k.norm_mode == PREP_NORM_HEAD;
+  const bool some_after = q.norm_mode == PREP_NORM_HEAD_AFTER || k.norm_mode == PREP_NORM_HEAD_AFTER;
+  if (some_first) norm(mode == PREP_NORM_HEAD);
+  const int rot_off = is_q ? q.rot_off : k.rot_off, r = i - rot_off, half = rot_dims >> 1;
+  const bool rotates = table != nullptr && live && !is_v && rot_off >= 0 && r >= 0 && r < rot_dims;
+  const float2* angles = table + (size_t)token * half;
+  if (interleaved) {
+    if (rotates) {
+      float a[4];
+      load4(reinterpret_cast<const float*>(angles + (r >> 1)), a);
+      const float u = x[0], v = x[2];
+      x[0] = u * a[0] - x[1] * a[1], x[1] = x[1] * a[0] + u * a[1];
+      x[2] = v * a[2] - x[3] * a[3], x[3] = x[3] * a[2] + v * a[3];
+    }
+  } else if (table != nullptr) {
+    const bool second = r >= half;
+    const int from = rotates ? (second ? lane - (half >> 2) : lane + (half >> 2)) : lane;
+    float y[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) y[e] = __shfl_sync(0xffffffffu, x[e], from);
+    if (rotates) {
+      float a[8];
+      load8(reinterpret_cast<const float*>(angles + (second ? r - half : r)), a);
+#pragma unroll
+      for (int e = 0; e < 4; ++e) x[e] = x[e] * a[2 * e] + y[e] * (second ? a[2 * e + 1] : -a[2 * e + 1]);
+    }
+  }
+  if (some_after) norm(mode == PREP_NORM_HEAD_AFTER);
+  if (dst != nullptr) store4(dst, x);
 }
 
 FE_EXPORT int fe_qkv_prepare(const void* q_in, int q_in_stride, int q_head_stride, int q_heads, int q_dim, int q_norm_mode, int q_norm_dims,
                              const float* q_norm_w, int q_rot_off, const void* k_in, int k_in_stride, int k_heads,
                              int k_dim, int k_norm_mode, int k_norm_dims, const float* k_norm_w, int k_rot_off,
-                             const void* v_in, int v_in_stride, int v_dim, int in_dtype, float eps, const float* table,
+                             const void* v_in, int v_in_stride, int v_dim, const float* q_bias, const float* k_bias,
+                             const float* v_bias, int in_dtype, float eps, const float* table,
                              int rot_dims, int interleaved, void* q_out, long long q_out_token_stride,
                              long long q_out_head_stride, int q_out_dim_offset, void* k_cache, void* v_cache,
                              int cache_dtype, const int* block_table, int max_pages, int page_size, int num_pages,
@@ -174,19 +392,70 @@ FE_EXPORT int fe_qkv_prepare(const void* q_in, int q_in_stride, int q_head_strid
                              cudaStream_t stream) {
   if (n_tokens <= 0) return 0;
   if (rot_dims % 2 || (q_in && q_rot_off >= 0 && q_rot_off + rot_dims > q_dim) || (k_in && k_rot_off >= 0 && k_rot_off + rot_dims > k_dim)) return FE_ERR_BAD_SHAPE;
-  PrepSide q{q_in, q_in_stride, q_head_stride > 0 ? q_head_stride : q_dim, q_heads, q_dim, q_norm_mode, q_norm_dims, q_norm_w, q_rot_off};
-  PrepSide k{k_in, k_in_stride, k_dim, k_heads, k_dim, k_norm_mode, k_norm_dims, k_norm_w, k_rot_off};
+  PrepSide q{q_in, q_in_stride, q_head_stride > 0 ? q_head_stride : q_dim, q_heads, q_dim, q_norm_mode, q_norm_dims, q_norm_w, q_rot_off, q_bias};
+  PrepSide k{k_in, k_in_stride, k_dim, k_heads, k_dim, k_norm_mode, k_norm_dims, k_norm_w, k_rot_off, k_bias};
   const size_t q_floats = q_in ? (size_t)q_heads * q_dim : 0, k_floats = k_in ? (size_t)k_heads * k_dim : 0;
   const int sides = (q_in && k_in) ? 2 : 1;
   const size_t smem = sizeof(float) * (q_floats > k_floats ? q_floats : k_floats);
-  if (smem > 200 * 1024) return FE_ERR_TOO_LARGE;
   int rc = 0;
+  if (q_norm_mode != PREP_NORM_WHOLE && k_norm_mode != PREP_NORM_WHOLE) {
+    const int total = (q_in ? q_heads : 0) + (k_in ? k_heads * (v_in && v_cache ? 2 : 1) : 0);
+    int widest = q_in ? q_dim : 0;
+    if (k_in && k_dim > widest) widest = k_dim;
+    widest = (widest + 3) / 4 * 4;
+    const size_t heads_smem = sizeof(float) * PREP_WARPS * (size_t)widest;
+    if (total > 65535 * PREP_WARPS) return FE_ERR_TOO_LARGE;
+    if (heads_smem <= 48 * 1024) {
+      uintptr_t pointers = (uintptr_t)q_in | (uintptr_t)k_in | (uintptr_t)v_in | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache |
+                           (uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)v_bias;
+      const long long sizes = (q_in ? q_in_stride | q.head_stride | q_dim | q_out_dim_offset | q_out_token_stride | q_out_head_stride : 0) |
+                              (k_in ? k_in_stride | k_dim : 0) | (v_in ? v_in_stride | v_dim : 0);
+      const bool wide = pointers % 16 == 0 && sizes % 4 == 0;
+      const int widest_v = v_in && v_dim > widest ? (v_dim + 3) / 4 * 4 : widest;
+      bool fours = wide && widest_v <= 128 && (uintptr_t)table % 16 == 0 && rot_dims % 4 == 0;
+      if (table != nullptr && rot_dims > 0) {
+        if (q_in && q_rot_off >= 0) fours = fours && q_rot_off % 4 == 0;
+        if (k_in && k_rot_off >= 0) fours = fours && k_rot_off % 4 == 0;
+        fours = fours && (interleaved || rot_dims % 8 == 0);
+      }
+      if (fours) {
+        int group = 1;
+        while (group * 4 < widest_v) group <<= 1;
+        const int per = PREP_WARPS * (32 / group);
+        const dim3 lanes_grid(n_tokens, (total + per - 1) / per);
+#define LAUNCH_LANES(TI, TC)                                                                                            \
+  rc = fe_launch_dependent(qkv_prepare_lanes_kernel<TI, TC>, lanes_grid, dim3(32 * PREP_WARPS), 0, stream, q, k,       \
+                           (const TI*)v_in, v_in_stride, v_dim, v_bias, eps, (const float2*)table, rot_dims, interleaved, \
+                           (TC*)q_out, q_out_token_stride, q_out_head_stride, q_out_dim_offset, (TC*)k_cache,          \
+                           (TC*)v_cache, block_table, max_pages, page_size, num_pages, positions, token_entry, group, status)
+        if (in_dtype == FE_DTYPE_F32 && cache_dtype == FE_DTYPE_F32) LAUNCH_LANES(float, float);
+        else if (in_dtype == FE_DTYPE_F32 && cache_dtype == FE_DTYPE_BF16) LAUNCH_LANES(float, bf16);
+        else if (in_dtype == FE_DTYPE_BF16 && cache_dtype == FE_DTYPE_BF16) LAUNCH_LANES(bf16, bf16);
+        else return FE_ERR_BAD_DTYPE;
+#undef LAUNCH_LANES
+        return rc ? rc : fe_last_error();
+      }
+      const dim3 grid(n_tokens, (total + PREP_WARPS - 1) / PREP_WARPS);
+#define LAUNCH_HEADS(TI, TC, V)                                                                                          \
+  rc = fe_launch_dependent(qkv_prepare_heads_kernel<TI, TC, V>, grid, dim3(32 * PREP_WARPS), heads_smem, stream, q, k,   \
+                           (const TI*)v_in, v_in_stride, v_dim, v_bias, eps, (const float2*)table, rot_dims, interleaved, \
+                           (TC*)q_out, q_out_token_stride, q_out_head_stride, q_out_dim_offset, (TC*)k_cache,            \
+                           (TC*)v_cache, block_table, max_pages, page_size, num_pages, positions, token_entry, widest, status)
+      if (in_dtype == FE_DTYPE_F32 && cache_dtype == FE_DTYPE_F32) { if (wide) LAUNCH_HEADS(float, float, 4); else LAUNCH_HEADS(float, float, 1); }
+      else if (in_dtype == FE_DTYPE_F32 && cache_dtype == FE_DTYPE_BF16) { if (wide) LAUNCH_HEADS(float, bf16, 4); else LAUNCH_HEADS(float, bf16, 1); }
+      else if (in_dtype == FE_DTYPE_BF16 && cache_dtype == FE_DTYPE_BF16) { if (wide) LAUNCH_HEADS(bf16, bf16, 4); else LAUNCH_HEADS(bf16, bf16, 1); }
+      else return FE_ERR_BAD_DTYPE;
+#undef LAUNCH_HEADS
+      return rc ? rc : fe_last_error();
+    }
+  }
+  if (smem > 200 * 1024) return FE_ERR_TOO_LARGE;
 #define LAUNCH(TI, TC)                                                                                              \
   do {                                                                                                              \
     if (smem > 48 * 1024)                                                                                           \
       cudaFuncSetAttribute(qkv_prepare_kernel<TI, TC>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);     \
     rc = fe_launch_dependent(qkv_prepare_kernel<TI, TC>, dim3(n_tokens, sides), dim3(256), smem, stream, q, k,             \
-                             (const TI*)v_in, v_in_stride, v_dim, eps, (const float2*)table, rot_dims, interleaved, \
+                             (const TI*)v_in, v_in_stride, v_dim, v_bias, eps, (const float2*)table, rot_dims, interleaved, \
                              (TC*)q_out, q_out_token_stride, q_out_head_stride, q_out_dim_offset, (TC*)k_cache,     \
                              (TC*)v_cache, block_table, max_pages, page_size, num_pages, positions, token_entry,    \
                              status);                                                                               \

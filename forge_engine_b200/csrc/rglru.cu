@@ -34,6 +34,7 @@ struct Rglru {
   const float* conv_b;      // [width]
   int taps;
   const void *wr, *wi;      // [blocks, part, part], a gate's row is the output channel
+  const float *y_bias, *x_bias;     // [width]: of the projection, not yet in proj
   const float *br, *bi, *rate;      // [width]
   float* state;             // [rows, width]
   float* conv_state;        // [rows, taps - 1, width], oldest first
@@ -49,16 +50,32 @@ struct Rglru {
 #define RG_WP (RG_KC + 8)   // pitch of a bfloat16 tile
 #define RG_FP (RG_KC + 4)   // pitch of a 32-bit tile
 
-__device__ __forceinline__ float rg_sigmoid(float z) { return __fdividef(1.f, 1.f + expf(-z)); }
+__device__ __forceinline__ float rg_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
 __device__ __forceinline__ float rg_gelu(float z) {
   // 0.5 (1 + tanh(t)) = sigmoid(2 t)
   return z * rg_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z));
+}
+// 1 - e^(-x) for x >= 0, given e = e^(-x): near zero by the power series, whose terms keep the digits
+// that the subtraction would lose
+__device__ __forceinline__ float rg_one_minus_exp(float x, float e) {
+  float s = fmaf(x, -1.f / 7.f, 1.f);
+  s = fmaf(-x * (1.f / 6.f), s, 1.f);
+  s = fmaf(-x * (1.f / 5.f), s, 1.f);
+  s = fmaf(-x * (1.f / 4.f), s, 1.f);
+  s = fmaf(-x * (1.f / 3.f), s, 1.f);
+  s = fmaf(-x * (1.f / 2.f), s, 1.f);
+  return x < 0.25f ? x * s : 1.f - e;
+}
+__device__ __forceinline__ float rg_sqrt(float x) {
+  float y;
+  asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
 // a and the input's factor sqrt(1 - a^2) i from the gates' sums
 __device__ __forceinline__ void rg_gates(float zr, float zi, float rate, float* a, float* scale) {
   const float log_a = rate * rg_sigmoid(zr);
   *a = expf(log_a);
-  *scale = sqrtf(-expm1f(2.f * log_a)) * rg_sigmoid(zi);
+  *scale = rg_sqrt(rg_one_minus_exp(-2.f * log_a, *a * *a)) * rg_sigmoid(zi);
 }
 __device__ __forceinline__ void rg_copy4(void* dst, const void* src, bool valid) {
   const int bytes = valid ? 4 : 0;
@@ -125,7 +142,7 @@ template <typename TW, int NC, int TAPS>
 __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int stage_bytes, int* status) {
   using Shape = RgShape<TW, NC>;
   extern __shared__ __align__(16) unsigned char raw[];
-  __shared__ int since[RG_RM], slot_of[RG_RM];       // tokens since the entry's first; the request's row (-1: past the end)
+  __shared__ int since[RG_RM], slot_of[RG_RM];       // tokens since the entry's first; the request's row (-1: none)
   __shared__ float seg_h[4][NC], seg_p[4][NC];
   pdl_trigger();
   pdl_wait();
@@ -137,19 +154,6 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
   float* xs = reinterpret_cast<float*>(raw + 2 * Shape::W_BYTES);              // [2 stages][RM + back][KC]
   unsigned char* as = raw + stage_bytes;                                       // u: hi and lo [RM][RG_WP], or 32-bit [RM][RG_FP]
   float* us = reinterpret_cast<float*>(as + Shape::A_BYTES);                   // [RM][NC]: u of the block's own channels
-  if (tid < RG_RM) {
-    int s = -1, n = 0;
-    if (tid < rows) {
-      const int entry = p.token_entry[t0 + tid];
-      n = t0 + tid - p.cu_tokens[entry];
-      s = p.slots[entry];
-      if (s < 0 || s >= p.state_rows) {
-        atomicOr(status, FE_STATUS_BAD_PAGE);
-        s = -1;
-      }
-    }
-    since[tid] = n, slot_of[tid] = s;
-  }
   const TW* wr = (const TW*)p.wr + (size_t)block * part * part;
   const TW* wi = (const TW*)p.wi + (size_t)block * part * part;
   const int x0 = block * part;                       // the part's first channel
@@ -175,6 +179,23 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
     }
     cp_commit();
   };
+  load(0, 0);
+  int n = 1 << 30;                                   // past the last token: as if far inside an entry
+  if (tid < RG_RM) {
+    int s = -1;
+    if (tid < rows) {
+      const int entry = p.token_entry[t0 + tid];
+      n = t0 + tid - p.cu_tokens[entry];
+      s = p.slots[entry];
+      if (s < 0 || s >= p.state_rows) {
+        atomicOr(status, FE_STATUS_BAD_PAGE);
+        s = -1;
+      }
+    }
+    since[tid] = n, slot_of[tid] = s;
+  }
+  const bool edge = __syncthreads_or(n < back);      // some tokens' taps reach into a request's state
+  const bool begins = __syncthreads_or(n == 0);      // an entry begins in this tile
 
   // products: a warp takes 16 tokens x 32 channels of both gates; 32-bit: a thread 4 x 4
   float acc[2][4][4];
@@ -186,8 +207,10 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
       for (int e = 0; e < 4; ++e) acc[g][j][e] = 0.f;
   const int rw = warp & 3, cw = warp >> 2;
   const int fr = (tid & 15) * 4, fc = tid >> 4;      // 32-bit: rows fr .. fr + 3, channels fc + NC / 4 * e
+  // the convolution: a thread takes two channels of PER neighbouring tokens
+  constexpr int PER = RG_RM / (Shape::THREADS / 32);
+  const int c2 = lane * 2, r0 = warp * PER;
 
-  load(0, 0);
   for (int k0 = 0, stage = 0; k0 < part; k0 += RG_KC, stage ^= 1) {
     if (k0 + RG_KC < part) {
       load(k0 + RG_KC, stage ^ 1);
@@ -197,56 +220,63 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
     }
     __syncthreads();
     {
-      // the convolution: a thread takes one channel of RM / (NC / 16) neighbouring tokens
-      constexpr int GROUPS = Shape::THREADS / RG_KC, PER = RG_RM / GROUPS;
-      const int c = tid & (RG_KC - 1), r0 = (tid / RG_KC) * PER, ch = x0 + k0 + c;
-      const bool live = k0 + c < part;
-      const float* x = xs + stage * (RG_RM + back) * RG_KC + c;
-      const float bias = live ? p.conv_b[ch] : 0.f;
-      float w[TAPS > 0 ? TAPS : 1], hist[TAPS > 0 ? TAPS : 1];
-      if constexpr (TAPS > 0) {
+      const float* x = xs + stage * (RG_RM + back) * RG_KC + c2;
+      const int ch = x0 + k0 + c2, own = k0 + c2 - n0;
+      const bool live0 = k0 + c2 < part, live1 = k0 + c2 + 1 < part;
+      auto put = [&](int r, float u0, float u1) {
+        if constexpr (Shape::MMA) {
+          unsigned h, l;
+          split2(u0, u1, h, l);
+          bf16* hi = reinterpret_cast<bf16*>(as) + r * RG_WP + c2;
+          *reinterpret_cast<unsigned*>(hi) = h;
+          *reinterpret_cast<unsigned*>(hi + RG_RM * RG_WP) = l;
+        } else {
+          *reinterpret_cast<float2*>(reinterpret_cast<float*>(as) + r * RG_FP + c2) = make_float2(u0, u1);
+        }
+        if (own >= 0 && own < NC) *reinterpret_cast<float2*>(us + r * NC + own) = make_float2(u0, u1);
+      };
+      if (TAPS > 0 && !edge) {
+        // every tap inside the step: the projection's bias goes through the taps' sum
+        float w0[TAPS > 0 ? TAPS : 1], w1[TAPS > 0 ? TAPS : 1], b0 = 0.f, b1 = 0.f;
+        float2 in[TAPS > 0 ? TAPS : 1];
 #pragma unroll
         for (int j = 0; j < TAPS; ++j) {
-          w[j] = live ? p.conv_w[(size_t)j * p.width + ch] : 0.f;
-          hist[j] = j < TAPS - 1 ? x[(r0 + j) * RG_KC] : 0.f;
+          w0[j] = live0 ? p.conv_w[(size_t)j * p.width + ch] : 0.f;
+          w1[j] = live1 ? p.conv_w[(size_t)j * p.width + ch + 1] : 0.f;
+          b0 += w0[j], b1 += w1[j];
+          in[j] = *reinterpret_cast<const float2*>(x + (r0 + (j < TAPS - 1 ? j : 0)) * RG_KC);
         }
-      }
-#pragma unroll 4
-      for (int r = r0; r < r0 + PER; ++r) {
-        float u = bias;
-        if constexpr (TAPS > 0) hist[TAPS - 1] = x[(r + back) * RG_KC];
-        if (since[r] >= back) {
-          if constexpr (TAPS > 0) {
+        b0 = live0 ? fmaf(b0, p.x_bias[ch], p.conv_b[ch]) : 0.f;
+        b1 = live1 ? fmaf(b1, p.x_bias[ch + 1], p.conv_b[ch + 1]) : 0.f;
 #pragma unroll
-            for (int j = 0; j < TAPS; ++j) u = fmaf(w[j], hist[j], u);
-          } else if (live) {
-            for (int j = 0; j < taps; ++j) u = fmaf(p.conv_w[(size_t)j * p.width + ch], x[(r + j) * RG_KC], u);
-          }
-        } else if (live) {
-          // an entry's first tokens: the inputs before them come from the request's state
-          for (int j = 0; j < taps; ++j) {
-            const int at = since[r] + j;             // index into (state rows, the entry's rows)
-            float v = 0.f;
-            if (at >= back) v = x[(r + j) * RG_KC];
-            else if (slot_of[r] >= 0) v = p.conv_state[((size_t)slot_of[r] * back + at) * p.width + ch];
-            u = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u);
-          }
-        }
-        if constexpr (TAPS > 0) {
+        for (int i = 0; i < PER; ++i) {
+          in[TAPS > 0 ? TAPS - 1 : 0] = *reinterpret_cast<const float2*>(x + (r0 + i + back) * RG_KC);
+          float u0 = b0, u1 = b1;
 #pragma unroll
-          for (int j = 0; j + 1 < TAPS; ++j) hist[j] = hist[j + 1];
+          for (int j = 0; j < TAPS; ++j) u0 = fmaf(w0[j], in[j].x, u0), u1 = fmaf(w1[j], in[j].y, u1);
+          put(r0 + i, u0, u1);
+#pragma unroll
+          for (int j = 0; j + 1 < TAPS; ++j) in[j] = in[j + 1];
         }
-        if (!live || r >= rows) u = 0.f;
-        if constexpr (Shape::MMA) {
-          bf16* hi = reinterpret_cast<bf16*>(as) + r * RG_WP + c;
-          const bf16 rounded = __float2bfloat16_rn(u);
-          hi[0] = rounded;
-          hi[RG_RM * RG_WP] = __float2bfloat16_rn(u - __bfloat162float(rounded));
-        } else {
-          reinterpret_cast<float*>(as)[r * RG_FP + c] = u;
+      } else {
+        for (int r = r0; r < r0 + PER; ++r) {
+          float u[2] = {0.f, 0.f};
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            if (!(e == 0 ? live0 : live1)) continue;
+            const float bias = p.x_bias[ch + e];
+            u[e] = p.conv_b[ch + e];
+            for (int j = 0; j < taps; ++j) {
+              // index into (the state's rows, the entry's rows)
+              const int at = since[r] < back ? since[r] + j : back;
+              float v = 0.f;
+              if (at >= back) v = x[(r + j) * RG_KC + e] + bias;
+              else if (slot_of[r] >= 0) v = p.conv_state[((size_t)slot_of[r] * back + at) * p.width + ch + e];
+              u[e] = fmaf(p.conv_w[(size_t)j * p.width + ch + e], v, u[e]);
+            }
+          }
+          put(r, u[0], u[1]);
         }
-        const int own = k0 + c - n0;
-        if (own >= 0 && own < NC) us[r * NC + own] = u;
       }
     }
     __syncthreads();
@@ -312,43 +342,45 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
   // earlier tokens leave (unless an entry begins in between)
   const int c = tid % NC, seg = tid / NC, r_from = seg * 16;
   const bool live = n0 + c < part;
-  const int ch = x0 + n0 + c;
-  float h = 0.f, prod = 1.f;
-  int fresh = RG_RM;                     // the segment's first row that begins an entry
-  if (live) {
-    const float br = p.br[ch], bi = p.bi[ch], rate = p.rate[ch];
-#pragma unroll 4
-    for (int r = r_from; r < r_from + 16; ++r) {
+  const int ch = live ? x0 + n0 + c : x0;
+  const float br = p.br[ch], bi = p.bi[ch], rate = p.rate[ch];
+  float h[16], prod[16];
+  int fresh = 16;                        // the segment's first row that begins an entry
+  {
+    float s = 0.f, q = 1.f;
+#pragma unroll
+    for (int i = 0; i < 16; ++i) {
+      const int r = r_from + i;
       float a, scale;
       rg_gates(gates[r * GP + c] + br, gates[(RG_RM + r) * GP + c] + bi, rate, &a, &scale);
-      if (since[r] == 0) {
-        h = 0.f, prod = 1.f;
-        if (fresh == RG_RM) fresh = r;
+      if (begins && since[r] == 0) {
+        s = 0.f, q = 1.f;
+        fresh = min(fresh, i);
       }
-      h = fmaf(a, h, scale * us[r * NC + c]);
-      prod *= a;
-      gates[r * GP + c] = h;
-      gates[(RG_RM + r) * GP + c] = prod;
+      s = fmaf(a, s, scale * us[r * NC + c]);
+      q *= a;
+      h[i] = s, prod[i] = q;
     }
+    seg_h[seg][c] = s, seg_p[seg][c] = q;
   }
-  seg_h[seg][c] = h, seg_p[seg][c] = prod;
   __syncthreads();
   if (!live) return;
-  float ch_in = 0.f, cp_in = 1.f;
+  float h_in = 0.f, p_in = 1.f;
   for (int s = 0; s < seg; ++s) {
-    bool begins = false;
-    for (int r = s * 16; r < s * 16 + 16; ++r) begins = begins || since[r] == 0;
-    ch_in = begins ? seg_h[s][c] : fmaf(seg_p[s][c], ch_in, seg_h[s][c]);
-    cp_in = begins ? seg_p[s][c] : seg_p[s][c] * cp_in;
+    bool cut = false;
+    if (begins)
+      for (int r = s * 16; r < s * 16 + 16; ++r) cut = cut || since[r] == 0;
+    h_in = cut ? seg_h[s][c] : fmaf(seg_p[s][c], h_in, seg_h[s][c]);
+    p_in = cut ? seg_p[s][c] : seg_p[s][c] * p_in;
   }
-#pragma unroll 4
-  for (int r = r_from; r < r_from + 16; ++r) {
-    if (r >= rows) break;
-    float hr = gates[r * GP + c], pr = gates[(RG_RM + r) * GP + c];
-    if (r < fresh) hr = fmaf(pr, ch_in, hr), pr *= cp_in;
-    const size_t at = (size_t)(t0 + r) * p.width + ch;
-    p.h[at] = hr;
-    p.prod[at] = pr;
+  float *hp = p.h + (size_t)(t0 + r_from) * p.width + ch, *pp = p.prod + (size_t)(t0 + r_from) * p.width + ch;
+#pragma unroll
+  for (int i = 0; i < 16; ++i) {
+    if (r_from + i < rows) {
+      const bool joined = i < fresh;
+      hp[(size_t)i * p.width] = joined ? fmaf(prod[i], h_in, h[i]) : h[i];
+      pp[(size_t)i * p.width] = joined ? prod[i] * p_in : prod[i];
+    }
   }
 }
 
@@ -386,7 +418,7 @@ __global__ void __launch_bounds__(64) rglru_chain_kernel(const Rglru p) {
   float* st = p.conv_state + (size_t)slot * back * p.width + c;
   for (int k = 0; k < back; ++k) {
     const int at = count + k;
-    st[(size_t)k * p.width] = at < back ? st[(size_t)at * p.width] : p.proj[(size_t)(first + at - back) * p.ld + p.x_off + c];
+    st[(size_t)k * p.width] = at < back ? st[(size_t)at * p.width] : p.proj[(size_t)(first + at - back) * p.ld + p.x_off + c] + p.x_bias[c];
   }
 }
 
@@ -403,11 +435,11 @@ __global__ void __launch_bounds__(256) rglru_out_kernel(const Rglru p) {
   const float* in = p.cu_tokens[entry] >= tile * RG_RM ? p.init + (size_t)entry * p.width : p.carry + (size_t)tile * p.width;
   const size_t at = (size_t)t * p.width + c;
   const float* yp = p.proj + (size_t)t * p.ld + p.y_off + c;
-  float h[V], a[V], s[V], y[V];
-  if constexpr (V == 4) load4(p.h + at, h), load4(p.prod + at, a), load4(in + c, s), load4(yp, y);
-  else h[0] = p.h[at], a[0] = p.prod[at], s[0] = in[c], y[0] = yp[0];
+  float h[V], a[V], s[V], y[V], b[V];
+  if constexpr (V == 4) load4(p.h + at, h), load4(p.prod + at, a), load4(in + c, s), load4(yp, y), load4(p.y_bias + c, b);
+  else h[0] = p.h[at], a[0] = p.prod[at], s[0] = in[c], y[0] = yp[0], b[0] = p.y_bias[c];
 #pragma unroll
-  for (int e = 0; e < V; ++e) h[e] = fmaf(a[e], s[e], h[e]) * rg_gelu(y[e]);
+  for (int e = 0; e < V; ++e) h[e] = fmaf(a[e], s[e], h[e]) * rg_gelu(y[e] + b[e]);
   if constexpr (V == 4) store4((TO*)p.out + at, h);
   else ((TO*)p.out)[at] = from_float<TO>(h[0]);
 }
@@ -451,7 +483,7 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
     float u = 0.f;
     if (r < rows && c < cols) {
       const int ch = x0 + n0 + c, slot = p.slots[t0 + r];
-      const float x = p.proj[(size_t)(t0 + r) * p.ld + p.x_off + ch];
+      const float x = p.proj[(size_t)(t0 + r) * p.ld + p.x_off + ch] + p.x_bias[ch];
       u = p.conv_b[ch];
       if (slot >= 0 && slot < p.state_rows) {
         // the oldest input leaves the history, the others move up
@@ -518,7 +550,7 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
     float* cell = p.state + (size_t)slot * p.width + ch;
     const float s = fmaf(a, *cell, scale * us[r * GP + c]);
     *cell = s;
-    ((TO*)p.out)[(size_t)(t0 + r) * p.width + ch] = from_float<TO>(s * rg_gelu(p.proj[(size_t)(t0 + r) * p.ld + p.y_off + ch]));
+    ((TO*)p.out)[(size_t)(t0 + r) * p.width + ch] = from_float<TO>(s * rg_gelu(p.proj[(size_t)(t0 + r) * p.ld + p.y_off + ch] + p.y_bias[ch]));
   }
 }
 
@@ -560,7 +592,7 @@ FE_EXPORT long long fe_rglru_scratch(int tokens, int entries, int width) {
 }
 
 FE_EXPORT int fe_rglru(const float* proj, long long ld, int y_off, int x_off, const float* conv_w, const float* conv_b, int taps,
-                       const void* wr, const void* wi, int weight_dtype, const float* br, const float* bi, const float* rate,
+                       const void* wr, const void* wi, int weight_dtype, const float* y_bias, const float* x_bias, const float* br, const float* bi, const float* rate,
                        float* state, float* conv_state, int state_rows, const int* slots, const int* cu_tokens,
                        const int* token_entry, void* out, int out_dtype, int width, int part, int tokens, int entries, int max_new,
                        float* scratch, int* status, cudaStream_t stream) {
@@ -569,7 +601,7 @@ FE_EXPORT int fe_rglru(const float* proj, long long ld, int y_off, int x_off, co
     return FE_ERR_BAD_SHAPE;
   if ((tokens + RG_SM - 1) / RG_SM > 65535) return FE_ERR_TOO_LARGE;
   if (((uintptr_t)wr | (uintptr_t)wi) & 15) return FE_ERR_BAD_ALIGN;
-  Rglru p{proj, ld, y_off, x_off, conv_w, conv_b, taps, wr, wi, br, bi, rate, state, conv_state, state_rows, slots, cu_tokens,
+  Rglru p{proj, ld, y_off, x_off, conv_w, conv_b, taps, wr, wi, y_bias, x_bias, br, bi, rate, state, conv_state, state_rows, slots, cu_tokens,
           token_entry, width, part, tokens, entries, nullptr, nullptr, nullptr, nullptr, out};
   int rc = FE_ERR_BAD_DTYPE;
   if (max_new == 1 && tokens == entries && fe_rglru_one_launch(part, weight_dtype)) {
@@ -584,12 +616,14 @@ FE_EXPORT int fe_rglru(const float* proj, long long ld, int y_off, int x_off, co
   p.prod = p.h + (size_t)tokens * pitch;
   p.carry = p.prod + (size_t)tokens * pitch;
   p.init = p.carry + (tiles + 1) * pitch;
-  if (weight_dtype == FE_DTYPE_BF16) rc = taps == 4 ? rg_launch_gates<bf16, 64, 4>(p, status, stream) : rg_launch_gates<bf16, 64, 0>(p, status, stream);
+  static const int nc = getenv("RG_NC") ? atoi(getenv("RG_NC")) : 128;
+  if (weight_dtype == FE_DTYPE_BF16 && nc == 128 && part >= 128) rc = taps == 4 ? rg_launch_gates<bf16, 128, 4>(p, status, stream) : rg_launch_gates<bf16, 128, 0>(p, status, stream);
+  else if (weight_dtype == FE_DTYPE_BF16) rc = taps == 4 ? rg_launch_gates<bf16, 64, 4>(p, status, stream) : rg_launch_gates<bf16, 64, 0>(p, status, stream);
   else if (weight_dtype == FE_DTYPE_F32) rc = taps == 4 ? rg_launch_gates<float, 64, 4>(p, status, stream) : rg_launch_gates<float, 64, 0>(p, status, stream);
   if (rc) return rc;
   rc = fe_launch_dependent(rglru_chain_kernel, dim3((width + 63) / 64, entries), dim3(64), 0, stream, p);
   if (rc) return rc;
-  const bool wide = width % 4 == 0 && ld % 4 == 0 && y_off % 4 == 0 && (((uintptr_t)proj | (uintptr_t)scratch | (uintptr_t)out) & 15) == 0;
+  const bool wide = width % 4 == 0 && ld % 4 == 0 && y_off % 4 == 0 && (((uintptr_t)proj | (uintptr_t)scratch | (uintptr_t)out | (uintptr_t)y_bias) & 15) == 0;
   const int per = wide ? 4 : 1;
   int threads = 32;
   while (threads < 256 && threads * per < width) threads <<= 1;

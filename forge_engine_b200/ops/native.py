@@ -60,7 +60,7 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_stream_mix_norm": [p, i, p, i, f, p, p, p, i, p, f, p, i, p, i, i, i, p],
         "fe_act_mul": [p, i, p, i, i, i, i, i, f, f, p],
         "fe_gated_rmsnorm": [p, p, i, i, p, p, i, i, i, f, p],
-        "fe_qkv_prepare": [p, i, i, i, i, i, i, p, i, p, i, i, i, i, i, p, i, p, i, i, i, f, p, i, i, p, ll, ll, i,
+        "fe_qkv_prepare": [p, i, i, i, i, i, i, p, i, p, i, i, i, i, i, p, i, p, i, i, p, p, p, i, f, p, i, i, p, ll, ll, i,
                            p, p, i, p, i, i, i, p, p, i, p, p],
         "fe_attention_general": [p, ll, ll, p, i, i, p, i, i, p, ll, ll, i, p, i, i, i, i, i, p, p, p, p, i, i, i, f,
                                  i, f, f, i, i, ll, i, ll, p, ll, i, i, p, i, p, p],
@@ -107,7 +107,7 @@ def _declare(handle: ctypes.CDLL) -> None:
         "fe_matrix_memory_scratch": [i, i, i, i, i, i],
         "fe_retention": [p, ll, i, i, i, i, f, p, p, i, i, p, f, p, i, p, p, p, i, i, i, i, i, i, i, p, p, p],
         "fe_retention_scratch": [i, i, i, i, i, i],
-        "fe_rglru": [p, ll, i, i, p, p, i, p, p, i, p, p, p, p, p, i, p, p, p, p, i, i, i, i, i, i, p, p, p],
+        "fe_rglru": [p, ll, i, i, p, p, i, p, p, i, p, p, p, p, p, p, p, i, p, p, p, p, i, i, i, i, i, i, p, p, p],
         "fe_rglru_scratch": [i, i, i],
         "fe_rglru_one_launch": [i, i],
         "fe_gemm_tc5_qkv_rope": [p, p, p, p, i, i, i, p, p, f, p, p, p, p, p, p, i, i, i, i, i, i, p, p],
@@ -746,6 +746,9 @@ def qkv_prepare(
     positions: torch.Tensor,
     token_entry: torch.Tensor,
     status: torch.Tensor,
+    q_bias: torch.Tensor | None = None,
+    k_bias: torch.Tensor | None = None,
+    v_bias: torch.Tensor | None = None,
 ) -> None:
     """Normalise, rotate and store one step's queries, keys and values (all optional).
 
@@ -757,7 +760,8 @@ def qkv_prepare(
     tokens' angles; elements [rot_off, rot_off + rot_dims) of every head are rotated (a
     negative ``rot_off`` leaves that side as it is), neighbours paired when ``interleaved``,
     else element j with j + rot_dims / 2.  Head h of a query token starts ``q_head_stride``
-    elements after head h - 1 (0: ``q_dim``).  Queries
+    elements after head h - 1 (0: ``q_dim``).  ``q_bias``, ``k_bias``, ``v_bias`` (32-bit, as long as a
+    token's q, k, v): added before anything else.  Queries
     go to ``q_out`` at token * q_out_strides[0] + head * q_out_strides[1] + q_out_offset,
     keys and values into the pages of ``k_cache`` / ``v_cache``
     [pages, k_heads, page_size, k_dim | v_dim]."""
@@ -772,6 +776,8 @@ def qkv_prepare(
         assert k_cache.shape[1] == k_heads and k_cache.shape[3] == k_dim
         assert v is None or (v_cache is not None and v_cache.shape[3] == v_dim and v_cache.dtype == k_cache.dtype)
     assert table is None or (table.dtype == torch.float32 and table.is_contiguous() and table.shape == (n, rot_dims // 2, 2))
+    for side, bias, size in ((q, q_bias, q_heads * q_dim), (k, k_bias, k_heads * k_dim), (v, v_bias, k_heads * v_dim)):
+        assert bias is None or side is None or (bias.dtype == torch.float32 and bias.is_cuda and bias.is_contiguous() and bias.numel() == size)
     for mode, dims, w in (q_norm, k_norm):
         assert w is None or (w.dtype == torch.float32 and w.is_cuda and w.is_contiguous())
         assert mode != PREP_NORM_WHOLE or w is not None     # the per-head norms take no weight as a weight of ones
@@ -781,7 +787,7 @@ def qkv_prepare(
         lib().fe_qkv_prepare(
             ptr(q), stride(q), int(q_head_stride), int(q_heads), int(q_dim), int(q_norm[0]), int(q_norm[1]), ptr(q_norm[2]), int(q_rot_off),
             ptr(k), stride(k), int(k_heads), int(k_dim), int(k_norm[0]), int(k_norm[1]), ptr(k_norm[2]), int(k_rot_off),
-            ptr(v), stride(v), int(v_dim), code(source), float(eps), ptr(table), int(rot_dims if table is not None else 0),
+            ptr(v), stride(v), int(v_dim), ptr(q_bias), ptr(k_bias), ptr(v_bias), code(source), float(eps), ptr(table), int(rot_dims if table is not None else 0),
             1 if interleaved else 0, ptr(q_out), int(q_out_strides[0]), int(q_out_strides[1]), int(q_out_offset),
             ptr(k_cache), ptr(v_cache), code(cache_dtype), ptr(block_table),
             0 if block_table is None else block_table.shape[1], 0 if k_cache is None else k_cache.shape[2], pages,
@@ -841,7 +847,7 @@ def general_splits(entries: list, groups: int, kv_heads: int, window: int | None
     if window:
         longest = min(longest, window + max(count for _, _, count in entries) + int(keep_first or 0))
     if chunk:
-        longest = min(longest, chunk + max(count for _, _, count in entries))
+        longest = max(start % chunk + count for _, start, count in entries)      # most keys an entry's rows see
     tiles = -(-longest // 64)
     wish = min(slots // max(1, len(entries) * kv_heads), tiles // 2, 32)
     return 1 if wish < 2 else 1 << (wish.bit_length() - 1)
@@ -1248,29 +1254,32 @@ def retention(proj: torch.Tensor, offsets: tuple, q_scale: float, decay: torch.T
 
 
 def rglru(proj: torch.Tensor, y_off: int, x_off: int, conv: torch.Tensor, conv_bias: torch.Tensor, w_r: torch.Tensor,
-          w_i: torch.Tensor, b_r: torch.Tensor, b_i: torch.Tensor, rate: torch.Tensor, state: torch.Tensor,
+          w_i: torch.Tensor, y_bias: torch.Tensor, x_bias: torch.Tensor, b_r: torch.Tensor, b_i: torch.Tensor, rate: torch.Tensor, state: torch.Tensor,
           conv_state: torch.Tensor | None, slots: torch.Tensor, cu_tokens: torch.Tensor, token_entry: torch.Tensor,
           out: torch.Tensor, n_entries: int, max_new: int, status: torch.Tensor) -> None:
     """out_t = S_t gelu_tanh(y_t) over the tokens of every entry, S_t = a S_(t-1) + sqrt(1 - a^2) i u_t per
     channel from and to the 32-bit ``state`` [rows, width]; u = conv(x) + conv_bias, a causal convolution over
     time (``conv`` [taps, width], the last tap weighing the token itself; ``conv_state`` [rows, taps - 1,
     width]: its last inputs); r, i = sigmoid(W u + b) per part of the channels (``w_r``, ``w_i`` [blocks, part,
-    part]), log a = ``rate`` r.  y and x: 32-bit columns of ``proj`` [N, C] from ``y_off``, ``x_off`` on."""
+    part]), log a = ``rate`` r.  y and x: 32-bit columns of ``proj`` [N, C] from ``y_off``, ``x_off`` on plus
+    ``y_bias``, ``x_bias`` [width]."""
     rows, width = state.shape
     taps, n = int(conv.shape[0]), int(out.shape[0])
     blocks, part = int(w_r.shape[0]), int(w_r.shape[1])
-    for name, t in (("conv", conv), ("conv_bias", conv_bias), ("b_r", b_r), ("b_i", b_i), ("rate", rate), ("state", state)):
+    for name, t in (("conv", conv), ("conv_bias", conv_bias), ("y_bias", y_bias), ("x_bias", x_bias), ("b_r", b_r), ("b_i", b_i), ("rate", rate),
+                    ("state", state)):
         _dense(t, name)
         assert t.dtype == torch.float32, name
     _dense(w_r, "w_r"), _dense(w_i, "w_i"), _dense(out, "out")
     assert w_r.shape == w_i.shape == (blocks, part, part) and w_r.dtype == w_i.dtype and blocks * part == width
-    assert conv.shape == (taps, width) and conv_bias.numel() == b_r.numel() == b_i.numel() == rate.numel() == width
+    assert conv.shape == (taps, width) and conv_bias.numel() == y_bias.numel() == x_bias.numel() == width
+    assert b_r.numel() == b_i.numel() == rate.numel() == width
     assert out.shape == (n, width) and slots.dtype == cu_tokens.dtype == token_entry.dtype == torch.int32
     assert taps == 1 or (conv_state.dtype == torch.float32 and conv_state.is_contiguous() and conv_state.shape == (rows, taps - 1, width))
     once = max_new == 1 and n == n_entries and bool(lib().fe_rglru_one_launch(part, code(w_r)))
     scratch = None if once else _state_scratch(out.device, int(lib().fe_rglru_scratch(n, int(n_entries), width)))
     check(lib().fe_rglru(ptr(proj), _columns(proj, max(y_off, x_off) + width), int(y_off), int(x_off), ptr(conv), ptr(conv_bias), taps,
-                         ptr(w_r), ptr(w_i), code(w_r), ptr(b_r), ptr(b_i), ptr(rate), ptr(state), ptr(conv_state), rows, ptr(slots),
+                         ptr(w_r), ptr(w_i), code(w_r), ptr(y_bias), ptr(x_bias), ptr(b_r), ptr(b_i), ptr(rate), ptr(state), ptr(conv_state), rows, ptr(slots),
                          ptr(cu_tokens), ptr(token_entry), ptr(out), code(out), width, part, n, int(n_entries), int(max_new),
                          ptr(scratch), ptr(status), stream()), "rglru")
     if not once:

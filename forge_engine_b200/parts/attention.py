@@ -19,7 +19,7 @@ from ..cache.manager import CacheNeeds, PagedKVSpec
 from ..config.specs import local_name
 from ..errors import ConfigError, UnsupportedShapeError
 from ..ops import native
-from .base import BuildContext, CacheView, Mixer, WeightInfo, build_part, register_part
+from .base import BuildContext, CacheView, Mixer, PositionEncoding, WeightInfo, build_part, register_part
 from .linear import Linear, fused_rows
 
 
@@ -232,9 +232,16 @@ class GQAttention(Mixer):
         self.distance_bias_unscaled = None
         if self.distance_bias is not None and spec.scale > 0:
             self.distance_bias_unscaled = (self.distance_bias.double() / float(spec.scale)).float().contiguous()
+        # a general layer whose keys are only prepared in another way (rotated neighbours, a norm after the
+        # rotation or over the whole projection): bfloat16 scores and values are the plain layer's
+        self.plain_core = (self.general and ctx.dtype == torch.bfloat16 and self.dv == self.d and self.d % 16 == 0 and 16 <= self.d <= 256
+                           and self.nq // self.nkv <= native.ATTN_DECODE_ROWS and self.parts == 1 and self.kv_projection
+                           and self.chunk is None and self.keep_first == 0 and self.softcap is None and self.query_temperature is None
+                           and self.slopes is None and self.distance_bias is None and self.sinks is None
+                           and not self.head_gate and not self.output_gate)
         self._slots = None
         self.plan_key = ("gqa_attention", self.nq, self.nkv, self.d, spec.window) + (
-            ("general", self.dv, self.parts, self.keep_first, self.chunk) if self.general else ())
+            ("general", self.dv, self.parts, self.keep_first, self.chunk) if self.general and not self.plain_core else ())
         self.last_splits = None   # what the last step's decode entries ran with (0: balanced kernel)
 
     @staticmethod
@@ -361,10 +368,12 @@ class GQAttention(Mixer):
         k_cache, v_cache = cache.kv
         table = batch.group_tables[cache.group]
         with self.ctx.section("mixer.qkv_rope_cache"):
-            qkv = self.qkv_proj(x, out_dtype=torch.float32)
+            qkv, bias = self.qkv_proj.sums(x), self.qkv_proj.bias      # the bias joins in the next kernel
             rotary = self.position.rotary()
             angles, rot_dims = None, 0
             if rotary is None:
+                if type(self.position).apply is not PositionEncoding.apply and bias is not None:
+                    qkv, bias = qkv + bias, None           # the encoding rewrites q and k as projected
                 self.position.apply(qkv, nq, nkv, d, batch)
             else:
                 angles, rot_dims = self.position.table(batch), rotary[1]
@@ -384,7 +393,15 @@ class GQAttention(Mixer):
                 table=angles, rot_dims=rot_dims, interleaved=getattr(self.position, "interleaved", False),
                 k_cache=k_cache, v_cache=v_cache, block_table=table, positions=batch.positions,
                 token_entry=batch.token_entry, status=self.ctx.status,
+                q_bias=None if bias is None else bias[:q_end], k_bias=None if bias is None else bias[q_end:k_end],
+                v_bias=None if bias is None else bias[k_end : k_end + nkv * dv],
             )
+        if self.plain_core:
+            # what follows is the plain layer's: its split and balanced decode kernels, its prefill kernels
+            out = torch.empty((n, nq * dv), dtype=k_cache.dtype, device=x.device)
+            with self.ctx.section("mixer.attention"):
+                self._tensor_core_attention(q, k_cache, v_cache, table, batch, out, nq // nkv)
+            return out
         parts = self.parts
         # a differential layer's maps are kept in 32-bit side by side until they are combined
         out = torch.empty((n, nq * parts * dv), dtype=k_cache.dtype if parts == 1 else torch.float32, device=x.device)
@@ -502,7 +519,7 @@ class GQAttention(Mixer):
         rest the prefill kernel; both may run in one step.  (run prefill, run decode, splits
         of the decode kernel - 0: the kernel that spreads all tiles evenly) under this
         mixer's key; layers with the same geometry share it."""
-        if self.general:
+        if self.general and not self.plain_core:
             # the general kernels: (how many blocks share a row tile's keys, whether entries go
             # to the tcgen05 prefill kernel, whether entries go to the general kernel)
             if self.plan_key not in plans:

@@ -65,25 +65,32 @@ class Linear:
                 and x.shape[0] <= native.TC5_MAX_ROWS and self.in_features % 8 == 0 and self.status is not None)
 
     def __call__(self, x: torch.Tensor, out_dtype=None) -> torch.Tensor:
-        out_dtype = out_dtype or x.dtype
+        return self._product(x, out_dtype or x.dtype, self.bias)
+
+    def sums(self, x: torch.Tensor) -> torch.Tensor:
+        """x W^T as 32-bit sums without the bias, for a kernel that adds it itself (the library product
+        takes a 32-bit bias only by writing it to the whole result first)."""
+        return self._product(x, torch.float32, None)
+
+    def _product(self, x: torch.Tensor, out_dtype, bias) -> torch.Tensor:
         n = x.shape[0]
         if self._tc5_ok(x) and out_dtype in (torch.bfloat16, torch.float32):
             out = torch.empty((n, self.out_features), dtype=out_dtype, device=x.device)
             mode = native.TC5_STORE_BF16 if out_dtype == torch.bfloat16 else native.TC5_STORE_F32
-            native.gemm_tc5(x, self.weight, out, mode, self.status, bias=self.bias,
+            native.gemm_tc5(x, self.weight, out, mode, self.status, bias=bias,
                             ksplit=native.tc5_ksplit(self.out_features, self.in_features))
             return out
         if x.dtype == torch.bfloat16 and self.weight.dtype == torch.bfloat16:
             if out_dtype == torch.bfloat16:
-                if self._bias_model is None:
+                if bias is None:
                     return torch.mm(x, self.weight.t())
                 return torch.addmm(self._bias_model, x, self.weight.t())
-            if self.bias is None and _mm_out_dtype_works(x.device):
+            if bias is None and _mm_out_dtype_works(x.device):
                 return torch.mm(x, self.weight.t(), out_dtype=torch.float32)
-            if self.bias is not None and out_dtype == torch.float32 and _addmm_out_dtype_works(x.device):
-                return torch.addmm(self.bias, x, self.weight.t(), out_dtype=torch.float32)
+            if bias is not None and out_dtype == torch.float32 and _addmm_out_dtype_works(x.device):
+                return torch.addmm(bias, x, self.weight.t(), out_dtype=torch.float32)
         out = torch.empty((n, self.out_features), dtype=out_dtype, device=x.device)
-        native.gemm_simt(x, self.weight, out, self.bias)
+        native.gemm_simt(x, self.weight, out, bias)
         return out
 
 

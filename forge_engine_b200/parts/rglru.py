@@ -5,7 +5,8 @@ bias per channel.  The channels fall into equal parts; in each r = sigmoid(R u +
 log a = -strength r softplus(lam); S_t = a S_(t-1) + sqrt(1 - a^2) i u_t per channel, zero at the start;
 the update is W_o (S y).
 
-One fused projection gives y and x as 32-bit sums; convolution, both gate products, recurrence and gate
+One fused projection gives y and x as 32-bit sums (their biases are added by the kernels that read them);
+convolution, both gate products, recurrence and gate
 are one kernel where every entry brings one token, else three (tiles of tokens side by side, their states
 chained, the outputs).  A request keeps S and the convolution's last taps - 1 inputs, 32-bit.
 """
@@ -32,12 +33,12 @@ class RGLRU(Mixer):
         self.width, self.taps = spec.width, spec.taps
         name = lambda canonical: local_name(spec, canonical)  # noqa: E731
         rows = [self.width, self.width]
-        self.proj = Linear(fused_rows(weights, [name("y"), name("x")], rows), fused_rows(weights, [name("y.b"), name("x.b")], rows),
-                           status=ctx.status)
+        self.proj = Linear(fused_rows(weights, [name("y"), name("x")], rows), status=ctx.status)
         vector = lambda key: weights[name(key)].to(device=ctx.device, dtype=torch.float32).reshape(-1).contiguous()  # noqa: E731
         # stored [channels, taps]; the kernels read a tap's weights side by side
         self.conv = weights[name("conv")].to(device=ctx.device, dtype=torch.float32).t().contiguous()
-        self.conv_bias, self.r_bias, self.i_bias = vector("conv.b"), vector("ra.b"), vector("ri.b")
+        self.y_bias, self.x_bias, self.conv_bias = vector("y.b"), vector("x.b"), vector("conv.b")
+        self.r_bias, self.i_bias = vector("ra.b"), vector("ri.b")
         self.r_weight, self.i_weight = weights[name("ra")].contiguous(), weights[name("ri")].contiguous()
         if self.r_weight.dtype != self.i_weight.dtype:
             self.r_weight, self.i_weight = self.r_weight.float(), self.i_weight.float()
@@ -73,11 +74,11 @@ class RGLRU(Mixer):
     def attend(self, x, batch, cache: CacheView):
         """Everything but the output projection: S y [N, width]."""
         with self.ctx.section("mixer.projection"):
-            proj = self.proj(x, out_dtype=torch.float32)
+            proj = self.proj.sums(x)
         out = torch.empty((x.shape[0], self.width), dtype=self.ctx.dtype, device=x.device)
         with self.ctx.section("mixer.recurrence"):
-            native.rglru(proj, 0, self.width, self.conv, self.conv_bias, self.r_weight, self.i_weight, self.r_bias, self.i_bias,
-                         self.rate, cache.state, cache.states.get("conv"), batch.slots, batch.cu_tokens, batch.token_entry, out,
+            native.rglru(proj, 0, self.width, self.conv, self.conv_bias, self.r_weight, self.i_weight, self.y_bias, self.x_bias,
+                         self.r_bias, self.i_bias, self.rate, cache.state, cache.states.get("conv"), batch.slots, batch.cu_tokens, batch.token_entry, out,
                          batch.n_entries, batch.max_new, self.ctx.status)
         return out
 

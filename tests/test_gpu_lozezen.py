@@ -579,6 +579,8 @@ def test_rglru_kernels(blocks, part, taps, counts, weights):
     rand = lambda *shape: torch.randn(*shape, generator=gen, dtype=torch.float64)  # noqa: E731
     n, width = sum(counts), blocks * part
     proj, conv, conv_bias = rand(n, 2 * width), 0.6 * rand(width, taps), 0.5 * rand(width)
+    bias, sums = 0.7 * rand(2 * width), proj
+    proj = sums + bias
     w = [(rand(blocks, part, part) * 1.5 / math.sqrt(part)).to(torch.bfloat16).double() for _ in range(2)]
     b = [0.5 * rand(width) for _ in range(2)]
     rate = -torch.exp(3.0 * rand(width) - 3.0)
@@ -599,8 +601,8 @@ def test_rglru_kernels(blocks, part, taps, counts, weights):
         want_history[s] = rows[len(rows) - (taps - 1):]
     dev = lambda t: t.float().cuda().contiguous()  # noqa: E731
     got_state, got_history, out, status = dev(state), dev(history), torch.empty(n, width, device="cuda"), status_word()
-    native.rglru(dev(proj), 0, width, dev(conv.T), dev(conv_bias), w[0].to(weights).cuda(), w[1].to(weights).cuda(), dev(b[0]), dev(b[1]),
-                 dev(rate), got_state, got_history if taps > 1 else None, slots, cu, entry, out, len(counts), max(counts), status)
+    native.rglru(dev(sums), 0, width, dev(conv.T), dev(conv_bias), w[0].to(weights).cuda(), w[1].to(weights).cuda(), dev(bias[:width]),
+                 dev(bias[width:]), dev(b[0]), dev(b[1]), dev(rate), got_state, got_history if taps > 1 else None, slots, cu, entry, out, len(counts), max(counts), status)
     assert int(status.item()) == 0 and not native.damaged_canaries()
     tol = 2e-5 if weights == torch.float32 else 1e-4        # u as a sum of two bfloat16 numbers
     assert float((out.cpu() - want).abs().max()) <= tol * max(1.0, float(want.abs().max()))
