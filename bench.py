@@ -690,15 +690,16 @@ def design_compare(args) -> int:
         })
         # Lozezen at the same sizes: the gated linear recurrent unit as wide as the stream in parts of 256
         # (4 taps), biased window attention with half the head rotated at Qwen3's head sizes, and chunked
-        # attention (chunks as long as the windows) beside retention with the other recurrences' states;
+        # attention (chunks of one and a half windows) beside retention with the other recurrences' states;
         # the dense feed-forward of ff.
         z_unit = {"type": "rglru", "mlp": mlp, "mixer": {"width": W, "blocks": W // 256, "conv": 4}}
         z_window = {"type": "attention", "mlp": mlp, "mixer": {
             "heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window},
             "rot": {"base": 1e6, "dims": D // 2, "scaling": {"factor": 2.0}}}}
+        chunk = window * 3 // 2
         z_parallel = {"type": "parallel", "mlp": mlp, "mixer": {
             "left_scale": 0.5, "right_scale": 0.5,
-            "left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": window}},
+            "left": {"heads": H, "kv_heads": G, "dim": D, "vdim": D, "scale": D ** -0.5, "mask": {"size": chunk}},
             "right": dict(rec, heads=H, rot={"base": 1e6, "dims": rec["dim"]}, decay=[1.0 - 2.0 ** (-5 - 3 * h / H) for h in range(H)])}}
 
         def lozezen(kinds):
@@ -738,8 +739,8 @@ def design_compare(args) -> int:
             8 * H * rec["dim"] * rec["vdim"] * CONTEXT, mixer_cost["zofadra-recurrence"][1])
         mixer_cost["lofuvik-parallel"] = mixer_cost["qwen3"]
         mixer_cost["lozezen-attention"] = mixer_cost["qwen3-window"]
-        # every query sees its own chunk up to itself; the token decoded here is one of a chunk's first
-        mixer_cost["lozezen-parallel"] = (4 * H * D * sum(i % window + 1 for i in range(CONTEXT)), batch * (CONTEXT % window + 24) * G * 2 * D * 2)
+        # every query sees its own chunk up to itself; some 24 tokens have been decoded on average
+        mixer_cost["lozezen-parallel"] = (4 * H * D * sum(i % chunk + 1 for i in range(CONTEXT)), batch * (CONTEXT % chunk + 24) * G * 2 * D * 2)
         # both gates' products; in decoding their matrices, the states and the convolution's inputs
         mixer_cost["lozezen-rglru"] = (4 * W * 256 * CONTEXT, 2 * W * 256 * 2 + batch * W * 4 * (2 + 2 * 3 + 2) + batch * W * 2)
         # what a prompt must move: x and y (32-bit) in, the heads (bfloat16) out

@@ -10,7 +10,7 @@
 // x and y are 32-bit sums of the projection.  Everything here is 32-bit; with bfloat16 gate matrices u
 // enters their product as the sum of two bfloat16 numbers (the rounded one and the rounded remainder).
 //
-//   rglru_gates   tiles of RM tokens of the step (whatever entries they belong to) x NC channels of one
+//   rglru_gates   tiles of 64 tokens of the step (whatever entries they belong to) x 64 channels of one
 //                 part: convolution, both products, gates, and the recurrence from zero inside the tile.
 //                 Leaves, per token, h (the state if the tile had started from zero, or the entry began
 //                 inside it) and the product of the a since then, so that S = h + prod * S_in.
@@ -50,7 +50,17 @@ struct Rglru {
 #define RG_WP (RG_KC + 8)   // pitch of a bfloat16 tile
 #define RG_FP (RG_KC + 4)   // pitch of a 32-bit tile
 
-__device__ __forceinline__ float rg_sigmoid(float z) { return __fdividef(1.f, 1.f + __expf(-z)); }
+__device__ __forceinline__ float rg_exp2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rg_reciprocal(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float rg_sigmoid(float z) { return rg_reciprocal(1.f + rg_exp2(-1.4426950408889634f * z)); }
 __device__ __forceinline__ float rg_gelu(float z) {
   // 0.5 (1 + tanh(t)) = sigmoid(2 t)
   return z * rg_sigmoid(1.5957691216057308f * (z + 0.044715f * z * z * z));
@@ -68,7 +78,7 @@ __device__ __forceinline__ float rg_one_minus_exp(float x, float e) {
 }
 __device__ __forceinline__ float rg_sqrt(float x) {
   float y;
-  asm("sqrt.approx.f32 %0, %1;" : "=f"(y) : "f"(x));
+  asm("sqrt.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
 // a and the input's factor sqrt(1 - a^2) i from the gates' sums
@@ -120,27 +130,25 @@ __device__ __forceinline__ void rg_load_weight(float* dst, int pitch, const floa
 // rglru_gates
 // ---------------------------------------------------------------------------
 #define RG_RM 64            // tokens of a tile
+#define RG_NC RG_KC         // channels of a block's tile: one chunk of its part
+#define RG_THREADS 256
 
-template <typename TW, int NC>
+template <typename TW>
 struct RgShape {
   static constexpr bool MMA = sizeof(TW) == 2;
-  static constexpr int THREADS = 4 * NC;
+  static constexpr int BLOCKS = MMA ? 3 : 1;                                           // an SM's share, by registers
   static constexpr int WPITCH = MMA ? RG_WP : RG_FP;
-  static constexpr size_t W_BYTES = sizeof(TW) * 2 * NC * WPITCH;                      // both gates, one stage
+  static constexpr size_t W_BYTES = sizeof(TW) * 2 * RG_NC * WPITCH;                   // both gates, one stage
   static constexpr size_t A_BYTES = MMA ? sizeof(bf16) * 2 * RG_RM * RG_WP : sizeof(float) * RG_RM * RG_FP;
-  static constexpr size_t U_BYTES = sizeof(float) * RG_RM * NC;
-  static constexpr size_t GATE_BYTES = sizeof(float) * 2 * RG_RM * (NC + 1);           // over the stages, afterwards
-  static size_t stages(int taps) {
-    const size_t s = 2 * (W_BYTES + sizeof(float) * (RG_RM + taps - 1) * RG_KC);
-    return s > GATE_BYTES ? s : GATE_BYTES;
-  }
-  static size_t bytes(int taps) { return stages(taps) + A_BYTES + U_BYTES; }
+  static_assert(2 * W_BYTES >= sizeof(float) * 2 * RG_RM * (RG_NC + 1), "the gates' sums lie over the matrices' stages");
+  static size_t bytes(int taps) { return A_BYTES + 2 * W_BYTES + sizeof(float) * (RG_RM + taps - 1) * RG_KC; }
 };
 
 // TAPS: 4, or 0 for any number.
-template <typename TW, int NC, int TAPS>
-__global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int stage_bytes, int* status) {
-  using Shape = RgShape<TW, NC>;
+template <typename TW, int TAPS>
+__global__ void __launch_bounds__(RG_THREADS, RgShape<TW>::BLOCKS) rglru_gates_kernel(const Rglru p, int* status) {
+  using Shape = RgShape<TW>;
+  constexpr int NC = RG_NC;
   extern __shared__ __align__(16) unsigned char raw[];
   __shared__ int since[RG_RM], slot_of[RG_RM];       // tokens since the entry's first; the request's row (-1: none)
   __shared__ float seg_h[4][NC], seg_p[4][NC];
@@ -150,10 +158,9 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
   const int n0 = blockIdx.x * NC, block = blockIdx.y, t0 = blockIdx.z * RG_RM;
   const int part = p.part, taps = TAPS > 0 ? TAPS : p.taps, back = taps - 1;
   const int rows = min(RG_RM, p.n_tokens - t0);
-  TW* ws = reinterpret_cast<TW*>(raw);                                         // [2 stages][2 gates][NC][pitch]
-  float* xs = reinterpret_cast<float*>(raw + 2 * Shape::W_BYTES);              // [2 stages][RM + back][KC]
-  unsigned char* as = raw + stage_bytes;                                       // u: hi and lo [RM][RG_WP], or 32-bit [RM][RG_FP]
-  float* us = reinterpret_cast<float*>(as + Shape::A_BYTES);                   // [RM][NC]: u of the block's own channels
+  unsigned char* as = raw;                                                     // u: hi and lo [RM][RG_WP], or 32-bit [RM][RG_FP]
+  TW* ws = reinterpret_cast<TW*>(raw + Shape::A_BYTES);                        // [2 stages][2 gates][NC][pitch]
+  float* xs = reinterpret_cast<float*>(raw + Shape::A_BYTES + 2 * Shape::W_BYTES);       // [RM + back][KC]
   const TW* wr = (const TW*)p.wr + (size_t)block * part * part;
   const TW* wi = (const TW*)p.wi + (size_t)block * part * part;
   const int x0 = block * part;                       // the part's first channel
@@ -162,16 +169,16 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
     TW* w = ws + stage * 2 * NC * Shape::WPITCH;
     rg_load_weight(w, Shape::WPITCH, wr, part, n0, NC, k0, RG_KC);
     rg_load_weight(w + NC * Shape::WPITCH, Shape::WPITCH, wi, part, n0, NC, k0, RG_KC);
-    float* x = xs + stage * (RG_RM + back) * RG_KC;
+    float* x = xs;
     const float* src = p.proj + p.x_off + x0 + k0;
     if (wide) {
-      for (int i = tid; i < (RG_RM + back) * (RG_KC / 4); i += Shape::THREADS) {
+      for (int i = tid; i < (RG_RM + back) * (RG_KC / 4); i += RG_THREADS) {
         const int r = i / (RG_KC / 4), c = (i - r * (RG_KC / 4)) * 4, t = t0 + r - back;
         const bool has = t >= 0 && t < p.n_tokens && k0 + c < part;
         cp_async16(x + r * RG_KC + c, has ? src + (size_t)t * p.ld + c : p.proj, has);
       }
     } else {
-      for (int i = tid; i < (RG_RM + back) * RG_KC; i += Shape::THREADS) {
+      for (int i = tid; i < (RG_RM + back) * RG_KC; i += RG_THREADS) {
         const int r = i / RG_KC, c = i - r * RG_KC, t = t0 + r - back;
         const bool has = t >= 0 && t < p.n_tokens && k0 + c < part;
         rg_copy4(x + r * RG_KC + c, has ? src + (size_t)t * p.ld + c : p.proj, has);
@@ -179,7 +186,10 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
     }
     cp_commit();
   };
-  load(0, 0);
+  // the part's chunks of channels, the block's own last: its u then stays where the products read it
+  const int chunks = (part + RG_KC - 1) / RG_KC, mine = n0 / RG_KC;
+  auto chunk_at = [&](int i) { return (i + mine + 1 < chunks ? i + mine + 1 : i + mine + 1 - chunks) * RG_KC; };
+  load(chunk_at(0), 0);
   int n = 1 << 30;                                   // past the last token: as if far inside an entry
   if (tid < RG_RM) {
     int s = -1;
@@ -208,20 +218,16 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
   const int rw = warp & 3, cw = warp >> 2;
   const int fr = (tid & 15) * 4, fc = tid >> 4;      // 32-bit: rows fr .. fr + 3, channels fc + NC / 4 * e
   // the convolution: a thread takes two channels of PER neighbouring tokens
-  constexpr int PER = RG_RM / (Shape::THREADS / 32);
+  constexpr int PER = RG_RM / (RG_THREADS / 32);
   const int c2 = lane * 2, r0 = warp * PER;
 
-  for (int k0 = 0, stage = 0; k0 < part; k0 += RG_KC, stage ^= 1) {
-    if (k0 + RG_KC < part) {
-      load(k0 + RG_KC, stage ^ 1);
-      cp_wait<1>();
-    } else {
-      cp_wait<0>();
-    }
+  for (int i = 0; i < chunks; ++i) {
+    const int k0 = chunk_at(i), stage = i & 1;
+    cp_wait<0>();
     __syncthreads();
     {
-      const float* x = xs + stage * (RG_RM + back) * RG_KC + c2;
-      const int ch = x0 + k0 + c2, own = k0 + c2 - n0;
+      const float* x = xs + c2;
+      const int ch = x0 + k0 + c2;
       const bool live0 = k0 + c2 < part, live1 = k0 + c2 + 1 < part;
       auto put = [&](int r, float u0, float u1) {
         if constexpr (Shape::MMA) {
@@ -233,7 +239,6 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
         } else {
           *reinterpret_cast<float2*>(reinterpret_cast<float*>(as) + r * RG_FP + c2) = make_float2(u0, u1);
         }
-        if (own >= 0 && own < NC) *reinterpret_cast<float2*>(us + r * NC + own) = make_float2(u0, u1);
       };
       if (TAPS > 0 && !edge) {
         // every tap inside the step: the projection's bias goes through the taps' sum
@@ -280,6 +285,7 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
       }
     }
     __syncthreads();
+    if (i + 1 < chunks) load(chunk_at(i + 1), stage ^ 1);      // while the products run
     const TW* w = ws + stage * 2 * NC * Shape::WPITCH;
     if constexpr (Shape::MMA) {
       const bf16* hi = reinterpret_cast<const bf16*>(as);
@@ -319,11 +325,11 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
           }
       }
     }
-    __syncthreads();
   }
+  __syncthreads();
 
-  // the sums of both gates, [gate][RM][NC + 1], over the stages
-  float* gates = reinterpret_cast<float*>(raw);
+  // the sums of both gates, [gate][RM][NC + 1], over the matrices
+  float* gates = reinterpret_cast<float*>(ws);
   constexpr int GP = NC + 1;
 #pragma unroll
   for (int g = 0; g < 2; ++g)
@@ -357,7 +363,14 @@ __global__ void __launch_bounds__(4 * NC) rglru_gates_kernel(const Rglru p, int 
         s = 0.f, q = 1.f;
         fresh = min(fresh, i);
       }
-      s = fmaf(a, s, scale * us[r * NC + c]);
+      float u;
+      if constexpr (Shape::MMA) {
+        const bf16* hi = reinterpret_cast<const bf16*>(as) + r * RG_WP + c;
+        u = __bfloat162float(hi[0]) + __bfloat162float(hi[RG_RM * RG_WP]);
+      } else {
+        u = reinterpret_cast<const float*>(as)[r * RG_FP + c];
+      }
+      s = fmaf(a, s, scale * u);
       q *= a;
       h[i] = s, prod[i] = q;
     }
@@ -448,6 +461,7 @@ __global__ void __launch_bounds__(256) rglru_out_kernel(const Rglru p) {
 // rglru_step
 // ---------------------------------------------------------------------------
 #define RG_SM 16            // entries of a tile
+#define RG_HIST 7           // earlier inputs of the convolution held in registers
 
 template <int NC>
 static size_t rg_step_smem(int part) {
@@ -475,40 +489,70 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
   cp_commit();
   for (int i = tid; i < 2 * RG_SM * pitch; i += THREADS) hi[i] = __float2bfloat16_rn(0.f);
   pdl_wait();
-  cluster.sync();                                     // every block of the cluster is there, its tiles are zero
+  // a thread's four (entry, channel) places; what they need is fetched before anything waits for it
   const int x0 = block * part, cols = min(NC, part - n0);
   const int peers = (int)cluster.num_blocks();
-  for (int i = tid; i < RG_SM * NC; i += THREADS) {
-    const int r = i / NC, c = i - r * NC;
-    float u = 0.f;
-    if (r < rows && c < cols) {
-      const int ch = x0 + n0 + c, slot = p.slots[t0 + r];
-      const float x = p.proj[(size_t)(t0 + r) * p.ld + p.x_off + ch] + p.x_bias[ch];
-      u = p.conv_b[ch];
-      if (slot >= 0 && slot < p.state_rows) {
-        // the oldest input leaves the history, the others move up
-        float* st = p.conv_state + (size_t)slot * back * p.width + ch;
+  const int c = tid % NC, ch = x0 + n0 + c;
+  const bool has = c < cols;
+  float u[4], y[4], before[4], fresh[4], hist[4][RG_HIST];
+  int slot[4];
+  const float br = has ? p.br[ch] : 0.f, bi = has ? p.bi[ch] : 0.f, rate = has ? p.rate[ch] : 0.f;
+  const float conv_b = has ? p.conv_b[ch] : 0.f, x_bias = has ? p.x_bias[ch] : 0.f, y_bias = has ? p.y_bias[ch] : 0.f;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int r = tid / NC + 4 * k;
+    slot[k] = has && r < rows ? p.slots[t0 + r] : -1;
+    if (has && r < rows && (slot[k] < 0 || slot[k] >= p.state_rows)) {
+      atomicOr(status, FE_STATUS_BAD_PAGE);
+      slot[k] = -1;
+    }
+    u[k] = y[k] = before[k] = fresh[k] = 0.f;
+    if (slot[k] < 0) continue;
+    const float* row = p.proj + (size_t)(t0 + r) * p.ld + ch;
+    fresh[k] = row[p.x_off] + x_bias, y[k] = row[p.y_off] + y_bias;
+    before[k] = p.state[(size_t)slot[k] * p.width + ch];
+    if (back <= RG_HIST) {
+#pragma unroll
+      for (int j = 0; j < RG_HIST; ++j)
+        hist[k][j] = j < back ? p.conv_state[((size_t)slot[k] * back + j) * p.width + ch] : 0.f;
+    }
+  }
+  cluster.sync();                                     // every block of the cluster is there, its tiles are zero
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    const int r = tid / NC + 4 * k;
+    if (slot[k] >= 0) {
+      // the oldest input leaves the history, the others move up
+      float* st = p.conv_state + (size_t)slot[k] * back * p.width + ch;
+      u[k] = conv_b;
+      if (back <= RG_HIST) {
+#pragma unroll
+        for (int j = 0; j < RG_HIST; ++j) {
+          if (j < back) {
+            u[k] = fmaf(p.conv_w[(size_t)j * p.width + ch], hist[k][j], u[k]);
+            if (j > 0) st[(size_t)(j - 1) * p.width] = hist[k][j];
+          }
+        }
+      } else {
         for (int j = 0; j < back; ++j) {
           const float v = st[(size_t)j * p.width];
-          u = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u);
+          u[k] = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u[k]);
           if (j > 0) st[(size_t)(j - 1) * p.width] = v;
         }
-        if (back > 0) st[(size_t)(back - 1) * p.width] = x;
-      } else {
-        atomicOr(status, FE_STATUS_BAD_PAGE);
       }
-      u = fmaf(p.conv_w[(size_t)back * p.width + ch], x, u);
+      if (back > 0) st[(size_t)(back - 1) * p.width] = fresh[k];
+      u[k] = fmaf(p.conv_w[(size_t)back * p.width + ch], fresh[k], u[k]);
     }
-    us[r * GP + c] = u;
+    us[r * GP + c] = u[k];
   }
   __syncthreads();
   // channels of a part in pairs: n0 is even
   for (int i = tid; i < rows * (NC / 2); i += THREADS) {
-    const int r = i / (NC / 2), c = (i - r * (NC / 2)) * 2;
-    if (c >= cols) continue;
+    const int r = i / (NC / 2), c2 = (i - r * (NC / 2)) * 2;
+    if (c2 >= cols) continue;
     unsigned h, l;
-    split2(us[r * GP + c], us[r * GP + c + 1], h, l);       // past the last channel: zero
-    const int at = r * pitch + n0 + c;
+    split2(us[r * GP + c2], us[r * GP + c2 + 1], h, l);     // past the last channel: zero
+    const int at = r * pitch + n0 + c2;
     for (int peer = 0; peer < peers; ++peer) {
       bf16* dst = cluster.map_shared_rank(hi, peer);
       *reinterpret_cast<unsigned*>(dst + at) = h;
@@ -540,17 +584,15 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
         gates[(g * RG_SM + (lane >> 2) + 8 * (e >> 1)) * GP + c0 + j * 8 + (lane & 3) * 2 + (e & 1)] = acc[j][e];
   }
   __syncthreads();
-  for (int i = tid; i < rows * NC; i += THREADS) {
-    const int r = i / NC, c = i - r * NC;
-    if (c >= cols) continue;
-    const int ch = x0 + n0 + c, slot = p.slots[t0 + r];
-    if (slot < 0 || slot >= p.state_rows) continue;
+#pragma unroll
+  for (int k = 0; k < 4; ++k) {
+    if (slot[k] < 0) continue;
+    const int r = tid / NC + 4 * k;
     float a, scale;
-    rg_gates(gates[r * GP + c] + p.br[ch], gates[(RG_SM + r) * GP + c] + p.bi[ch], p.rate[ch], &a, &scale);
-    float* cell = p.state + (size_t)slot * p.width + ch;
-    const float s = fmaf(a, *cell, scale * us[r * GP + c]);
-    *cell = s;
-    ((TO*)p.out)[(size_t)(t0 + r) * p.width + ch] = from_float<TO>(s * rg_gelu(p.proj[(size_t)(t0 + r) * p.ld + p.y_off + ch] + p.y_bias[ch]));
+    rg_gates(gates[r * GP + c] + br, gates[(RG_SM + r) * GP + c] + bi, rate, &a, &scale);
+    const float s = fmaf(a, before[k], scale * u[k]);
+    p.state[(size_t)slot[k] * p.width + ch] = s;
+    ((TO*)p.out)[(size_t)(t0 + r) * p.width + ch] = from_float<TO>(s * rg_gelu(y[k]));
   }
 }
 
@@ -573,14 +615,14 @@ static int rg_step_cols(int part) {
   return 0;
 }
 
-template <typename TW, int NC, int TAPS>
+template <typename TW, int TAPS>
 static int rg_launch_gates(const Rglru& p, int* status, cudaStream_t stream) {
-  using Shape = RgShape<TW, NC>;
+  using Shape = RgShape<TW>;
   const size_t smem = Shape::bytes(p.taps);
   if (smem > 220 * 1024) return FE_ERR_TOO_LARGE;
-  cudaFuncSetAttribute(rglru_gates_kernel<TW, NC, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
-  const dim3 grid((p.part + NC - 1) / NC, p.width / p.part, (p.n_tokens + RG_RM - 1) / RG_RM);
-  return fe_launch_dependent(rglru_gates_kernel<TW, NC, TAPS>, grid, dim3(Shape::THREADS), smem, stream, p, (int)Shape::stages(p.taps), status);
+  cudaFuncSetAttribute(rglru_gates_kernel<TW, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+  const dim3 grid((p.part + RG_NC - 1) / RG_NC, p.width / p.part, (p.n_tokens + RG_RM - 1) / RG_RM);
+  return fe_launch_dependent(rglru_gates_kernel<TW, TAPS>, grid, dim3(RG_THREADS), smem, stream, p, status);
 }
 
 // Whether a step in which every entry brings one token is one launch.
@@ -616,10 +658,8 @@ FE_EXPORT int fe_rglru(const float* proj, long long ld, int y_off, int x_off, co
   p.prod = p.h + (size_t)tokens * pitch;
   p.carry = p.prod + (size_t)tokens * pitch;
   p.init = p.carry + (tiles + 1) * pitch;
-  static const int nc = getenv("RG_NC") ? atoi(getenv("RG_NC")) : 128;
-  if (weight_dtype == FE_DTYPE_BF16 && nc == 128 && part >= 128) rc = taps == 4 ? rg_launch_gates<bf16, 128, 4>(p, status, stream) : rg_launch_gates<bf16, 128, 0>(p, status, stream);
-  else if (weight_dtype == FE_DTYPE_BF16) rc = taps == 4 ? rg_launch_gates<bf16, 64, 4>(p, status, stream) : rg_launch_gates<bf16, 64, 0>(p, status, stream);
-  else if (weight_dtype == FE_DTYPE_F32) rc = taps == 4 ? rg_launch_gates<float, 64, 4>(p, status, stream) : rg_launch_gates<float, 64, 0>(p, status, stream);
+  if (weight_dtype == FE_DTYPE_BF16) rc = taps == 4 ? rg_launch_gates<bf16, 4>(p, status, stream) : rg_launch_gates<bf16, 0>(p, status, stream);
+  else if (weight_dtype == FE_DTYPE_F32) rc = taps == 4 ? rg_launch_gates<float, 4>(p, status, stream) : rg_launch_gates<float, 0>(p, status, stream);
   if (rc) return rc;
   rc = fe_launch_dependent(rglru_chain_kernel, dim3((width + 63) / 64, entries), dim3(64), 0, stream, p);
   if (rc) return rc;
