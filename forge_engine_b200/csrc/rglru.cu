@@ -487,17 +487,20 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
   rg_load_weight(ws, pitch, (const bf16*)p.wr + (size_t)block * part * part, part, n0, NC, 0, k_all);
   rg_load_weight(ws + NC * pitch, pitch, (const bf16*)p.wi + (size_t)block * part * part, part, n0, NC, 0, k_all);
   cp_commit();
-  for (int i = tid; i < 2 * RG_SM * pitch; i += THREADS) hi[i] = __float2bfloat16_rn(0.f);
-  pdl_wait();
+  for (int i = tid; i < RG_SM * pitch / 4; i += THREADS) reinterpret_cast<uint4*>(hi)[i] = make_uint4(0u, 0u, 0u, 0u);
+  auto arrived = cluster.barrier_arrive();            // this block is there and its tiles are zero
   // a thread's four (entry, channel) places; what they need is fetched before anything waits for it
   const int x0 = block * part, cols = min(NC, part - n0);
   const int peers = (int)cluster.num_blocks();
   const int c = tid % NC, ch = x0 + n0 + c;
   const bool has = c < cols;
-  float u[4], y[4], before[4], fresh[4], hist[4][RG_HIST];
+  float u[4], y[4], before[4], fresh[4], hist[4][RG_HIST], taps_w[RG_HIST + 1];
   int slot[4];
   const float br = has ? p.br[ch] : 0.f, bi = has ? p.bi[ch] : 0.f, rate = has ? p.rate[ch] : 0.f;
   const float conv_b = has ? p.conv_b[ch] : 0.f, x_bias = has ? p.x_bias[ch] : 0.f, y_bias = has ? p.y_bias[ch] : 0.f;
+#pragma unroll
+  for (int j = 0; j < RG_HIST + 1; ++j) taps_w[j] = has && j <= back ? p.conv_w[(size_t)j * p.width + ch] : 0.f;
+  pdl_wait();
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const int r = tid / NC + 4 * k;
@@ -517,7 +520,6 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
         hist[k][j] = j < back ? p.conv_state[((size_t)slot[k] * back + j) * p.width + ch] : 0.f;
     }
   }
-  cluster.sync();                                     // every block of the cluster is there, its tiles are zero
 #pragma unroll
   for (int k = 0; k < 4; ++k) {
     const int r = tid / NC + 4 * k;
@@ -529,23 +531,27 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
 #pragma unroll
         for (int j = 0; j < RG_HIST; ++j) {
           if (j < back) {
-            u[k] = fmaf(p.conv_w[(size_t)j * p.width + ch], hist[k][j], u[k]);
+            u[k] = fmaf(taps_w[j], hist[k][j], u[k]);
             if (j > 0) st[(size_t)(j - 1) * p.width] = hist[k][j];
           }
         }
+#pragma unroll
+        for (int j = 0; j < RG_HIST + 1; ++j)
+          if (j == back) u[k] = fmaf(taps_w[j], fresh[k], u[k]);
       } else {
         for (int j = 0; j < back; ++j) {
           const float v = st[(size_t)j * p.width];
           u[k] = fmaf(p.conv_w[(size_t)j * p.width + ch], v, u[k]);
           if (j > 0) st[(size_t)(j - 1) * p.width] = v;
         }
+        u[k] = fmaf(p.conv_w[(size_t)back * p.width + ch], fresh[k], u[k]);
       }
       if (back > 0) st[(size_t)(back - 1) * p.width] = fresh[k];
-      u[k] = fmaf(p.conv_w[(size_t)back * p.width + ch], fresh[k], u[k]);
     }
     us[r * GP + c] = u[k];
   }
   __syncthreads();
+  cluster.barrier_wait(std::move(arrived));           // every block of the cluster is there
   // channels of a part in pairs: n0 is even
   for (int i = tid; i < rows * (NC / 2); i += THREADS) {
     const int r = i / (NC / 2), c2 = (i - r * (NC / 2)) * 2;
@@ -565,7 +571,8 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
   {
     // a warp takes 16 channels of one gate
     const int g = warp / (NC / 16), c0 = (warp - g * (NC / 16)) * 16;
-    float acc[2][4] = {};
+    float acc[4][4] = {};        // products of the rounded numbers, then of the remainders
+#pragma unroll 4
     for (int kk = 0; kk < k_all / 16; ++kk) {
       unsigned ah[4], al[4], b0, b1, b2, b3;
       const int a_at = (lane & 15) * pitch + kk * 16 + (lane >> 4) * 8;
@@ -574,14 +581,14 @@ __global__ void __launch_bounds__(4 * NC) rglru_step_kernel(const Rglru p, int* 
       ldsm4(b0, b1, b2, b3, ws + (g * NC + c0 + (lane >> 4) * 8 + (lane & 7)) * pitch + kk * 16 + ((lane >> 3) & 1) * 8);
       mma16816(acc[0], ah, b0, b1);
       mma16816(acc[1], ah, b2, b3);
-      mma16816(acc[0], al, b0, b1);
-      mma16816(acc[1], al, b2, b3);
+      mma16816(acc[2], al, b0, b1);
+      mma16816(acc[3], al, b2, b3);
     }
 #pragma unroll
     for (int j = 0; j < 2; ++j)
 #pragma unroll
       for (int e = 0; e < 4; ++e)
-        gates[(g * RG_SM + (lane >> 2) + 8 * (e >> 1)) * GP + c0 + j * 8 + (lane & 3) * 2 + (e & 1)] = acc[j][e];
+        gates[(g * RG_SM + (lane >> 2) + 8 * (e >> 1)) * GP + c0 + j * 8 + (lane & 3) * 2 + (e & 1)] = acc[j][e] + acc[2 + j][e];
   }
   __syncthreads();
 #pragma unroll

@@ -666,6 +666,65 @@ def test_retention_kernels(heads, dk, dv, rot, interleaved, counts):
     assert float((got_state.cpu() - want_state).abs().max()) <= 3e-5 * max(1.0, float(want_state.abs().max()))
 
 
+@pytest.mark.parametrize("interleaved", (False, True))
+@pytest.mark.parametrize("mode", ("none", "before", "after"))
+@pytest.mark.parametrize("heads, kv, dim, vdim, rot", ((4, 2, 64, 64, 64), (4, 2, 64, 32, 16), (3, 3, 24, 20, 8), (6, 1, 128, 128, 96), (2, 1, 48, 100, 0),
+                                                       (2, 2, 10, 7, 6), (2, 1, 160, 64, 40), (1, 1, 256, 256, 256), (3, 1, 20, 16, 12)))
+def test_preparation_of_queries_keys_and_values(heads, kv, dim, vdim, rot, mode, interleaved):
+    """Bias, norm per head (before or after the rotation), rotation, pages: by heads in registers where the
+    sizes keep to fours, else by heads in shared memory; the queries written where they were read."""
+    from forge_engine_b200.ops import native
+
+    gen = torch.Generator().manual_seed(dim + rot)
+    rand = lambda *shape: torch.randn(*shape, generator=gen, dtype=torch.float64)  # noqa: E731
+    n, page_size, pages = 13, 4, 9
+    sizes = [heads * dim, kv * dim, kv * vdim]
+    sums, bias = rand(n, sum(sizes)), rand(sum(sizes))
+    qw, kw = 1 + 0.2 * rand(dim), 1 + 0.2 * rand(dim)
+    angle = 3.0 * rand(n, max(rot // 2, 1))
+    positions = torch.tensor(list(range(3, 12)) + list(range(4)), dtype=torch.int32)
+    entry = torch.tensor([0] * 9 + [1] * 4, dtype=torch.int32)
+    table = torch.tensor([[7, 2, 5], [0, -1, -1]], dtype=torch.int32)
+
+    def turned(x):
+        if rot == 0:
+            return x
+        head = x[..., :rot]
+        a, b = (head[..., 0::2], head[..., 1::2]) if interleaved else (head[..., : rot // 2], head[..., rot // 2 :])
+        c, s = torch.cos(angle)[:, None, :], torch.sin(angle)[:, None, :]
+        pair = (a * c - b * s, b * c + a * s)
+        return torch.cat([torch.stack(pair, dim=-1).flatten(-2) if interleaved else torch.cat(pair, dim=-1), x[..., rot:]], dim=-1)
+
+    def prepared(x, w):
+        if mode == "after":
+            return pl.rms(turned(x), 1e-3) * w
+        return turned(pl.rms(x, 1e-3) * w) if mode == "before" else turned(x)
+
+    q, k, v = (sums + bias).split(sizes, dim=1)
+    want_q, want_k, want_v = prepared(q.reshape(n, heads, dim), qw), prepared(k.reshape(n, kv, dim), kw), v.reshape(n, kv, vdim)
+    dev = lambda t: t.float().cuda().contiguous()  # noqa: E731
+    proj, k_cache, v_cache, status = dev(sums), torch.zeros(pages, kv, page_size, dim, device="cuda"), torch.zeros(pages, kv, page_size, vdim, device="cuda"), status_word()
+    norm = {"none": native.PREP_NORM_NONE, "before": native.PREP_NORM_HEAD, "after": native.PREP_NORM_HEAD_AFTER}[mode]
+    ends = (sizes[0], sizes[0] + sizes[1])
+    all_bias = dev(bias)
+    native.qkv_prepare(
+        q=proj[:, : ends[0]], q_heads=heads, q_dim=dim, q_norm=(norm, dim, dev(qw)), q_out=proj, q_out_strides=(sum(sizes), dim),
+        k=proj[:, ends[0] : ends[1]], k_heads=kv, k_dim=dim, k_norm=(norm, dim, dev(kw)), v=proj[:, ends[1] :], v_dim=vdim, eps=1e-3,
+        table=dev(torch.stack([torch.cos(angle), torch.sin(angle)], dim=-1)) if rot else None, rot_dims=rot, interleaved=interleaved,
+        k_cache=k_cache, v_cache=v_cache, block_table=table.cuda(), positions=positions.cuda(), token_entry=entry.cuda(), status=status,
+        q_bias=all_bias[: ends[0]], k_bias=all_bias[ends[0] : ends[1]], v_bias=all_bias[ends[1] :])
+    assert int(status.item()) == 0
+    assert float((proj[:, : ends[0]].cpu().view(n, heads, dim) - want_q).abs().max()) <= 2e-5 * float(want_q.abs().max())
+    filled = torch.zeros(pages, page_size, dtype=torch.bool)
+    for t in range(n):
+        page, slot = int(table[entry[t], positions[t] // page_size]), int(positions[t] % page_size)
+        filled[page, slot] = True
+        assert float((k_cache[page, :, slot].cpu() - want_k[t]).abs().max()) <= 2e-5 * float(want_k.abs().max())
+        assert float((v_cache[page, :, slot].cpu() - want_v[t]).abs().max()) <= 2e-5 * float(want_v.abs().max())
+    for cache in (k_cache, v_cache):
+        assert float((cache.cpu() * ~filled[:, None, :, None]).abs().max()) == 0.0
+
+
 def test_weighted_sum_kernel():
     from forge_engine_b200.ops import native
 
